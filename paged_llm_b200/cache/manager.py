@@ -13,7 +13,8 @@ What is added here:
   head counts or head sizes) form groups with pages, tables and free queues of
   their own.  A request has one block table per group.  A group with a window
   gives pages back as soon as the window has passed them
-  (`release_behind_window`); their table entries become `NO_PAGE`.
+  (`release_behind_window`); their table entries become `NO_PAGE`.  If the window
+  keeps the first tokens of a request visible, their pages stay.
 * **State slots.**  A pool of slot numbers for per-request state of fixed size,
   taken at admission and given back with the pages.
 * The hash is a 64-bit BLAKE2 digest (stable across processes) and a hit is
@@ -59,6 +60,7 @@ class GroupSpec:
     num_pages: int
     window: int | None = None
     chunk: int | None = None        # queries read no key in front of their own chunk of this many positions
+    keep_first: int = 0             # with a window: every query reads the request's first `keep_first` keys too
 
 
 def chain_hash(prev: int | None, tokens) -> int:
@@ -317,6 +319,7 @@ class CacheManager:
         """Give back the pages that no later query of `seq` can read: with `c`
         tokens computed, a window w needs keys from position c - w + 1 on, and a
         chunked mask of size s those from c - c % s on (the next query sits at c).
+        Pages that hold one of the first `keep_first` tokens beside a window stay.
         Returns the number of pages released."""
         released = 0
         bs = self.block_size
@@ -330,7 +333,7 @@ class CacheManager:
             if spec.chunk is not None:
                 first_needed = max(first_needed, c - c % spec.chunk)
             table = self._tables(seq)[g]
-            j = 0
+            j = self.pages_for(spec.keep_first) if spec.window is not None else 0
             while j < len(table) and (j + 1) * bs <= first_needed:
                 if table[j] != NO_PAGE:
                     self.pools[g].release(table[j])

@@ -45,7 +45,7 @@ class CacheStorage:
                  num_state_slots: int = 0):
         self.page_size, self.dtype, self.device = page_size, dtype, torch.device(device)
         self.num_pages = num_pages
-        # group paged requirements: same (heads, head_dim, window, chunk) -> same group.  A mixer made of several
+        # group paged requirements: same (heads, head_dim, window, chunk, kept tokens) -> same group.  A mixer made of several
         # gives a tuple of requirements; every single need gets memory of its own and the run a view with `parts`.
         self.group_keys: list[PagedKV] = []
         counts: list[int] = []
@@ -98,7 +98,7 @@ class CacheStorage:
         return len(self.group_keys)
 
     def group_specs(self) -> list[GroupSpec]:
-        return [GroupSpec(self.num_pages, key.window, key.chunk) for key in self.group_keys]
+        return [GroupSpec(self.num_pages, key.window, key.chunk, key.keep_first) for key in self.group_keys]
 
     def page_bytes(self) -> int:
         """Bytes of one page id across all groups and layers."""

@@ -70,6 +70,10 @@ def _register_builtin() -> None:
     from .pirerax import PireraxConfig
     if "Pirerax" not in ARCHITECTURES:
         register_architecture("Pirerax", PireraxConfig, pirerax_spec)
+    from ..models.tagelorn import tagelorn_spec
+    from .tagelorn import TagelornConfig
+    if "Tagelorn" not in ARCHITECTURES:
+        register_architecture("Tagelorn", TagelornConfig, tagelorn_spec)
 
 
 _register_builtin()

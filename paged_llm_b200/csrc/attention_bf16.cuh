@@ -88,8 +88,8 @@ struct AttnShape {
 // CLUSTER: the blocks of a thread-block cluster take the splits of one (request, kv head) and
 // merge their partial results through distributed shared memory: no partials in global memory,
 // no counter, no work list.
-// MOD: the score modifiers of AttnParams (cap, bias by distance) are applied; the kernel without
-// them is the one the Llama decoder runs and carries none of their code.
+// MOD: the score modifiers of AttnParams (cap, bias by distance) are applied and the first keys may be kept beside a
+// window; the kernel without them is the one the Llama decoder runs and carries none of their code.
 // STAGES: key tiles in flight (a ring of that many K and V stages).
 // ROPE (cluster form only): q, k, v arrive as the projection left them.  The queries are rotated as
 // they are loaded (xiyiji/paged-llm llama.py:117-128: pairs i, i + d/2, float32 angles from the
@@ -140,7 +140,8 @@ __global__ void __launch_bounds__(32 * MW * NW) attn_bf16_kernel(AttnParams p) {
     const size_t v_off = (size_t)p.nkv * p.ps * d;
     // The step's own keys (the last nq of the request) are written by the kernel in front, or, with
     // ROPE, made here: then the tiles below stop in front of them and they come as a tile of their own.
-    const int own_lo = CLUSTER ? it.lk - it.nq : 0x7fffffff;
+    // (counted in places of the item's range, see attention_common.cuh)
+    const int own_lo = CLUSTER ? it.lk - it.nq - (MOD ? it.gap : 0) : 0x7fffffff;
     const int main_hi = ROPE ? min(it.key_hi, max(own_lo, it.key_lo)) : it.key_hi;
     int hi_cur = main_hi;                                  // keys at or behind it are not part of the tile at hand
 
@@ -168,7 +169,8 @@ __global__ void __launch_bounds__(32 * MW * NW) attn_bf16_kernel(AttnParams p) {
         for (int i = 0; i < LOAD_ITERS; ++i) {
             const int n = kt + j0 + i * J_STEP;
             const bool ok = e_first + i * E_STEP < E_COUNT && col_ok && n < main_hi && n < skip_from && n >= only_from;
-            const int pi = p.ps_shift >= 0 ? n >> p.ps_shift : n / p.ps;
+            const int key = MOD && n >= p.keep_first ? n + it.gap : n;
+            const int pi = p.ps_shift >= 0 ? key >> p.ps_shift : key / p.ps;
             pg[i] = ok ? bt[pi] : -1;
         }
 #pragma unroll
@@ -177,7 +179,8 @@ __global__ void __launch_bounds__(32 * MW * NW) attn_bf16_kernel(AttnParams p) {
             const int n = kt + j0 + i * J_STEP;
             if (n >= skip_from && n < main_hi) continue;          // keys past the range are still zero-filled
             if (only_from >= 0 && (n < only_from || n >= main_hi)) continue;
-            const int po = p.ps_shift >= 0 ? n & (p.ps - 1) : n % p.ps;
+            const int key = MOD && n >= p.keep_first ? n + it.gap : n;
+            const int po = p.ps_shift >= 0 ? key & (p.ps - 1) : key % p.ps;
             const bool ok = pg[i] >= 0;
             const __nv_bfloat16* src = ok ? kv_head + (size_t)pg[i] * page_stride + po * d : kv;
             cp_async16(kd + i * J_STEP * PITCH, src, ok ? 16 : 0);
@@ -301,9 +304,10 @@ __global__ void __launch_bounds__(32 * MW * NW) attn_bf16_kernel(AttnParams p) {
                 for (int j = 0; j < KPW / 8; ++j)
 #pragma unroll
                     for (int e = 0; e < 4; ++e) {
-                        const int n = kbase + 8 * j + 2 * t4 + (e & 1);
+                        const int place = kbase + 8 * j + 2 * t4 + (e & 1);
+                        const int n = MOD && place >= p.keep_first ? place + it.gap : place;
                         const int pr = pos[e >> 1];
-                        const bool vis = n < hi_cur && n <= pr && n >= first[e >> 1];
+                        const bool vis = place < hi_cur && n <= pr && (n >= first[e >> 1] || (MOD && n < p.keep_first));
                         const float s = !vis ? -INFINITY
                                         : modified ? attn_score(p, sacc[j][e], slope[e >> 1], n, pr, brow[e >> 1]) * LOG2E
                                                    : sacc[j][e] * scale_log2;
@@ -665,6 +669,8 @@ PL_EXPORT int PL_CAT(pl_attention_bf16_d, PL_DPAD)(const AttnParams* params, cud
     PL_REQUIRE(((uintptr_t)p.q & 15) == 0 && ((uintptr_t)p.kv & 15) == 0, "attention_bf16: q and kv must be 16-byte aligned");
     PL_REQUIRE(p.softcap >= 0.f, "attention_bf16: softcap=%f must not be negative", (double)p.softcap);
     PL_REQUIRE(p.chunk >= 0 && p.window >= 0, "attention_bf16: window=%d, chunk=%d", p.window, p.chunk);
+    PL_REQUIRE(p.keep_first == 0 || (p.keep_first > 0 && p.window > 0 && p.chunk == 0),
+               "attention_bf16: keep_first=%d goes with a window (%d) and without chunks (%d)", p.keep_first, p.window, p.chunk);
     // Shapes of the decode kernel, by measurement (B200; with so few warps per SM the dependent chain of a
     // warp and the shared memory a block takes decide): head sizes up to 64 walk 128 keys per tile, but 64
     // keys in a ring of three tiles where the work list says that the ranges are long (is_small == 2:
@@ -676,13 +682,13 @@ PL_EXPORT int PL_CAT(pl_attention_bf16_d, PL_DPAD)(const AttnParams* params, cud
     // prompt portions of head sizes 64 and 128 with a cap on the scores (and no bias by distance): the
     // tcgen05 kernel applies the cap itself
     static const bool no_tc_cap = getenv("PAGED_LLM_B200_NO_TCGEN05") != nullptr;
-    // (and so it does a bias by distance, read from its table per score)
-    if ((p.softcap > 0.f || p.dist_bias != nullptr) && p.slopes == nullptr && p.rope_table == nullptr && p.cluster <= 0 &&
+    // (and so it does a bias by distance, read from its table per score, and first keys kept beside a window)
+    if ((p.softcap > 0.f || p.dist_bias != nullptr || p.keep_first > 0) && p.slopes == nullptr && p.rope_table == nullptr && p.cluster <= 0 &&
         !p.is_small && p.d == PL_DPAD && !no_tc_cap && tc2::takes(p) && p.scale > 0.f)
         return tc2::launch<PL_DPAD>(p, stream);
 #endif
     PL_REQUIRE(p.dist_bias == nullptr || p.dist_len > 0, "attention_bf16: a bias by distance of %d entries", p.dist_len);
-    if (p.softcap > 0.f || p.slopes != nullptr || p.dist_bias != nullptr) {
+    if (p.softcap > 0.f || p.slopes != nullptr || p.dist_bias != nullptr || p.keep_first > 0) {
         PL_REQUIRE(p.rope_table == nullptr, "attention_bf16: score modifiers and rotary positions inside the kernel "
                                             "do not combine");
         // the score modifiers live in instantiations of their own of the mma.sync kernel (the tcgen05

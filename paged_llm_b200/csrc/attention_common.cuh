@@ -5,8 +5,12 @@
 // triton_kernel.py:22-93): request s has nq new query tokens and a context of Lk
 // keys that includes them; query token i sits at position Lk - nq + i and sees
 // keys 0..position (with a window w: the last w of them; with a chunk c: those from
-// position - position % c on); query head h reads kv
+// position - position % c on; with a window and `keep_first` k also the first k keys); query head h reads kv
 // head h / (heads / kv_heads); keys and values are read through the block table.
+//
+// A window with kept first keys leaves a gap between them and the window.  An item's key range is then counted
+// without the gap: place v < keep stands for key v, place v >= keep for key v + gap, so that ranges are cut and
+// walked as if the visible keys were one row.
 #pragma once
 
 #include "common.cuh"
@@ -18,8 +22,19 @@ struct AttnItem {
     int key_lo, key_hi;      // keys [key_lo, key_hi) are this item's share
     int split, splits;
     int scratch_base;        // first scratch row of the request (split items)
+    int gap;                 // keys left out between the kept first keys and the window (0: the range has no gap)
     bool valid;
 };
+
+// The lowest key of an item's window, taken down to 0 if it reaches the kept first keys, and the gap behind them.
+__device__ __forceinline__ int attn_window_start(const AttnParams& p, int pos_first, int& gap) {
+    const int lo = attn_first_key(p, pos_first);
+    gap = 0;
+    if (p.keep_first <= 0) return lo;
+    if (lo <= p.keep_first) return 0;
+    gap = lo - p.keep_first;
+    return lo;
+}
 
 __device__ __forceinline__ AttnItem attn_decode_item(const AttnParams& p, int idx, int block_rows, int key_align) {
     AttnItem it;
@@ -41,8 +56,12 @@ __device__ __forceinline__ AttnItem attn_decode_item(const AttnParams& p, int id
     const int last_row = min(it.rows_total, it.row_base + block_rows) - 1;
     const int pos_first = it.lk - it.nq + it.row_base / G;
     const int pos_last = it.lk - it.nq + last_row / G;
-    int lo = attn_first_key(p, pos_first);
+    int lo = attn_window_start(p, pos_first, it.gap);
     int hi = pos_last + 1;
+    if (it.gap > 0) {                    // in places from here on
+        lo = 0;
+        hi -= it.gap;
+    }
     if (it.splits > 1) {
         int chunk = (hi - lo + it.splits - 1) / it.splits;
         chunk = (chunk + key_align - 1) / key_align * key_align;
@@ -72,8 +91,11 @@ __device__ __forceinline__ AttnItem attn_cluster_item(const AttnParams& p, int s
     it.splits = splits;
     if (it.nq <= 0) return it;
     const int pos_first = it.lk - it.nq;
-    const int lo = attn_first_key(p, pos_first);
-    const int hi = it.lk;
+    int lo = attn_window_start(p, pos_first, it.gap), hi = it.lk;
+    if (it.gap > 0) {
+        lo = 0;
+        hi -= it.gap;
+    }
     int chunk = (hi - lo + splits - 1) / splits;
     chunk = (chunk + 31) / 32 * 32;
     it.key_lo = min(hi, lo + rank * chunk);

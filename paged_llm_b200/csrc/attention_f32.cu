@@ -51,9 +51,10 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(AttnParams p) {
         __syncthreads();
         for (int e = tid; e < F32_KEYS * d; e += 128) {
             const int j = e / d, c = e - j * d;
-            const int n = kt + j;
+            int n = kt + j;
             float kk = 0.f, vv = 0.f;
             if (n < it.key_hi) {
+                if (n >= p.keep_first) n += it.gap;
                 const int page = bt[n / p.ps];      // (ps_shift is for the bfloat16 kernels)
                 if (page >= 0) {
                     const size_t base = ((((size_t)page * 2) * p.nkv + kvh) * p.ps + n % p.ps) * d + c;
@@ -65,7 +66,7 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(AttnParams p) {
             Vs[j * d + c] = vv;
         }
         __syncthreads();
-        const int n = kt + lane;
+        const int place = kt + lane, n = place + (place >= p.keep_first ? it.gap : 0);
 #pragma unroll
         for (int rr = 0; rr < 4; ++rr) {
             if (pos[rr] < 0) continue;                   // uniform per warp
@@ -74,7 +75,7 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(AttnParams p) {
             float s = 0.f;
             for (int c = 0; c < d; ++c) s = fmaf(qr[c], kr[c], s);
             s = attn_score(p, s, slope[rr], n, pos[rr], brow[rr]);
-            const bool vis = n < it.key_hi && n <= pos[rr] && n >= first[rr];
+            const bool vis = place < it.key_hi && n <= pos[rr] && (n >= first[rr] || n < p.keep_first);
             const float m_new = fmaxf(m[rr], warp_max(vis ? s : -INFINITY));
             if (m_new == -INFINITY) continue;
             const float pj = vis ? expf(s - m_new) : 0.f;
@@ -164,6 +165,8 @@ int pl_attn_check(const AttnParams& p, const char* who) {
     PL_REQUIRE(p.ps > 0, "%s: page_size=%d", who, p.ps);
     PL_REQUIRE(p.window >= 0, "%s: window=%d", who, p.window);
     PL_REQUIRE(p.chunk >= 0, "%s: chunk=%d", who, p.chunk);
+    PL_REQUIRE(p.keep_first == 0 || (p.keep_first > 0 && p.window > 0 && p.chunk == 0),
+               "%s: keep_first=%d goes with a window (%d) and without chunks (%d)", who, p.keep_first, p.window, p.chunk);
     PL_REQUIRE(p.max_splits >= 1, "%s: max_splits=%d", who, p.max_splits);
     PL_REQUIRE(p.softcap >= 0.f, "%s: softcap=%f must not be negative", who, (double)p.softcap);
     PL_REQUIRE(p.dist_bias == nullptr || p.dist_len > 0, "%s: a bias by distance of %d entries", who, p.dist_len);

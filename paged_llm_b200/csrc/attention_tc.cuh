@@ -441,8 +441,16 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int kvh = blockIdx.x % p.nkv, G = p.nh / p.nkv;
     const __nv_bfloat16* q = (const __nv_bfloat16*)p.q;
-    const int key0 = it.key_lo & ~(BN - 1);                    // tiles start at multiples of 64
-    const int n_tiles = (it.key_hi - key0 + BN - 1) / BN;
+    // Keys [0, kept) and [key_lo, key_hi), by position: the first keys of the request kept beside the window, if any,
+    // and the item's window.  Tiles start at multiples of 64; the kept keys' tiles come first unless one of them is the
+    // window's first tile.
+    const int kept = it.gap > 0 ? p.keep_first : 0;
+    const int key_lo = it.gap > 0 ? p.keep_first + it.gap : it.key_lo, key_hi = it.key_hi + it.gap;
+    const int near_tile = kept > 0 && ((kept + BN - 1) & ~(BN - 1)) > key_lo ? 0 : key_lo & ~(BN - 1);
+    const int kept_tiles = near_tile > 0 ? (kept + BN - 1) / BN : 0;
+    const int n_tiles = kept_tiles + (key_hi - near_tile + BN - 1) / BN;
+    auto tile_key = [&](int t) { return t < kept_tiles ? t * BN : near_tile + (t - kept_tiles) * BN; };
+    auto in_range = [&](int n) { return n < kept || (n >= key_lo && n < key_hi); };
 
     if (warp == MMA_WARP) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n" ::"r"(saddr(&tmem_base_slot)),
@@ -489,8 +497,8 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
         uint64_t* full = values ? v_full : k_full;
         uint64_t* empty = values ? v_empty : k_empty;
         auto page_of = [&](int t) {                             // page of this lane's box of tile t, or -1
-            const int n0 = key0 + t * BN + lane * box_rows;
-            if (t >= n_tiles || lane >= boxes || n0 >= it.key_hi || n0 + box_rows <= it.key_lo) return -1;
+            const int n0 = tile_key(t) + lane * box_rows;
+            if (t >= n_tiles || lane >= boxes || n0 >= key_hi || (n0 + box_rows <= key_lo && n0 >= kept)) return -1;
             return bt[n0 >> p.ps_shift];
         };
         int pg_next = page_of(0);
@@ -504,7 +512,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
             if (lane == 0) mbar_arrive_expect(&full[s], n_ok * box_bytes * PANELS);
             __syncwarp();
             if (ok) {
-                const int n0 = key0 + t * BN + lane * box_rows;
+                const int n0 = tile_key(t) + lane * box_rows;
                 const int row = (pg * 2 * p.nkv + kvh) * p.ps + (n0 & (p.ps - 1)) + row_add;
 #pragma unroll
                 for (int c = 0; c < PANELS; ++c)
@@ -584,7 +592,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
             __syncwarp();
             fence_after_sync();
             tmem_ld64(tmem_row + b * 64, sv);
-            const int kbase = key0 + t * BN;
+            const int kbase = tile_key(t);
             if (capped) {
 #pragma unroll
                 for (int i = 0; i < 64; ++i) {
@@ -601,13 +609,13 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
                 for (int i = 0; i < 64; ++i)
                     sv[i] = fmaf(__ldg(bias_row + min(max(pos - kbase - i, 0), far)), bias_unit, sv[i]);
             }
-            const bool row_full = kbase >= it.key_lo && kbase >= first && kbase + BN <= it.key_hi && kbase + BN - 1 <= pos;
+            const bool row_full = ((kbase >= key_lo && kbase >= first) || kbase + BN <= kept) && kbase + BN <= key_hi && kbase + BN - 1 <= pos;
             const bool warp_full = __all_sync(0xffffffffu, row_full);
             if (!warp_full) {
 #pragma unroll
                 for (int i = 0; i < 64; ++i) {
                     const int n = kbase + i;
-                    const bool vis = n >= it.key_lo && n < it.key_hi && n <= pos && n >= first;
+                    const bool vis = in_range(n) && n <= pos && (n >= first || n < p.keep_first);
                     sv[i] = vis ? sv[i] : -INFINITY;
                 }
             }
@@ -656,14 +664,14 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
                     tmem_st_wait();
                 }
             }
-            if (kbase < it.key_lo || kbase + BN > it.key_hi) {
+            if (kbase + BN > kept && (kbase < key_lo || kbase + BN > key_hi)) {
                 // Value rows of keys outside the range are zeroed, so that 0 * anything stays 0 (a
                 // page may hold anything behind the last token).
                 mbar_wait(&v_full[t % STAGES], (t / STAGES) & 1);
                 unsigned char* vd = Vs + (t % STAGES) * K_BYTES;
                 for (int e = tid; e < BN * 8 * PANELS; e += SOFTMAX_WARPS * 32) {      // panels are [64 keys][8 chunks]
                     const int n = kbase + ((e >> 3) & (BN - 1));
-                    if (n < it.key_lo || n >= it.key_hi) *reinterpret_cast<uint4*>(vd + e * 16) = make_uint4(0, 0, 0, 0);
+                    if (!in_range(n)) *reinterpret_cast<uint4*>(vd + e * 16) = make_uint4(0, 0, 0, 0);
                 }
                 fence_async_smem();                                  // generic stores -> tensor-core reads
             }

@@ -35,7 +35,7 @@ HEAD_DIM_BUILDS = (16, 32, 64, 128, 256)
 
 MODULES: dict[str, list[str]] = {
     "core": ["common.cu", "elementwise.cu", "mixers.cu", "gemm_f32.cu", "gemm_skinny.cu", "gemm_tc.cu", "attention_f32.cu",
-             "sampling.cu"],
+             "sampling.cu", "token_input.cu"],
     **{f"attn_bf16_d{d}": ["common.cu", f"attention_bf16_d{d}.cu"] for d in HEAD_DIM_BUILDS},
     # decode attention whose scratch is a static array of the library (see attention_decode_static.h)
     "attn_static": ["common.cu", "attention_decode_static.cu"],
@@ -45,8 +45,10 @@ MODULES: dict[str, list[str]] = {
     "ssm": ["common.cu", "ssm.cu"],
     # several copies of the residual stream, norms in parts, PolyNorm
     "streams": ["common.cu", "streams.cu"],
-    # convolution with a gated recurrence per channel; gated linear attention
+    # convolution with a gated recurrence per channel; gated linear attention; the delta rule
     "recurrent": ["common.cu", "recurrent.cu"],
+    # the generalized delta rule and the convolution added to a mixer's input
+    "general_delta": ["common.cu", "general_delta.cu"],
 }
 
 

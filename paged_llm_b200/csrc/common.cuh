@@ -42,6 +42,11 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_float<__nv_bfloat16>(f
 __device__ __forceinline__ float gelu_tanh_f(float z) {
     return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
+// The square of relu.
+__device__ __forceinline__ float relu2_f(float z) {
+    const float r = fmaxf(z, 0.f);
+    return r * r;
+}
 __device__ __forceinline__ float silu_f(float z) { return z / (1.0f + expf(-z)); }
 // act(gate) * up of a gated feed-forward.  act 0: silu(gate) * up; 1: gelu_tanh(gate) * up; 2, the clamped form with
 // a limit L: g = min(gate, L), u = clamp(up, -L, L), g * sigmoid(1.702 g) * (u + 1).
@@ -160,6 +165,9 @@ struct AttnParams {
     // A sink in the softmax: [nh] float32 or null.  The denominator of head h also holds exp(sink[h]): a term that has
     // no key and no value, is not scaled, masked or modified, and counts once however the keys are split.
     const float* sink;
+    // With a window: > 0: the first `keep_first` keys of a request stay visible to every later query beside the window
+    // (at their true positions).  Without a window it means nothing.
+    int keep_first;
 };
 
 // What the sink adds to a row's sum of exponentials taken relative to the maximum `m` (natural-log units; -inf:

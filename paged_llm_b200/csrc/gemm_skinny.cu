@@ -44,7 +44,7 @@ struct SkinnyParams {
     int ldx, ldy, M, N, K;
     int num_blocks;              // 16-row blocks of this product
     int I;                       // SiLU: N == 2 * I
-    int act;                     // the gate's activation: 0 SiLU, 1 the tanh form of GELU
+    int act;                     // SiLU: the gate's activation, 0 SiLU, 1 the tanh form of GELU; plain bfloat16: 3 the square of relu
     int v_from_k;                // rotary: no value heads; the values are the keys before the rotation
     // rotary + cache write
     int nh, nkv, d, ps, bt_stride, num_pages, table_len, write;
@@ -462,8 +462,8 @@ __global__ void __launch_bounds__(SK_THREADS, 1) gemm_skinny_kernel(SkinnyParams
             const float lo = v[e], hi = v[2 + e];
             if (EPI == EPI_BF16) {
                 __nv_bfloat16* y = (__nv_bfloat16*)p.Y + (size_t)tok * p.ldy;
-                if (row_lo >= 0) y[row_lo] = __float2bfloat16_rn(lo);
-                if (row_hi >= 0) y[row_hi] = __float2bfloat16_rn(hi);
+                if (row_lo >= 0) y[row_lo] = __float2bfloat16_rn(p.act == 3 ? relu2_f(lo) : lo);
+                if (row_hi >= 0) y[row_hi] = __float2bfloat16_rn(p.act == 3 ? relu2_f(hi) : hi);
             } else if (EPI == EPI_F32) {
                 float* y = (float*)p.Y + (size_t)tok * p.ldy;
                 if (row_lo >= 0) y[row_lo] = lo;
@@ -605,13 +605,16 @@ PL_EXPORT int pl_gemm_skinny_supported(int M, int N, int K, int ldx) {
     return M >= 1 && M <= 16 && N >= 1 && K >= 32 && K % 32 == 0 && ldx % 8 == 0;
 }
 
+// pl_gemm_skinny: act 3 applies the square of relu to a bfloat16 output (0: none).
 // In all entry points: with part_in non-null X is the float32 residual stream [M, ldx] and the
 // operand is RMSNorm(X) * norm_w, sum(x^2) taken from part_in[K/16][16] (left by pl_gemm_skinny_add).
 
 PL_EXPORT int pl_gemm_skinny(const void* X, int ldx, const void* W, void* Y, int ldy, int M, int N, int K,
-                             int out_float32, const float* part_in, const void* norm_w, int norm_w_dtype, float eps,
+                             int out_float32, const float* part_in, const void* norm_w, int norm_w_dtype, float eps, int act,
                              cudaStream_t stream) {
     SkinnyParams p = {};
+    PL_REQUIRE(act == 0 || (act == 3 && !out_float32), "gemm_skinny: activation %d", act);
+    p.act = act;
     p.X = X;
     p.W = (const __nv_bfloat16*)W;
     p.Y = Y;

@@ -15,14 +15,15 @@ PL_EXPORT int pl_gemm_tc(const void* X, int ldx, const void* W, void* Y, int ldy
     return gemm_tc_duo_launch(X, ldx, W, Y, ldy, resid, M, N, K, epi, stream);
 }
 
-// The same with the gate's activation chosen: act 0 SiLU, 1 the tanh form of GELU (epilogue 2 only).
+// The same with an activation: act 0 SiLU, 1 the tanh form of GELU of a gate (W = [Wg; Wu]); 3: Y = relu(X W^T)^2.
 PL_EXPORT int pl_gemm_tc_act(const void* X, int ldx, const void* W, void* Y, int ldy, int M, int N, int K, int act,
                              cudaStream_t stream) {
-    return gemm_tc_duo_launch(X, ldx, W, Y, ldy, nullptr, M, N, K, TC_SILU, stream, act);
+    return gemm_tc_duo_launch(X, ldx, W, Y, ldy, nullptr, M, N, K, act == 3 ? TC_BF16 : TC_SILU, stream, act);
 }
 
 // Grouped: X [cap, K] holds rows sorted by expert in tiles of 256 (tile i belongs to expert tile_expert[i], *n_tiles
-// tiles are in use), W is [experts][N (or 2N for epilogue 2)][K]; Y [cap, ldy] in the order of X.  epi 0, 1 or 2.
+// tiles are in use), W is [experts][N (or 2N for epilogue 2)][K]; Y [cap, ldy] in the order of X.  epi 0 (with act 3: the
+// square of relu), 1 or 2.
 PL_EXPORT int pl_gemm_tc_grouped(const void* X, int ldx, const void* W, void* Y, int ldy, int cap, int N, int K, int epi,
                                  int act, float act_limit, int experts, const int* n_tiles, const int* tile_expert,
                                  cudaStream_t stream) {

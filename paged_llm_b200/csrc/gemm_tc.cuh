@@ -22,7 +22,8 @@ struct TcParams {
     int ldy, M, N, K, I;
     int epi;
     int m_tiles, n_tiles;
-    int act;                    // SiLU epilogue: the gate's activation (0 SiLU, 1 the tanh form of GELU, 2 the clamped form)
+    int act;                    // SiLU epilogue: the gate's activation (0 SiLU, 1 the tanh form of GELU, 2 the clamped form);
+                                // plain bfloat16 epilogue: 3 the square of relu, else none
     float act_limit;            // the clamped form's limit
     // Grouped form (null / 0: one W for all rows): the rows of X are sorted by expert in tiles of 256, tile mp
     // multiplies the rows of W that start at tile_expert[mp] * expert_rows, and only *m_pairs_dev tiles exist.
@@ -99,6 +100,10 @@ __device__ __forceinline__ void tc_drain_row(const TcParams& p, uint32_t acc, in
             tmem_ld32(acc + cb * 32, v);
             if (tok >= p.M) continue;
             const int n = n0 + cb * 32;
+            if (p.epi == TC_BF16 && p.act == 3) {
+#pragma unroll
+                for (int i = 0; i < 32; ++i) v[i] = relu2_f(v[i]);
+            }
             if (p.epi == TC_BF16) {
                 __nv_bfloat16* y = (__nv_bfloat16*)p.Y + (size_t)tok * p.ldy + n;
 #pragma unroll

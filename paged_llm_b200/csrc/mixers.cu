@@ -355,6 +355,94 @@ PL_EXPORT int pl_normed_qkv_write(const void* proj, int dtype, int T, int ld, co
     return 0;
 }
 
+// ------------------------------------------------------------------ unit root mean square per head + cache write
+// proj row: [q: nh*d | k: nkv*d | v: nkv*dv | ...], plus `bias` (float32, the same layout, may be null).  Every head of q
+// and k is divided by its own root mean square, x / sqrt(mean(x^2) + eps) over the d elements; Q out [T, nh*D], K and V to
+// the page slot, all padded to D with zeros.  A warp per (token, head): heads 0..nh-1 are queries, then keys, then values.
+template <typename T>
+__global__ void __launch_bounds__(256) unit_qkv_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ bias, float eps,
+                                                       T* __restrict__ q_out, T* __restrict__ kv, SlotArgs sa, int nh, int nkv, int d,
+                                                       int dv, int D, int write, int vec, long long items) {
+    pdl_launch_dependents();
+    const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (item >= items) {
+        pdl_wait();
+        return;
+    }
+    const int lane = threadIdx.x & 31, heads = nh + 2 * nkv;
+    const int t = (int)(item / heads), head = (int)(item - (long long)t * heads);
+    const int s = sa.token_seq[t];
+    const bool is_q = head < nh, is_v = head >= nh + nkv;
+    const int n = is_v ? dv : d;
+    const int col = is_v ? (nh + nkv) * d + (head - nh - nkv) * dv : head * d;
+    T* dst = nullptr;
+    if (is_q) {
+        dst = q_out + ((size_t)t * nh + head) * D;
+    } else if (write && s >= 0) {
+        const long long slot = key_slot(sa, t, s, sa.positions[t], nkv, D);
+        if (slot >= 0) dst = kv + slot + (size_t)(is_v ? head - nkv - nh : head - nh) * sa.ps * D + (is_v ? (size_t)nkv * sa.ps * D : 0);
+    }
+    pdl_wait();
+    if (dst == nullptr) return;
+    const T* src = proj + (size_t)t * ld + col;
+    const float* b = bias != nullptr ? bias + col : nullptr;
+    if (vec) {
+        // d, dv and D are multiples of 4 up to 256: a lane holds two quads of the head
+        float4 v[2];
+        float sq = 0.f;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int c = (lane + 32 * i) * 4;
+            v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (c < n && s >= 0) {
+                v[i] = Quad4<T>::load(src + c);
+                if (b != nullptr) {
+                    const float4 w = Quad4<float>::load(b + c);
+                    v[i] = make_float4(v[i].x + w.x, v[i].y + w.y, v[i].z + w.z, v[i].w + w.w);
+                }
+            }
+            sq += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+        }
+        const float f = is_v ? 1.f : 1.0f / sqrtf(warp_sum(sq) / (float)d + eps);
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const int c = (lane + 32 * i) * 4;
+            if (c < D) Quad4<T>::store(dst + c, make_float4(v[i].x * f, v[i].y * f, v[i].z * f, v[i].w * f));
+        }
+        return;
+    }
+    auto value = [&](int c) { return c < n && s >= 0 ? to_float(src[c]) + (b != nullptr ? __ldg(b + c) : 0.f) : 0.f; };
+    float sq = 0.f;
+    for (int c = lane; c < n; c += 32) {
+        const float x = value(c);
+        sq = fmaf(x, x, sq);
+    }
+    const float f = is_v ? 1.f : 1.0f / sqrtf(warp_sum(sq) / (float)d + eps);
+    for (int c = lane; c < D; c += 32) dst[c] = from_float<T>(value(c) * f);
+}
+
+PL_EXPORT int pl_unit_qkv_write(const void* proj, int dtype, int T, int ld, const float* bias, float eps, void* q_out, void* kv,
+                                const int* positions, const int* token_seq, const int* block_table, int bt_stride, int num_pages,
+                                int ps, int nh, int nkv, int d, int dv, int D, int write, cudaStream_t stream) {
+    if (T == 0) return 0;
+    PL_REQUIRE(T > 0 && nh > 0 && nkv > 0 && d > 0 && dv > 0 && D >= d && D >= dv && ps > 0 && ld >= nh * d + nkv * (d + dv),
+               "unit_qkv_write: bad sizes d=%d dv=%d D=%d ld=%d", d, dv, D, ld);
+    SlotArgs sa{positions, token_seq, block_table, bt_stride, num_pages, ps};
+    const long long items = (long long)T * (nh + 2 * nkv), blocks = (items + 7) / 8;
+    PL_REQUIRE(blocks < (1ll << 31), "unit_qkv_write: %d tokens", T);
+    const int vec = d % 4 == 0 && dv % 4 == 0 && D % 4 == 0 && D <= 256 && ld % 4 == 0 &&
+                    (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)kv | (uintptr_t)bias) & 15) == 0;
+    if (dtype == PL_F32)
+        PL_CUDA(launch_pdl(unit_qkv_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, (const float*)proj, ld, bias, eps,
+                           (float*)q_out, (float*)kv, sa, nh, nkv, d, dv, D, write, vec, items));
+    else if (dtype == PL_BF16)
+        PL_CUDA(launch_pdl(unit_qkv_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(256), 0, stream, (const __nv_bfloat16*)proj, ld,
+                           bias, eps, (__nv_bfloat16*)q_out, (__nv_bfloat16*)kv, sa, nh, nkv, d, dv, D, write, vec, items));
+    else
+        return pl_fail("unit_qkv_write: unknown dtype %d", dtype);
+    return 0;
+}
+
 // ------------------------------------------------------------------ sigmoid gate on the heads' outputs
 // out[t, h*dv + c] = o[t, h*D + c] * sigmoid(gate[t, h*dv + c]),  c < dv (the padding of a head is dropped).
 // gate null: the copy without the padding.
@@ -700,19 +788,19 @@ __global__ void __launch_bounds__(256) normed_pair_kernel(const T* __restrict__ 
             va[i] = vb[i] = make_float4(0.f, 0.f, 0.f, 0.f);
             if (c < W) {
                 va[i] = Quad4<T>::load(a + base + c);
-                vb[i] = Quad4<T>::load(b + base + c);
+                if (b != nullptr) vb[i] = Quad4<T>::load(b + base + c);
                 ssa += va[i].x * va[i].x + va[i].y * va[i].y + va[i].z * va[i].z + va[i].w * va[i].w;
                 ssb += vb[i].x * vb[i].x + vb[i].y * vb[i].y + vb[i].z * vb[i].z + vb[i].w * vb[i].w;
             }
         }
         const float ra = sa / sqrtf(block_sum(ssa, red) / (float)W + pair_eps);
-        const float rb = sb / sqrtf(block_sum(ssb, red) / (float)W + pair_eps);
+        const float rb = b != nullptr ? sb / sqrtf(block_sum(ssb, red) / (float)W + pair_eps) : 0.f;
         float ssx = 0.f;
 #pragma unroll
         for (int i = 0; i < IT; ++i) {
             const int c = (threadIdx.x + i * 256) * 4;
             if (c < W) {
-                const float4 ga = Quad4<float>::load(wa + c), gb = Quad4<float>::load(wb + c);
+                const float4 ga = Quad4<float>::load(wa + c), gb = b != nullptr ? Quad4<float>::load(wb + c) : ga;
                 float4 v = make_float4(va[i].x * ra * ga.x + vb[i].x * rb * gb.x, va[i].y * ra * ga.y + vb[i].y * rb * gb.y,
                                        va[i].z * ra * ga.z + vb[i].z * rb * gb.z, va[i].w * ra * ga.w + vb[i].w * rb * gb.w);
                 if (x != nullptr) {
@@ -740,15 +828,15 @@ __global__ void __launch_bounds__(256) normed_pair_kernel(const T* __restrict__ 
     }
     float ssa = 0.f, ssb = 0.f;
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
-        const float va = to_float(a[base + c]), vb = to_float(b[base + c]);
+        const float va = to_float(a[base + c]), vb = b != nullptr ? to_float(b[base + c]) : 0.f;
         ssa = fmaf(va, va, ssa);
         ssb = fmaf(vb, vb, ssb);
     }
     const float ra = sa / sqrtf(block_sum(ssa, red) / (float)W + pair_eps);
-    const float rb = sb / sqrtf(block_sum(ssb, red) / (float)W + pair_eps);
+    const float rb = b != nullptr ? sb / sqrtf(block_sum(ssb, red) / (float)W + pair_eps) : 0.f;
     float ssx = 0.f;
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
-        float v = to_float(a[base + c]) * ra * __ldg(wa + c) + to_float(b[base + c]) * rb * __ldg(wb + c);
+        float v = to_float(a[base + c]) * ra * __ldg(wa + c) + (b != nullptr ? to_float(b[base + c]) * rb * __ldg(wb + c) : 0.f);
         if (x != nullptr) {
             v += x[base + c];
             x[base + c] = v;
@@ -775,7 +863,7 @@ static int launch_normed_pair(const void* a, const void* b, const float* wa, con
     return 0;
 }
 
-// dtype: of a and b.  x null: sum_out gets the sum; else x is updated and y (y_dtype) gets its norm with nw (nw_dtype).
+// dtype: of a and b; b null: a alone.  x null: sum_out gets the sum; else x is updated and y (y_dtype) gets its norm with nw (nw_dtype).
 PL_EXPORT int pl_normed_pair(const void* a, const void* b, int dtype, const float* wa, const float* wb, float sa, float sb,
                              float pair_eps, float* x, float* sum_out, const void* nw, int nw_dtype, float eps, void* y,
                              int y_dtype, long long rows, int W, cudaStream_t stream) {

@@ -1,9 +1,12 @@
-// A feed-forward of routed experts: router, the list of (token, expert) pairs sorted by expert, the
+// A feed-forward of routed experts (gated, or with one matrix in front of the activation): router, the list of (token, expert) pairs sorted by expert, the
 // experts' products over that list, and the weighted sum.
 //
 //   z = W_r h (float32, a product of the kernel library);  the k largest z choose the experts;  their weights
 //   are the softmax over those k;
 //   y = sum_j weight_j * down_e(j)(act(gate_e(j) h) * up_e(j) h)  [+ sigmoid(w_s . h) * shared(h)]
+//
+// or, by scores: s = sigmoid(z) or softmax(z) over all experts, chosen with an optional correction and within the best
+// groups of experts (MoeChoice); experts without a gate are down_e(act(up_e h)).
 //
 // Nothing here looks at the batch on the host: the counts per expert stay on the device, every kernel is
 // launched for the most tiles the step can have and blocks beyond the real count leave at once, so a step
@@ -96,12 +99,20 @@ __device__ __forceinline__ void warp_argmax(const float* v, int n, int lane, flo
     if (arg >= n) arg = 0;                              // (only if every value left is NaN)
 }
 
-// Choice by sigmoid scores: s = sigmoid(z) per expert; with groups (count > 0) the experts form `count` equal groups
-// of neighbours, a group scores the sum of its `group_top` largest s, and only experts of the `keep` best groups can be
-// chosen; the k largest s among those choose the experts, and the weights are those s as they are.  One warp per token.
-__global__ void __launch_bounds__(128) moe_sigmoid_topk_kernel(const float* __restrict__ z_all, int ldz, int tokens, int E, int k,
-                                                               int count, int keep, int group_top, int* __restrict__ top_idx,
-                                                               float* __restrict__ top_w) {
+// How the router's logits become a choice and weights.
+struct MoeChoice {
+    int softmax;                // scores: 0 sigmoid(z) per expert, 1 the softmax of z over all experts
+    const float* correction;    // [E] or null: joins the scores for the choice, not for the weights
+    int count, keep, group_top; // count > 0: `count` equal groups of neighbours; a group scores the sum of its `group_top`
+                                // largest choice scores, and only experts of the `keep` best groups can be chosen
+    int renorm;                 // 1: the weights are divided by their sum (+ 1e-20)
+    float scale;                // and multiplied by this
+};
+
+// Choice by scores that are formed in front of it: the k largest choice scores among the experts that may be chosen, the
+// weights from the scores as they are.  One warp per token.
+__global__ void __launch_bounds__(128) moe_scored_topk_kernel(const float* __restrict__ z_all, int ldz, int tokens, int E, int k,
+                                                              MoeChoice mc, int* __restrict__ top_idx, float* __restrict__ top_w) {
     extern __shared__ float z_smem[];                   // per warp: scores [E], what may still be chosen [E], group scores [E]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * 4 + warp;
@@ -110,21 +121,36 @@ __global__ void __launch_bounds__(128) moe_sigmoid_topk_kernel(const float* __re
     float* pick = sc + E;
     float* gsc = pick + E;
     const float* src = z_all + (size_t)t * ldz;
-    for (int e = lane; e < E; e += 32) pick[e] = sc[e] = 1.0f / (1.0f + expf(-src[e]));
+    if (mc.softmax) {
+        float mx = -INFINITY;
+        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, src[e]);
+        mx = warp_max(mx);
+        float sum = 0.f;
+        for (int e = lane; e < E; e += 32) {
+            const float x = expf(src[e] - mx);
+            sc[e] = x;
+            sum += x;
+        }
+        sum = warp_sum(sum);
+        for (int e = lane; e < E; e += 32) sc[e] = sc[e] / sum;
+    } else {
+        for (int e = lane; e < E; e += 32) sc[e] = 1.0f / (1.0f + expf(-src[e]));
+    }
+    for (int e = lane; e < E; e += 32) pick[e] = mc.correction != nullptr ? sc[e] + __ldg(mc.correction + e) : sc[e];
     __syncwarp();
-    if (count > 0) {
-        const int size = E / count;
-        // a lane per group: the sum of the group's `group_top` largest scores, taken one after the other
-        for (int g = lane; g < count; g += 32) {
+    if (mc.count > 0) {
+        const int size = E / mc.count;
+        // a lane per group: the sum of the group's `group_top` largest choice scores, taken one after the other
+        for (int g = lane; g < mc.count; g += 32) {
             float sum = 0.f;
             int taken[8];                               // group_top <= 8
-            for (int r = 0; r < group_top && r < size; ++r) {
+            for (int r = 0; r < mc.group_top && r < size; ++r) {
                 float best = -INFINITY;
                 int arg = -1;
                 for (int i = 0; i < size; ++i) {
                     bool used = false;
                     for (int q = 0; q < r; ++q) used |= taken[q] == i;
-                    const float x = sc[g * size + i];
+                    const float x = pick[g * size + i];
                     if (!used && x > best) {
                         best = x;
                         arg = i;
@@ -137,29 +163,36 @@ __global__ void __launch_bounds__(128) moe_sigmoid_topk_kernel(const float* __re
         }
         __syncwarp();
         // the best groups stay; their score is taken out as they are found, the others' experts cannot be chosen
-        for (int r = 0; r < keep; ++r) {
+        for (int r = 0; r < mc.keep; ++r) {
             float best;
             int arg;
-            warp_argmax(gsc, count, lane, best, arg);
+            warp_argmax(gsc, mc.count, lane, best, arg);
             __syncwarp();
             if (lane == 0) gsc[arg] = -INFINITY;
             __syncwarp();
         }
         for (int e = lane; e < E; e += 32)
-            if (gsc[e / size] != -INFINITY) pick[e] = -1.0f;
+            if (gsc[e / size] != -INFINITY) pick[e] = -INFINITY;
         __syncwarp();
     }
+    float sum = 0.f;
     for (int j = 0; j < k; ++j) {
         float best;
         int arg;
         warp_argmax(pick, E, lane, best, arg);
         __syncwarp();
+        const float s = sc[arg];
+        sum += s;
         if (lane == 0) {
             top_idx[(size_t)t * k + j] = arg;
-            top_w[(size_t)t * k + j] = sc[arg];
+            top_w[(size_t)t * k + j] = s * mc.scale;    // (the sum is not known yet)
             pick[arg] = -INFINITY;
         }
         __syncwarp();
+    }
+    if (mc.renorm) {
+        const float f = mc.scale / (sum + 1e-20f);
+        for (int j = lane; j < k; j += 32) top_w[(size_t)t * k + j] = sc[top_idx[(size_t)t * k + j]] * f;
     }
 }
 
@@ -220,6 +253,11 @@ struct MoeGemm {
     float act_limit;
 };
 
+// What a product of the list writes.
+enum { MG_DOWN = 0,     // float32, times the pair's weight
+       MG_GATED = 1,    // act(A W_gate^T) * (A W_up^T) in the compute type
+       MG_ACT = 2 };    // act(A W_up^T) in the compute type
+
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void cp_async16(void* dst, const void* src, int src_bytes) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(smem_u32(dst)), "l"(src), "r"(src_bytes));
@@ -240,17 +278,17 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
 
 constexpr int MG_BN = 64, MG_BK = 64, MG_PITCH = MG_BK + 8, MG_STAGES = 3;
 
-template <int BM, bool GATED>
-constexpr int moe_gemm_smem() { return MG_STAGES * (BM + (GATED ? 2 : 1) * MG_BN) * MG_PITCH * 2; }
+template <int BM, int MODE>
+constexpr int moe_gemm_smem() { return MG_STAGES * (BM + (MODE == MG_GATED ? 2 : 1) * MG_BN) * MG_PITCH * 2; }
 
 // bfloat16 on the tensor cores (mma.sync m16n8k16, float32 accumulation).  grid: (tiles, ceil(N / 64)); a
 // block takes BM pairs of one expert and 64 columns (gated: 64 gate and the 64 matching up columns);
 // operands come in through a ring of three cp.async stages of 64 k each, zero-filled outside the matrices.
 // BM = 64: four warps of 16 rows; BM = 16 (few pairs per expert: decoding): four warps of 16 columns.
-template <int BM, bool GATED>
+template <int BM, int MODE>
 __global__ void __launch_bounds__(128) moe_gemm_bf16_kernel(MoeGemm p) {
     constexpr int BN = MG_BN, BK = MG_BK, PITCH = MG_PITCH, STAGES = MG_STAGES;
-    constexpr int NB = GATED ? 2 : 1;
+    constexpr int NB = MODE == MG_GATED ? 2 : 1;
     constexpr int WM = BM / 16, WNW = 4 / WM, WN = BN / WNW, NF = WN / 8;
     const int tile = blockIdx.x;
     if (tile >= *p.n_tiles) return;
@@ -329,16 +367,18 @@ __global__ void __launch_bounds__(128) moe_gemm_bf16_kernel(MoeGemm p) {
     for (int hh = 0; hh < 2; ++hh) {
         const int id = rows[wm * 16 + g + 8 * hh];
         if (id < 0) continue;
-        const float sc = !GATED && p.row_scale != nullptr ? p.row_scale[id] : 1.f;
+        const float sc = MODE == MG_DOWN && p.row_scale != nullptr ? p.row_scale[id] : 1.f;
 #pragma unroll
         for (int j = 0; j < NF; ++j)
 #pragma unroll
             for (int q = 0; q < 2; ++q) {
                 const int col = n0 + wn * WN + 8 * j + 2 * t4 + q;
                 if (col >= p.N) continue;
-                if (GATED) {
+                if (MODE == MG_GATED) {
                     const float v = act_mul_f(p.act, p.act_limit, acc[0][j][2 * hh + q], acc[NB - 1][j][2 * hh + q]);
                     ((__nv_bfloat16*)p.out)[(size_t)id * p.ldo + col] = __float2bfloat16_rn(v);
+                } else if (MODE == MG_ACT) {
+                    ((__nv_bfloat16*)p.out)[(size_t)id * p.ldo + col] = __float2bfloat16_rn(relu2_f(acc[0][j][2 * hh + q]));
                 } else {
                     ((float*)p.out)[(size_t)id * p.ldo + col] = acc[0][j][2 * hh + q] * sc;
                 }
@@ -349,9 +389,9 @@ __global__ void __launch_bounds__(128) moe_gemm_bf16_kernel(MoeGemm p) {
 // The same on the CUDA cores with one FFMA chain per result in k order, for float32 (true 32-bit) and for
 // bfloat16 sizes that the tensor-core form does not take.  Tiles of 16 pairs x 64 columns, 256 threads,
 // four columns each.
-template <typename T, bool GATED>
+template <typename T, int MODE>
 __global__ void __launch_bounds__(256) moe_gemm_plain_kernel(MoeGemm p) {
-    constexpr int BM = 16, BN = 64, BK = 32, NB = GATED ? 2 : 1;
+    constexpr int BM = 16, BN = 64, BK = 32, NB = MODE == MG_GATED ? 2 : 1;
     const int tile = blockIdx.x;
     if (tile >= *p.n_tiles) return;
     const int e = p.tile_expert[tile], n0 = blockIdx.y * BN;
@@ -394,17 +434,18 @@ __global__ void __launch_bounds__(256) moe_gemm_plain_kernel(MoeGemm p) {
     }
     const int id = rows[r];
     if (id < 0) return;
-    const float sc = !GATED && p.row_scale != nullptr ? p.row_scale[id] : 1.f;
+    const float sc = MODE == MG_DOWN && p.row_scale != nullptr ? p.row_scale[id] : 1.f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
         const int col = n0 + c4 + j;
         if (col >= p.N) continue;
-        if (GATED) ((T*)p.out)[(size_t)id * p.ldo + col] = from_float<T>(act_mul_f(p.act, p.act_limit, acc[0][j], acc[NB - 1][j]));
+        if (MODE == MG_GATED) ((T*)p.out)[(size_t)id * p.ldo + col] = from_float<T>(act_mul_f(p.act, p.act_limit, acc[0][j], acc[NB - 1][j]));
+        else if (MODE == MG_ACT) ((T*)p.out)[(size_t)id * p.ldo + col] = from_float<T>(relu2_f(acc[0][j]));
         else ((float*)p.out)[(size_t)id * p.ldo + col] = acc[0][j] * sc;
     }
 }
 
-// y[t] = sum_j w_j * pair_out[row_j]  (+ gate[t] * shared[t]), float32, with row_j = place[t * k + j] (null:
+// y[t] = sum_j w_j * pair_out[row_j]  (+ gate[t] * shared[t], gate null: + shared[t]), float32, with row_j = place[t * k + j] (null:
 // t * k + j) and w_j = weight[t * k + j] (null: 1, the rows are weighted already).  pair_out is float32 or (from
 // the grouped tensor-core product) bfloat16.
 __device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
@@ -419,7 +460,7 @@ __global__ void moe_combine_kernel(const TP* __restrict__ pair_out, int k, const
                                    const float* __restrict__ weight, const T* __restrict__ shared,
                                    const float* __restrict__ gate, float* __restrict__ y, int D, int vec) {
     const size_t t = blockIdx.x;
-    const float gt = shared != nullptr ? gate[t] : 0.f;
+    const float gt = shared != nullptr && gate != nullptr ? gate[t] : 1.f;
     if (vec) {
         // four columns per thread (D % 4 == 0, 16-byte aligned bases)
         for (int c = threadIdx.x * 4; c < D; c += blockDim.x * 4) {
@@ -465,18 +506,18 @@ __global__ void moe_gather_kernel(const uint4* __restrict__ A, int row_chunks, i
     for (int c = threadIdx.x; c < row_chunks; c += blockDim.x) dst[c] = ok ? src[c] : make_uint4(0, 0, 0, 0);
 }
 
-template <int BM, bool GATED>
+template <int BM, int MODE>
 int launch_moe_bf16(const MoeGemm& p, int max_tiles, cudaStream_t stream) {
-    auto kernel = moe_gemm_bf16_kernel<BM, GATED>;
+    auto kernel = moe_gemm_bf16_kernel<BM, MODE>;
     static bool attr_set[64] = {};
     int dev = 0;
     PL_CUDA(cudaGetDevice(&dev));
     PL_REQUIRE(dev >= 0 && dev < 64, "moe_gemm: device index %d is out of range", dev);
     if (!attr_set[dev]) {
-        PL_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, moe_gemm_smem<BM, GATED>()));
+        PL_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, moe_gemm_smem<BM, MODE>()));
         attr_set[dev] = true;
     }
-    kernel<<<dim3(max_tiles, (p.N + MG_BN - 1) / MG_BN), 128, moe_gemm_smem<BM, GATED>(), stream>>>(p);
+    kernel<<<dim3(max_tiles, (p.N + MG_BN - 1) / MG_BN), 128, moe_gemm_smem<BM, MODE>(), stream>>>(p);
     PL_LAUNCHED("moe_gemm_bf16");
     return 0;
 }
@@ -494,18 +535,27 @@ PL_EXPORT int pl_moe_topk(const float* z, int ldz, int tokens, int E, int k, int
     return 0;
 }
 
-PL_EXPORT int pl_moe_sigmoid_topk(const float* z, int ldz, int tokens, int E, int k, int count, int keep, int group_top,
-                                  int* top_idx, float* top_w, cudaStream_t stream) {
+// softmax: 0 sigmoid scores, 1 softmax scores; correction: [E] float32 or null; count 0: no groups.
+PL_EXPORT int pl_moe_scored_topk(const float* z, int ldz, int tokens, int E, int k, int softmax, const float* correction, int count,
+                                 int keep, int group_top, int renorm, float scale, int* top_idx, float* top_w,
+                                 cudaStream_t stream) {
     if (tokens == 0) return 0;
-    PL_REQUIRE(tokens > 0 && E > 0 && k > 0 && k <= E && E <= 1024 && ldz >= E, "moe_sigmoid_topk: tokens=%d experts=%d top=%d",
+    PL_REQUIRE(tokens > 0 && E > 0 && k > 0 && k <= E && E <= 1024 && ldz >= E, "moe_scored_topk: tokens=%d experts=%d top=%d",
                tokens, E, k);
     PL_REQUIRE(count == 0 || (count > 0 && E % count == 0 && keep >= 1 && keep <= count && group_top >= 1 && group_top <= 8 &&
                               k <= E / count * keep),
-               "moe_sigmoid_topk: %d groups of which %d stay, scored by their %d best (at most 8)", count, keep, group_top);
-    moe_sigmoid_topk_kernel<<<(tokens + 3) / 4, 128, (size_t)4 * 3 * E * sizeof(float), stream>>>(z, ldz, tokens, E, k, count, keep,
-                                                                                              group_top, top_idx, top_w);
-    PL_LAUNCHED("moe_sigmoid_topk");
+               "moe_scored_topk: %d groups of which %d stay, scored by their %d best (at most 8)", count, keep, group_top);
+    const MoeChoice mc = {softmax, correction, count, keep, group_top, renorm, scale};
+    moe_scored_topk_kernel<<<(tokens + 3) / 4, 128, (size_t)4 * 3 * E * sizeof(float), stream>>>(z, ldz, tokens, E, k, mc, top_idx,
+                                                                                             top_w);
+    PL_LAUNCHED("moe_scored_topk");
     return 0;
+}
+
+// Sigmoid scores without a correction; the weights are the scores as they are.
+PL_EXPORT int pl_moe_sigmoid_topk(const float* z, int ldz, int tokens, int E, int k, int count, int keep, int group_top,
+                                  int* top_idx, float* top_w, cudaStream_t stream) {
+    return pl_moe_scored_topk(z, ldz, tokens, E, k, 0, nullptr, count, keep, group_top, 0, 1.0f, top_idx, top_w, stream);
 }
 
 PL_EXPORT int pl_moe_align(const int* top_idx, int n_pairs, int E, int BM, int cap, int* sorted, int* tile_expert,
@@ -527,34 +577,37 @@ PL_EXPORT int pl_moe_gather(const void* A, int lda, int a_div, const int* sorted
     return 0;
 }
 
-// gated != 0: out[pair][N] = act(A W_gate^T) * (A W_up^T) in `dtype`; else out[pair][N] = (A W^T) * row_scale in float32.
+// mode 0: out[pair][N] = (A W^T) * row_scale in float32; 1: act(A W_gate^T) * (A W_up^T) in `dtype`; 2: act(A W^T) in `dtype`.
 // BM is the tile height `sorted` was made for; tensor_cores != 0 asks for the mma.sync form (bfloat16, K % 8 == 0,
 // lda % 8 == 0), which takes BM 16 or 64; the plain form takes BM 16 only.
 PL_EXPORT int pl_moe_gemm(const void* A, int lda, int a_div, const void* W, void* out, int ldo, const int* sorted,
                           const int* tile_expert, const int* n_tiles, const float* row_scale, int n_pairs, int N, int K,
-                          int gated, int act, float act_limit, int dtype, int BM, int max_tiles, int tensor_cores,
+                          int mode, int act, float act_limit, int dtype, int BM, int max_tiles, int tensor_cores,
                           cudaStream_t stream) {
     PL_REQUIRE(n_pairs > 0 && N > 0 && K > 0 && a_div > 0 && max_tiles > 0, "moe_gemm: bad sizes");
-    PL_REQUIRE(act >= 0 && act <= 2 && (act != 2 || act_limit > 0.f), "moe_gemm: unknown activation %d (limit %g)", act, act_limit);
+    PL_REQUIRE(mode == MG_DOWN || (mode == MG_GATED && act >= 0 && act <= 2 && (act != 2 || act_limit > 0.f)) || (mode == MG_ACT && act == 3),
+               "moe_gemm: mode %d with activation %d (limit %g)", mode, act, act_limit);
     MoeGemm p = {A, W, out, sorted, tile_expert, n_tiles, row_scale, lda, a_div, ldo, n_pairs, N, K, act, act_limit};
     if (tensor_cores) {
         PL_REQUIRE(dtype == PL_BF16 && K % 8 == 0 && lda % 8 == 0 && ((uintptr_t)A & 15) == 0 && ((uintptr_t)W & 15) == 0,
                    "moe_gemm: the tensor-core form takes bfloat16 with K and lda multiples of 8");
-        if (BM == 64) return gated ? launch_moe_bf16<64, true>(p, max_tiles, stream) : launch_moe_bf16<64, false>(p, max_tiles, stream);
-        if (BM == 16) return gated ? launch_moe_bf16<16, true>(p, max_tiles, stream) : launch_moe_bf16<16, false>(p, max_tiles, stream);
-        return pl_fail("moe_gemm: BM=%d", BM);
+        PL_REQUIRE(BM == 16 || BM == 64, "moe_gemm: BM=%d", BM);
+        if (mode == MG_GATED) return BM == 64 ? launch_moe_bf16<64, MG_GATED>(p, max_tiles, stream) : launch_moe_bf16<16, MG_GATED>(p, max_tiles, stream);
+        if (mode == MG_ACT) return BM == 64 ? launch_moe_bf16<64, MG_ACT>(p, max_tiles, stream) : launch_moe_bf16<16, MG_ACT>(p, max_tiles, stream);
+        return BM == 64 ? launch_moe_bf16<64, MG_DOWN>(p, max_tiles, stream) : launch_moe_bf16<16, MG_DOWN>(p, max_tiles, stream);
     }
     PL_REQUIRE(BM == 16, "moe_gemm: the plain form takes tiles of 16 pairs, not %d", BM);
     const dim3 grid(max_tiles, (N + 63) / 64);
-    if (dtype == PL_F32) {
-        if (gated) moe_gemm_plain_kernel<float, true><<<grid, 256, 0, stream>>>(p);
-        else moe_gemm_plain_kernel<float, false><<<grid, 256, 0, stream>>>(p);
-    } else if (dtype == PL_BF16) {
-        if (gated) moe_gemm_plain_kernel<__nv_bfloat16, true><<<grid, 256, 0, stream>>>(p);
-        else moe_gemm_plain_kernel<__nv_bfloat16, false><<<grid, 256, 0, stream>>>(p);
-    } else {
-        return pl_fail("moe_gemm: unknown dtype %d", dtype);
-    }
+#define MOE_PLAIN(TT)                                                                                     \
+    do {                                                                                                  \
+        if (mode == MG_GATED) moe_gemm_plain_kernel<TT, MG_GATED><<<grid, 256, 0, stream>>>(p);           \
+        else if (mode == MG_ACT) moe_gemm_plain_kernel<TT, MG_ACT><<<grid, 256, 0, stream>>>(p);          \
+        else moe_gemm_plain_kernel<TT, MG_DOWN><<<grid, 256, 0, stream>>>(p);                             \
+    } while (0)
+    if (dtype == PL_F32) MOE_PLAIN(float);
+    else if (dtype == PL_BF16) MOE_PLAIN(__nv_bfloat16);
+    else return pl_fail("moe_gemm: unknown dtype %d", dtype);
+#undef MOE_PLAIN
     PL_LAUNCHED("moe_gemm_plain");
     return 0;
 }

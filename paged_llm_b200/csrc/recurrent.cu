@@ -8,7 +8,7 @@
 //        alpha = exp(log_sigmoid(z) / tau),   S_t = diag(alpha_t) S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t
 //  * the gated delta rule, a matrix state per head:
 //        S <- g S;   w = beta (v - S^T k);   S <- S + k w^T;   o = S^T q
-//  * the norm of each head's output over its value size, times silu(gate).
+//  * the norm of each head's output over its value size, times silu or sigmoid of a gate.
 //
 // Every request of the step brings its next tokens (one when it decodes, many in a prompt portion); its state lives
 // in a slot of [slots, state_stride] floats.  The recurrences run in the order of the tokens with a fixed order of
@@ -721,13 +721,14 @@ PL_EXPORT int pl_delta_rule(float* u, int C, const void* proj, int dtype, int ld
     return 0;
 }
 
-// ------------------------------------------------------------------ norm per head, times silu(gate)
+// ------------------------------------------------------------------ norm per head, times a gate
 // out[t, h*dv + c] = o[t, h, c] / sqrt(mean_c(o[t, h, :]^2) + eps) * w[c] * silu(gate[t, h*dv + c]); one warp per
-// (token, head); `gate`: columns of a row-major tensor with row stride ldg.
+// (token, head); `gate`: columns of a row-major tensor with row stride ldg.  `w_stride` dv: the weight spans all heads,
+// w[h*dv + c] (0: one weight for all heads).  `sig`: sigmoid in place of silu.
 template <typename T>
 __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* __restrict__ o, const T* __restrict__ gate, int ldg,
                                                              const float* __restrict__ w, float eps, T* __restrict__ out,
-                                                             long long rows, int H, int dv) {
+                                                             long long rows, int H, int dv, int w_stride, int sig) {
     pdl_launch_dependents();
     pdl_wait();
     const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
@@ -744,21 +745,25 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* __rest
     const float f = 1.0f / sqrtf(sq / (float)dv + eps);
     const T* g = gate + (size_t)t * ldg + (size_t)h * dv;
     T* dst = out + (size_t)item * dv;
-    for (int c = lane; c < dv; c += 32) dst[c] = from_float<T>(orow[c] * f * __ldg(w + c) * silu_f(to_float(g[c])));
+    const float* wh = w + (size_t)h * w_stride;
+    for (int c = lane; c < dv; c += 32) {
+        const float x = to_float(g[c]);
+        dst[c] = from_float<T>(orow[c] * f * __ldg(wh + c) * (sig ? sigmoid_f(x) : silu_f(x)));
+    }
 }
 
 PL_EXPORT int pl_head_norm_gate(const float* o, const void* gate, int dtype, int ldg, const float* w, float eps, void* out,
-                                long long rows, int H, int dv, cudaStream_t stream) {
+                                long long rows, int H, int dv, int w_per_head, int sig, cudaStream_t stream) {
     if (rows == 0) return 0;
     PL_REQUIRE(rows > 0 && H > 0 && dv > 0, "head_norm_gate: bad sizes rows=%lld H=%d dv=%d", rows, H, dv);
     const long long blocks = (rows * H + 7) / 8;
     PL_REQUIRE(blocks < (1ll << 31), "head_norm_gate: %lld rows", rows);
     if (dtype == PL_F32)
         PL_CUDA(launch_pdl(head_norm_gate_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, o, (const float*)gate, ldg,
-                           w, eps, (float*)out, rows, H, dv));
+                           w, eps, (float*)out, rows, H, dv, w_per_head ? dv : 0, sig));
     else if (dtype == PL_BF16)
         PL_CUDA(launch_pdl(head_norm_gate_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(256), 0, stream, o,
-                           (const __nv_bfloat16*)gate, ldg, w, eps, (__nv_bfloat16*)out, rows, H, dv));
+                           (const __nv_bfloat16*)gate, ldg, w, eps, (__nv_bfloat16*)out, rows, H, dv, w_per_head ? dv : 0, sig));
     else
         return pl_fail("head_norm_gate: unknown dtype %d", dtype);
     return 0;

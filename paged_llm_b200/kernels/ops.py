@@ -46,7 +46,7 @@ class AttnParams(ctypes.Structure):
         ("scale", c_float), ("ps_shift", c_int), ("counters", c_void_p), ("num_pages", c_int), ("cluster", c_int),
         ("softcap", c_float), ("slopes", c_void_p), ("rope_table", c_void_p), ("rope_len", c_int),
         ("pad_seqs", c_int), ("pad_to", c_int), ("chunk", c_int), ("dist_bias", c_void_p), ("dist_len", c_int),
-        ("sink", c_void_p),
+        ("sink", c_void_p), ("keep_first", c_int),
     ]
 
 
@@ -54,12 +54,16 @@ ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}       # codes of the gate's activation
 # the routed experts' kernels also take the clamped form with a limit L:
 # g = min(gate, L), u = clamp(up, -L, L), g * sigmoid(1.702 g) * (u + 1)
 EXPERT_ACTIVATIONS = dict(ACTIVATIONS, swish_clamped=2)
+# activations without a gate, as the kernels number them
+ACT_RELU2, ACT_TANH = 3, 4
 
 
-def attention_plan_key(num_heads: int, num_kv_heads: int, window, head_dim: int, chunk=None) -> tuple:
-    """What a step's attention work lists depend on: (query heads per kv head, kv heads, window, head size) and,
-    for a chunked mask, the chunk."""
+def attention_plan_key(num_heads: int, num_kv_heads: int, window, head_dim: int, chunk=None, keep_first=0) -> tuple:
+    """What a step's attention work lists depend on: (query heads per kv head, kv heads, window, head size), for a
+    chunked mask the chunk, and for a window with kept first tokens (no chunk and) their number."""
     key = (num_heads // num_kv_heads, num_kv_heads, window, head_dim)
+    if keep_first:
+        return key + (chunk, keep_first)
     return key + (chunk,) if chunk else key
 
 
@@ -236,6 +240,79 @@ class CudaOps:
         self.launches += 1
         return out
 
+    def embedding_sinusoid(self, table: torch.Tensor, ids: torch.Tensor, scale: float, turns: torch.Tensor,
+                           positions: torch.Tensor) -> torch.Tensor:
+        """Rows of `table` times `scale` plus the sinusoidal vector of each token's position: entries 2i and 2i + 1 are
+        the sine and cosine of 2 pi * position * turns[i] (`turns` double).  float32."""
+        T, (V, H) = ids.numel(), table.shape
+        assert turns.dtype == torch.float64 and turns.is_cuda and turns.numel() == (H + 1) // 2 and table.is_contiguous()
+        out = torch.empty((T, H), dtype=torch.float32, device=self.device)
+        _check(self.core, self.core.pl_embedding_sinusoid(self._p(table), self._code(table), self._p(ids), self._p(positions),
+                                                          self._p(turns), self._p(out), T, H, V, c_float(scale), self._stream))
+        self.launches += 1
+        return out
+
+    def softcap(self, logits: torch.Tensor, cap: float) -> torch.Tensor:
+        """cap * tanh(logits / cap) in place."""
+        assert logits.dtype == torch.float32 and logits.is_contiguous()
+        _check(self.core, self.core.pl_softcap(self._p(logits), c_longlong(logits.numel()), c_float(cap), self._stream))
+        self.launches += 1
+        return logits
+
+    def add_copy(self, x: torch.Tensor, branch=None) -> torch.Tensor:
+        """x += branch in place (float32 stream; the branch may be None); returns x in the compute dtype."""
+        if self.compute_dtype == torch.float32:
+            return self.add_rows(x, branch)
+        assert x.dtype == torch.float32 and x.is_contiguous()
+        assert branch is None or (branch.shape == x.shape and branch.is_contiguous())
+        copy = torch.empty(x.shape, dtype=self.compute_dtype, device=self.device)
+        _check(self.core, self.core.pl_add_copy(self._p(x), self._p(branch), self._code(branch) if branch is not None else PL_F32,
+                                                self._p(copy), c_longlong(x.numel()), self._stream))
+        self.launches += 1
+        return copy
+
+    def token_side_gate(self, x: torch.Tensor, branch, w_gate: torch.Tensor, table: torch.Tensor, offset: int, dim: int,
+                        ids: torch.Tensor) -> torch.Tensor:
+        """x += branch (in place; a tensor or a lazy branch), then gelu_tanh(x @ w_gate^T) * table[ids, offset : offset + dim].
+        `w_gate` may have rows beyond `dim`; the result's columns there are zero."""
+        if hasattr(branch, "materialize"):
+            branch = branch.materialize(self)
+        z = self.linear(self.add_copy(x, branch), w_gate)
+        T, n = z.shape
+        assert z.is_contiguous() and table.dtype == z.dtype and table.is_contiguous() and dim <= n
+        out = torch.empty_like(z)
+        _check(self.core, self.core.pl_token_gate(self._p(z), self._code(z), self._p(table), table.shape[1], offset, dim,
+                                                  self._p(ids), table.shape[0], self._p(out), T, n, self._stream))
+        self.launches += 1
+        return out
+
+    def _act_columns(self, x: torch.Tensor, col0: int, n: int, act: int) -> torch.Tensor:
+        rows, ld = x.shape
+        assert x.is_contiguous()
+        out = torch.empty((rows, n), dtype=x.dtype, device=self.device)
+        _check(self.core, self.core.pl_act_columns(self._p(x), self._code(x), ld, col0, self._p(out), rows, n, act, self._stream))
+        self.launches += 1
+        return out
+
+    def tanh_columns(self, x: torch.Tensor, col0: int, n: int) -> torch.Tensor:
+        """tanh(x[:, col0 : col0 + n]) as a tensor of its own."""
+        return self._act_columns(x, col0, n, ACT_TANH)
+
+    def relu2_linear(self, h, w: torch.Tensor) -> torch.Tensor:
+        """relu(h @ w^T)^2: the activation sits in the product's epilogue where the product is this package's own."""
+        M, K = h.shape
+        N = w.shape[0]
+        if self._skinny_ok(h, N) and w.dtype == torch.bfloat16:
+            return self._skinny_linear(h, w, False, ACT_RELU2)
+        h = self.materialize(h)
+        if self._gemm_tc_ok(h, w, "silu") and h.is_contiguous() and N % 8 == 0:
+            out = torch.empty((M, N), dtype=torch.bfloat16, device=self.device)
+            _check(self.core, self.core.pl_gemm_tc_act(self._p(h), h.stride(0), self._p(w), self._p(out), N, M, N, K, ACT_RELU2,
+                                                       self._stream))
+            self.launches += 1
+            return out
+        return self._act_columns(self.linear(h, w), 0, N, ACT_RELU2)
+
     def rms_norm(self, x: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
         return self._norm(x, None, w, eps)
 
@@ -352,12 +429,7 @@ class CudaOps:
         N = w.shape[0]
         assert w.shape[1] == K and w.is_contiguous()
         if self._skinny_ok(h, N) and w.dtype == torch.bfloat16:
-            x, ldx, part, nw, nwc, eps = self._norm_args(h)
-            out = torch.empty((M, N), dtype=torch.float32 if out_float32 else torch.bfloat16, device=self.device)
-            _check(self.core, self.core.pl_gemm_skinny(x, ldx, self._p(w), self._p(out), N, M, N, K,
-                                                       1 if out_float32 else 0, part, nw, nwc, eps, self._stream))
-            self.launches += 1
-            return out
+            return self._skinny_linear(h, w, out_float32)
         h = self.materialize(h)
         assert h.is_contiguous()
         if self._gemm_tc_ok(h, w, "plain") and N % 8 == 0:
@@ -375,6 +447,16 @@ class CudaOps:
         if out_float32:
             return torch.mm(h, w.t(), out_dtype=torch.float32)
         return torch.nn.functional.linear(h, w)
+
+    def _skinny_linear(self, h, w, out_float32: bool, act: int = 0) -> torch.Tensor:
+        M, K = h.shape
+        N = w.shape[0]
+        x, ldx, part, nw, nwc, eps = self._norm_args(h)
+        out = torch.empty((M, N), dtype=torch.float32 if out_float32 else torch.bfloat16, device=self.device)
+        _check(self.core, self.core.pl_gemm_skinny(x, ldx, self._p(w), self._p(out), N, M, N, K,
+                                                   1 if out_float32 else 0, part, nw, nwc, eps, act, self._stream))
+        self.launches += 1
+        return out
 
     def linear_add_rms_norm(self, h, w, x, norm_w, eps):
         """x += h @ w^T (float32 stream, in place), then RMSNorm(x) * norm_w.  With few tokens
@@ -492,6 +574,21 @@ class CudaOps:
             kv.shape[0], kv.shape[3], nh, nkv, d, dv, D, 1 if has_kv else 0, 1 if write else 0, *self._rot_args(position),
             c_float(query_temperature[0] if query_temperature else 0.0), int(query_temperature[1]) if query_temperature else 0,
             self._stream))
+        self.launches += 1
+        return q
+
+    def unit_qkv_write(self, proj, bias, nh, nkv, d, dv, D, eps, ctx, kv, block_table, write=True) -> torch.Tensor:
+        """proj rows [q: nh*d | k: nkv*d | v: nkv*dv | ...] (+ `bias`, float32, the same layout): every head of q and k is
+        divided by its own root mean square; returns the queries [T, nh*D] (heads padded to D with zeros) and writes keys and
+        values, padded the same way, to their page slots."""
+        T, ld = proj.shape
+        assert proj.is_contiguous() and kv.is_contiguous() and kv.dtype == proj.dtype and kv.shape[4] == D
+        assert bias is None or (bias.dtype == torch.float32 and bias.numel() == nh * d + nkv * (d + dv))
+        q = torch.empty((T, nh * D), dtype=proj.dtype, device=self.device)
+        _check(self.core, self.core.pl_unit_qkv_write(
+            self._p(proj), self._code(proj), T, ld, self._p(bias), c_float(eps), self._p(q), self._p(kv), self._p(ctx.positions),
+            self._p(ctx.token_seq), self._p(block_table), block_table.shape[1], kv.shape[0], kv.shape[3], nh, nkv, d, dv, D,
+            1 if write else 0, self._stream))
         self.launches += 1
         return q
 
@@ -722,6 +819,49 @@ class CudaOps:
         self.launches += 2
         return o
 
+    def residual_conv(self, h: torch.Tensor, conv_w: torch.Tensor, state, ctx) -> torch.Tensor:
+        """h + conv(h) per channel in the compute dtype, causal: conv(h)_t = sum_j conv_w[j] * h_(t - taps + 1 + j).  `conv_w`
+        float32 [taps, C]; the request's last taps-1 inputs are its state slot ([taps-1][C] float32) and are replaced by the
+        new ones (state None: one tap, nothing to keep)."""
+        lib = load_module("general_delta")
+        T, C = h.shape
+        taps = conv_w.shape[0]
+        assert h.is_contiguous() and conv_w.dtype == torch.float32 and conv_w.is_contiguous() and conv_w.shape[1] == C
+        assert state is None or (state.dtype == torch.float32 and state.is_contiguous() and state.dim() == 2)
+        out = torch.empty_like(h)
+        # (a graph of mixed items replays steps of other portions than it was captured with)
+        longest = max(T if getattr(ctx, "padded", False) else int(ctx.max_q_len), 1)
+        _check(lib, lib.pl_residual_conv(self._p(h), self._code(h), C, self._p(conv_w), taps, self._p(state),
+                                         c_longlong(state.shape[1] if state is not None else 0), self._p(ctx.cu_seqlens_q),
+                                         self._p(ctx.state_slots), ctx.num_seqs, longest, self._p(out), self._stream))
+        self.launches += 1
+        return out
+
+    def general_delta_scan(self, proj, a_col0, z, w0, a_bias, H, d, decay_scale, unit_eps, state, ctx) -> torch.Tensor:
+        """The generalized delta rule's recurrence.  proj rows [r: C | k: C | v: C | ...] with the removal rates' input at
+        columns [a_col0, + C), C = H*d; z float32 [T, C] the decay's input.  Per head, with w = exp(decay_scale *
+        sigmoid(z + w0)), a = sigmoid(removal + a_bias), u = k / sqrt(sum k^2 + unit_eps):
+        S <- diag(w) S - (a u)(u^T S) + k v^T, o = S^T r.  state: [slots, H*d*d] float32 (a head's columns one after the
+        other), updated in place.  Returns o float32 [T, C]."""
+        lib = load_module("general_delta")
+        T, ld = proj.shape
+        C = H * d
+        assert proj.is_contiguous() and z.dtype == torch.float32 and z.is_contiguous() and z.shape == (T, C)
+        assert w0.dtype == torch.float32 and a_bias.dtype == torch.float32 and w0.numel() == C and a_bias.numel() == C
+        assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] == C * d
+        o = torch.empty((T, C), dtype=torch.float32, device=self.device)
+        vec = scal = None
+        if int(ctx.max_q_len) > 4 or getattr(ctx, "padded", False):
+            # longer portions: what does not depend on the state is formed for all tokens at once in front
+            vec = torch.empty((T, H, 6, d), dtype=torch.float32, device=self.device)
+            scal = torch.empty((T, H, 2), dtype=torch.float32, device=self.device)
+        _check(lib, lib.pl_general_delta(self._p(proj), self._code(proj), ld, a_col0, self._p(z), self._p(w0), self._p(a_bias), H, d,
+                                         c_float(decay_scale), c_float(unit_eps), self._p(vec), self._p(scal), self._p(state),
+                                         c_longlong(state.shape[1]), self._p(ctx.cu_seqlens_q), self._p(ctx.state_slots),
+                                         ctx.num_seqs, c_longlong(T), self._p(o), self._stream))
+        self.launches += 1 if vec is None else 2
+        return o
+
     # ---- two branches that are normed before they meet ---------------------------------
     def normed_pair_sum(self, a, b, wa, wb, sa, sb, eps) -> torch.Tensor:
         """sa * rms_norm(a) * wa + sb * rms_norm(b) * wb as float32 (norms over the row, eps inside the root)."""
@@ -745,6 +885,32 @@ class CudaOps:
         y = torch.empty((rows, W), dtype=self.compute_dtype, device=self.device)
         _check(self.core, self.core.pl_normed_pair(self._p(a), self._p(b), self._code(a), self._p(wa), self._p(wb), c_float(sa),
                                                    c_float(sb), c_float(pair_eps), self._p(x), c_void_p(0), self._p(norm_w),
+                                                   self._code(norm_w), c_float(eps), self._p(y), self._code(y),
+                                                   c_longlong(rows), W, self._stream))
+        self.launches += 1
+        return y
+
+    # ---- one branch that is normed before it joins the stream --------------------------
+    def normed_branch(self, a, wa, eps) -> torch.Tensor:
+        """rms_norm(a) * wa as float32."""
+        rows, W = a.shape
+        assert a.is_contiguous() and wa.numel() == W
+        wa = wa.float()
+        out = torch.empty((rows, W), dtype=torch.float32, device=self.device)
+        _check(self.core, self.core.pl_normed_pair(self._p(a), c_void_p(0), self._code(a), self._p(wa), c_void_p(0), c_float(1.0),
+                                                   c_float(0.0), c_float(eps), c_void_p(0), self._p(out), c_void_p(0), 0,
+                                                   c_float(0.0), c_void_p(0), 0, c_longlong(rows), W, self._stream))
+        self.launches += 1
+        return out
+
+    def normed_add_rms_norm(self, x, a, wa, branch_eps, norm_w, eps) -> torch.Tensor:
+        """x += rms_norm(a) * wa (float32 stream, in place), then RMSNorm(x) * norm_w in the compute dtype: one kernel."""
+        rows, W = x.shape
+        assert x.dtype == torch.float32 and x.is_contiguous() and a.shape == x.shape and a.is_contiguous()
+        assert wa.dtype == torch.float32 and wa.numel() == W
+        y = torch.empty((rows, W), dtype=self.compute_dtype, device=self.device)
+        _check(self.core, self.core.pl_normed_pair(self._p(a), c_void_p(0), self._code(a), self._p(wa), c_void_p(0), c_float(1.0),
+                                                   c_float(0.0), c_float(branch_eps), self._p(x), c_void_p(0), self._p(norm_w),
                                                    self._code(norm_w), c_float(eps), self._p(y), self._code(y),
                                                    c_longlong(rows), W, self._stream))
         self.launches += 1
@@ -795,23 +961,26 @@ class CudaOps:
         self.launches += 3 if cut else 1
         return o
 
-    def head_norm_gate(self, o, proj, g_col0, H, dv, norm_w, eps) -> torch.Tensor:
-        """Each head of o (float32 [T, H*dv]) divided by its root mean square over dv, times `norm_w` [dv], times
-        silu(proj[:, g_col0 : g_col0 + H*dv]); in the compute dtype."""
+    def head_norm_gate(self, o, proj, g_col0, H, dv, norm_w, eps, gate="silu") -> torch.Tensor:
+        """Each head of o (float32 [T, H*dv]) divided by its root mean square over dv, times `norm_w` ([dv] for all heads
+        or [H*dv]), times silu (or `gate` "sigmoid") of proj[:, g_col0 : g_col0 + H*dv]; in the compute dtype."""
         lib = load_module("recurrent")
         T = o.shape[0]
-        assert o.is_contiguous() and proj.is_contiguous() and norm_w.dtype == torch.float32 and norm_w.numel() == dv
+        assert o.is_contiguous() and proj.is_contiguous() and norm_w.dtype == torch.float32
+        assert norm_w.numel() in (dv, H * dv) and gate in ("silu", "sigmoid")
         out = torch.empty((T, H * dv), dtype=proj.dtype, device=self.device)
-        gate = c_void_p(proj.data_ptr() + g_col0 * proj.element_size())
-        _check(lib, lib.pl_head_norm_gate(self._p(o), gate, self._code(proj), proj.shape[1], self._p(norm_w), c_float(eps),
-                                          self._p(out), c_longlong(T), H, dv, self._stream))
+        g = c_void_p(proj.data_ptr() + g_col0 * proj.element_size())
+        _check(lib, lib.pl_head_norm_gate(self._p(o), g, self._code(proj), proj.shape[1], self._p(norm_w), c_float(eps),
+                                          self._p(out), c_longlong(T), H, dv, 1 if norm_w.numel() == H * dv else 0,
+                                          1 if gate == "sigmoid" else 0, self._stream))
         self.launches += 1
         return out
 
     # ---- routed experts ----------------------------------------------------------
     def routed_experts(self, h, w_router, w_gate_up, w_down, top_k: int, activation: str = "silu", shared=None,
                        shared_activation: str = "silu", activation_limit: float = 0.0, scoring: str = "softmax_top",
-                       groups=None) -> torch.Tensor:
+                       groups=None, gated: bool = True, shared_gate: bool = True, correction=None, renorm: bool = False,
+                       weight_scale: float = 1.0) -> torch.Tensor:
         """The feed-forward of routed experts for the step's tokens: float32 [T, D].
 
         w_router [E (+1) or more, D]: the router's rows and, with a shared expert, the row of its gate (further rows
@@ -825,29 +994,36 @@ class CudaOps:
         Nothing is read back, so the step can be captured.  `scoring` "sigmoid": the scores sigmoid(z) choose and are the
         weights as they are; `groups` (count, keep, best): only experts of the `keep` groups (of `count` equal groups
         of neighbours) with the largest sum of their `best` largest scores can be chosen.  `activation`
-        "swish_clamped" takes `activation_limit`."""
+        "swish_clamped" takes `activation_limit`.  `scoring` "softmax": the scores are the softmax over all experts.  With
+        these two, `correction` (float32 [E]) joins the scores for the choice only, `renorm` divides the weights by their
+        sum (+ 1e-20), `weight_scale` multiplies them.  Not `gated`: w_gate_up is [E, F, D] and an expert is
+        down(relu(up h)^2), the shared one likewise ([Fs, D], [D, Fs]).  Not `shared_gate`: the shared expert is added as
+        it is, and w_router has no row for its gate."""
         h = self.materialize(h)
         assert h.is_contiguous() and w_gate_up.is_contiguous() and w_down.is_contiguous() and w_router.is_contiguous()
         T, D = h.shape
         E, F2, _ = w_gate_up.shape
-        F = F2 // 2
-        assert w_down.shape == (E, D, F) and w_router.shape[0] >= E + (1 if shared is not None else 0) and w_router.shape[1] == D
+        F = F2 // 2 if gated else F2
+        gate_row = shared is not None and shared_gate
+        assert w_down.shape == (E, D, F) and w_router.shape[0] >= E + (1 if gate_row else 0) and w_router.shape[1] == D
         assert w_gate_up.dtype == h.dtype and w_down.dtype == h.dtype and w_router.dtype == h.dtype
         lib = load_module("moe")
         dev, code = self.device, self._code(h)
         pairs = T * top_k
         top_idx = torch.empty(pairs, dtype=torch.int32, device=dev)
         top_w = torch.empty(pairs, dtype=torch.float32, device=dev)
-        gate = torch.empty(T, dtype=torch.float32, device=dev) if shared is not None else None
+        gate = torch.empty(T, dtype=torch.float32, device=dev) if gate_row else None
         z = self.linear(h, w_router, out_float32=True)          # float32 logits (and the shared expert's gate)
-        if scoring == "sigmoid":
-            if shared is not None:
-                raise KernelError("routed_experts: a shared expert's gate rides with the softmax scoring only")
+        if scoring in ("sigmoid", "softmax"):
+            if gate_row:
+                raise KernelError("routed_experts: a shared expert's gate rides with the softmax over the chosen experts only")
             count, keep, best = groups if groups is not None else (0, 0, 0)
-            _check(lib, lib.pl_moe_sigmoid_topk(self._p(z), z.shape[1], T, E, top_k, count, keep, best, self._p(top_idx),
-                                                self._p(top_w), self._stream))
+            assert correction is None or (correction.dtype == torch.float32 and correction.numel() == E)
+            _check(lib, lib.pl_moe_scored_topk(self._p(z), z.shape[1], T, E, top_k, 1 if scoring == "softmax" else 0,
+                                               self._p(correction), count, keep, best, 1 if renorm else 0, c_float(weight_scale),
+                                               self._p(top_idx), self._p(top_w), self._stream))
         else:
-            _check(lib, lib.pl_moe_topk(self._p(z), z.shape[1], T, E, top_k, 1 if shared is not None else 0,
+            _check(lib, lib.pl_moe_topk(self._p(z), z.shape[1], T, E, top_k, 1 if gate_row else 0,
                                         self._p(top_idx), self._p(top_w), self._p(gate), self._stream))
         tensor_cores = h.dtype == torch.bfloat16 and D % 8 == 0 and F % 8 == 0
         # Many pairs per expert (prompt portions): the experts' products run on the tcgen05 kernel of the dense
@@ -863,23 +1039,24 @@ class CudaOps:
         place = torch.empty(pairs, dtype=torch.int32, device=dev) if grouped_tc else None
         _check(lib, lib.pl_moe_align(self._p(top_idx), pairs, E, BM, cap, self._p(sorted_pairs),
                                      self._p(tile_expert), self._p(n_tiles), self._p(place), self._stream))
-        act, lim = EXPERT_ACTIVATIONS[activation], c_float(activation_limit)
+        act, lim = EXPERT_ACTIVATIONS[activation] if gated else ACT_RELU2, c_float(activation_limit)
+        mode = 1 if gated else 2
         if grouped_tc:
             xs = torch.empty((cap, D), dtype=h.dtype, device=dev)
             _check(lib, lib.pl_moe_gather(self._p(h), D, top_k, self._p(sorted_pairs), self._p(n_tiles), BM, cap, pairs, D,
                                           self._p(xs), self._stream))
             inter = torch.empty((cap, F), dtype=h.dtype, device=dev)
             _check(self.core, self.core.pl_gemm_tc_grouped(self._p(xs), D, self._p(w_gate_up), self._p(inter), F, cap, F, D,
-                                                           2, act, lim, E, self._p(n_tiles), self._p(tile_expert), self._stream))
+                                                           2 if gated else 0, act, lim, E, self._p(n_tiles), self._p(tile_expert), self._stream))
             # (each expert's output is rounded to bfloat16, as a dense layer's branch is; the weighted sum is float32)
             pair_out = torch.empty((cap, D), dtype=torch.bfloat16, device=dev)
             _check(self.core, self.core.pl_gemm_tc_grouped(self._p(inter), F, self._p(w_down), self._p(pair_out), D, cap, D, F,
-                                                           0, act, lim, E, self._p(n_tiles), self._p(tile_expert), self._stream))
+                                                           0, 0, c_float(0.0), E, self._p(n_tiles), self._p(tile_expert), self._stream))
             self.launches += 5
         else:
             inter = torch.empty((pairs, F), dtype=h.dtype, device=dev)
             _check(lib, lib.pl_moe_gemm(self._p(h), D, top_k, self._p(w_gate_up), self._p(inter), F, self._p(sorted_pairs),
-                                        self._p(tile_expert), self._p(n_tiles), c_void_p(0), pairs, F, D, 1, act, lim, code, BM,
+                                        self._p(tile_expert), self._p(n_tiles), c_void_p(0), pairs, F, D, mode, act, lim, code, BM,
                                         max_tiles, 1 if tensor_cores else 0, self._stream))
             pair_out = torch.empty((pairs, D), dtype=torch.float32, device=dev)
             _check(lib, lib.pl_moe_gemm(self._p(inter), F, 1, self._p(w_down), self._p(pair_out), D, self._p(sorted_pairs),
@@ -888,7 +1065,8 @@ class CudaOps:
             self.launches += 4
         s = None
         if shared is not None:
-            s = self.linear(self.gated_act_linear(h, shared[0], shared_activation), shared[1])
+            inner = self.gated_act_linear(h, shared[0], shared_activation) if gated else self.relu2_linear(h, shared[0])
+            s = self.linear(inner, shared[1])
         y = torch.empty((T, D), dtype=torch.float32, device=dev)
         _check(lib, lib.pl_moe_combine(self._p(pair_out), self._code(pair_out), top_k, self._p(place),
                                        self._p(top_w) if grouped_tc else c_void_p(0),
@@ -942,10 +1120,10 @@ class CudaOps:
         return planning.is_long_context(num_requests, num_kv_heads, self.num_sms, self.MAX_SPLITS,
                                         self.MAX_CLUSTER if self.cluster_attention else 0, self.CLUSTER_KEYS, max_context)
 
-    def plan_attention(self, q_lens, k_lens, group_size, num_kv_heads, window, head_dim, chunk=None, pad_requests=None,
-                       fixed_capacity=False, pad_tokens=None) -> dict:
+    def plan_attention(self, q_lens, k_lens, group_size, num_kv_heads, window, head_dim, chunk=None, keep_first=None,
+                       pad_requests=None, fixed_capacity=False, pad_tokens=None) -> dict:
         return planning.plan_attention(
-            q_lens, k_lens, group_size, num_kv_heads, window, chunk=chunk, small_rows=self.SMALL_ROWS,
+            q_lens, k_lens, group_size, num_kv_heads, window, chunk=chunk, keep_first=keep_first, small_rows=self.SMALL_ROWS,
             large_rows=self._large_rows(head_dim), min_split_keys=self.MIN_SPLIT_KEYS, num_sms=self.num_sms,
             max_splits=self.MAX_SPLITS, pad_requests=pad_requests, fixed_capacity=fixed_capacity,
             cluster_max=self.MAX_CLUSTER if self.cluster_attention else 0, long_keys=self.CLUSTER_KEYS,
@@ -993,7 +1171,7 @@ class CudaOps:
                                     chunk=chunk)
 
     def paged_attention(self, qkv, nh, nkv, d, kv, block_table, ctx, scale, window, softcap=None, slopes=None,
-                        rope=None, chunk=None, dist_bias=None, sink=None):
+                        rope=None, chunk=None, dist_bias=None, sink=None, keep_first=0):
         """Attention of the step's tokens over the paged cache.  `softcap` (scores become
         softcap * tanh(score / softcap)) and `slopes` (a float32 tensor [nh]: head h adds
         slopes[h] * (key position - query position) to its scores) modify the scores; both off
@@ -1001,9 +1179,11 @@ class CudaOps:
         `chunk` c lets a query at position p see the keys from p - p % c on only.  `rope` (a prepared rotary encoding; only where the step runs as clusters, see
         `qkv_attention`): qkv is the unrotated projection, and the kernel rotates q and the step's own
         keys and writes those keys and values to the cache itself.  `sink` (float32 [nh]): the softmax's denominator
-        of head h also holds exp(sink[h]), a term without key or value that counts once however the keys are split."""
+        of head h also holds exp(sink[h]), a term without key or value that counts once however the keys are split.
+        `keep_first` k (with a window): every query sees the request's first k keys too."""
         T = ctx.num_tokens
-        plan = ctx.attention_plans[attention_plan_key(nh, nkv, window, d, chunk)]
+        keep_first = int(keep_first or 0) if window else 0
+        plan = ctx.attention_plans[attention_plan_key(nh, nkv, window, d, chunk, keep_first)]
         out = torch.empty((T, nh * d), dtype=qkv.dtype, device=self.device)
         p = AttnParams()
         real = sum(ctx.host.q_lens)
@@ -1021,7 +1201,7 @@ class CudaOps:
         p.nh, p.nkv, p.d, p.ps, p.num_pages = nh, nkv, d, kv.shape[3], kv.shape[0]
         p.window, p.scale, p.max_splits = int(window or 0), float(scale), plan.max_splits
         p.softcap = float(softcap or 0.0)
-        p.chunk = int(chunk or 0)
+        p.chunk, p.keep_first = int(chunk or 0), keep_first
         if slopes is not None:
             assert slopes.dtype == torch.float32 and slopes.numel() == nh and slopes.is_contiguous() and slopes.is_cuda
             p.slopes = slopes.data_ptr()
@@ -1042,7 +1222,7 @@ class CudaOps:
             lib, fn = self.core, self.core.pl_attention_f32
         p.cluster = 0
         if rope is not None:
-            if not self._runs_as_clusters(plan, ctx, nh, nkv, bf16) or softcap or slopes is not None or dist_bias is not None:
+            if not self._runs_as_clusters(plan, ctx, nh, nkv, bf16) or softcap or slopes is not None or dist_bias is not None or keep_first:
                 raise KernelError("rotary positions inside the attention kernel: only for decode steps that run as "
                                   "clusters, without score modifiers")
             assert qkv.shape[1] == (nh + 2 * nkv) * d and rope.table.is_contiguous() and rope.rotary_dim == d

@@ -97,10 +97,18 @@ def first_visible_key(pos: int, window: int | None, chunk: int | None) -> int:
     return lo
 
 
+def visible_keys(first_pos: int, context: int, window: int | None, chunk: int | None, keep_first: int | None = None) -> int:
+    """How many keys the queries from `first_pos` on walk together: from the first one's lowest key to the end of the
+    context, and the first `keep_first` keys of the request that lie in front of the window."""
+    lo = first_visible_key(first_pos, window, chunk)
+    return context - lo + (min(lo, keep_first) if window and keep_first else 0)
+
+
 def plan_attention(q_lens, k_lens, group_size: int, num_kv_heads: int, window: int | None, *, small_rows: int,
                    large_rows: int, min_split_keys: int, num_sms: int, max_splits: int = 32,
                    pad_requests: int | None = None, fixed_capacity: bool = False, cluster_max: int = 0,
-                   long_keys: int = 0, pad_tokens: int | None = None, chunk: int | None = None) -> dict:
+                   long_keys: int = 0, pad_tokens: int | None = None, chunk: int | None = None,
+                   keep_first: int | None = None) -> dict:
     """`pad_tokens` (with `fixed_capacity`, for a step of mixed items that replays a captured graph): both lists
     get the capacity of any step of that many tokens and `pad_requests` requests, filled up with items of
     request -1 that the kernels skip."""
@@ -119,8 +127,7 @@ def plan_attention(q_lens, k_lens, group_size: int, num_kv_heads: int, window: i
     for s in small_ids:
         nq, lk = q_lens[s], k_lens[s]
         first_pos = lk - nq
-        lo = first_visible_key(first_pos, window, chunk)
-        n_keys = lk - lo
+        n_keys = visible_keys(first_pos, lk, window, chunk, keep_first)
         ns = max(1, min(want, -(-n_keys // min_split_keys)))
         splits[s] = (ns, scratch_base)
         for j in range(ns):

@@ -139,7 +139,10 @@ class GatedAttention(Mixer):
     `query_temperature` (coef, every): the normed query at position p is multiplied by
     1 + coef * ln(floor((p + 1) / every) + 1), so that late queries look harder; `sink`: one learned number per query
     head (tensor `sink`) whose exponential joins the softmax's denominator, a term without key or value that is
-    neither scaled nor masked and counts once.
+    neither scaled nor masked and counts once; `head_norm`: in place of the norm over whole projections every head of q
+    and k is divided by its own root mean square, without a weight; `bias`: q, k and v have biases (tensors
+    `q_proj_bias`, ...); `keep_first` k: beside a window every query sees the request's first k tokens too, at their
+    true distances, and the cache keeps their pages.
 
     `window` w: the query at position p sees keys p-w+1 .. p.  `keep_window`: what the cache has to keep (the
     largest window of the layers that read it; a layer with `shares_cache` has no key and value projections and
@@ -151,7 +154,8 @@ class GatedAttention(Mixer):
     def __init__(self, weights: dict[str, str], hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int,
                  value_dim: int, scale: float, eps: float, window: int | None = None, keep_window: int | None = 0,
                  distance_bias: bool = False, bias_far: float = 0.0, bias_rows: int = 32, gate: bool = True,
-                 shares_cache: bool = False, sink: bool = False, position=None, query_temperature=None):
+                 shares_cache: bool = False, sink: bool = False, position=None, query_temperature=None,
+                 head_norm: bool = False, bias: bool = False, keep_first: int = 0):
         if num_heads % num_kv_heads:
             raise ValueError(f"num_heads={num_heads} is not a multiple of num_kv_heads={num_kv_heads}")
         self.hidden_size, self.num_heads, self.num_kv_heads = hidden_size, num_heads, num_kv_heads
@@ -165,6 +169,14 @@ class GatedAttention(Mixer):
         self.has_sink, self.position = bool(sink), position
         if position is not None and position.rotary_dim > head_dim:
             raise ValueError(f"a rotation of {position.rotary_dim} elements in heads of {head_dim}")
+        self.head_norm, self.bias = bool(head_norm), bool(bias)
+        if self.bias and not self.head_norm:
+            raise ValueError("biases on q, k and v come with the norm per head")
+        if self.head_norm and (shares_cache or gate or position is not None or query_temperature is not None):
+            raise ValueError("the norm per head comes without a gate, a rotation, a temperature or a shared cache")
+        self.keep_first = int(keep_first) if self.window is not None else 0
+        if self.keep_first < 0:
+            raise ValueError(f"keep_first={keep_first}")
         self.query_temperature = None
         if query_temperature is not None:
             coef, every = query_temperature
@@ -176,23 +188,29 @@ class GatedAttention(Mixer):
         if self.cache_dim > MAX_HEAD_DIM:
             raise ValueError(f"head sizes {head_dim} / {value_dim}: the attention kernels take heads of at most {MAX_HEAD_DIM}")
         self.names = weights
-        self.w_in = self.w_o = self.q_weight = self.k_weight = self.bias_by_distance = None
+        self.w_in = self.b_in = self.w_o = self.q_weight = self.k_weight = self.bias_by_distance = None
 
     def cache_requirement(self):
-        return PagedKV(self.num_kv_heads, self.cache_dim, self.keep_window)
+        return PagedKV(self.num_kv_heads, self.cache_dim, self.keep_window, keep_first=self.keep_first)
 
     def attention_plan_key(self):
-        return (self.num_heads // self.num_kv_heads, self.num_kv_heads, self.window, self.cache_dim)
+        key = (self.num_heads // self.num_kv_heads, self.num_kv_heads, self.window, self.cache_dim)
+        return key + (None, self.keep_first) if self.keep_first else key
 
     def tensor_specs(self):
         h, d, dv = self.hidden_size, self.head_dim, self.value_dim
         out = {self.names["q_proj"]: TensorSpec((self.num_heads * d, h)),
-               self.names["q_norm"]: TensorSpec((self.num_heads * d,), role="vector", init="norm"),
                self.names["o_proj"]: TensorSpec((h, self.num_heads * dv))}
+        if not self.head_norm:
+            out[self.names["q_norm"]] = TensorSpec((self.num_heads * d,), role="vector", init="norm")
         if not self.shares_cache:
             out[self.names["k_proj"]] = TensorSpec((self.num_kv_heads * d, h))
             out[self.names["v_proj"]] = TensorSpec((self.num_kv_heads * dv, h))
-            out[self.names["k_norm"]] = TensorSpec((self.num_kv_heads * d,), role="vector", init="norm")
+            if not self.head_norm:
+                out[self.names["k_norm"]] = TensorSpec((self.num_kv_heads * d,), role="vector", init="norm")
+        if self.bias:
+            for k in ("q_proj", "k_proj", "v_proj"):
+                out[self.names[k + "_bias"]] = TensorSpec((out[self.names[k]].shape[0],), role="vector", init="norm_zero")
         if self.distance_bias:
             out[self.names["rel"]] = TensorSpec((-1, self.num_heads), role="vector", draw_shape=(self.bias_rows, self.num_heads))
         if self.gate:
@@ -207,16 +225,20 @@ class GatedAttention(Mixer):
         stack = ["q_proj"] + ([] if self.shares_cache else ["k_proj", "v_proj"]) + (["g_proj"] if self.gate else [])
         self.w_in = torch.cat([tensors[self.names[k]] for k in stack], dim=0).contiguous()
         self.w_o = tensors[self.names["o_proj"]].contiguous()
-        self.q_weight = tensors[self.names["q_norm"]].float().contiguous()
-        self.k_weight = None if self.shares_cache else tensors[self.names["k_norm"]].float().contiguous()
+        if not self.head_norm:
+            self.q_weight = tensors[self.names["q_norm"]].float().contiguous()
+            self.k_weight = None if self.shares_cache else tensors[self.names["k_norm"]].float().contiguous()
+        if self.bias:
+            self.b_in = torch.cat([tensors[self.names[k + "_bias"]].float() for k in ("q_proj", "k_proj", "v_proj")]).contiguous()
         if self.distance_bias:
             rel = tensors[self.names["rel"]].float()
             if rel.shape[0] < 2 or not self.bias_far > rel.shape[0] // 2:
                 raise ValueError(f"a bias table of {rel.shape[0]} rows needs at least two rows and a farthest distance "
                                  f"above {rel.shape[0] // 2}, not {self.bias_far}")
-            # all distances from the farthest on share a row; no query reaches further back than its window
+            # all distances from the farthest on share a row; no query reaches further back than its window, unless the
+            # first tokens are kept beside it
             far = int(math.ceil(self.bias_far)) + 1
-            length = min(self.window, far) if self.window else far
+            length = min(self.window, far) if self.window and not self.keep_first else far
             rows = log_distance_buckets(rel.shape[0], self.bias_far, length)
             self.bias_by_distance = rel[torch.tensor(rows, device=rel.device)].t().contiguous()      # [heads, length]
 
@@ -228,11 +250,17 @@ class GatedAttention(Mixer):
         nh, nkv, d, dv, D = self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim, self.cache_dim
         block_table = ctx.block_tables[cache.group]
         proj = ops.linear(h, self.w_in)
-        q = ops.normed_qkv_write(proj, nh, nkv, d, dv, D, self.q_weight, self.k_weight, self.eps, ctx, cache.kv,
-                                 block_table, has_kv=not self.shares_cache, write=cache.owner and not self.shares_cache,
-                                 position=self.position, query_temperature=self.query_temperature)
+        if self.head_norm:
+            q = ops.unit_qkv_write(proj, self.b_in, nh, nkv, d, dv, D, self.eps, ctx, cache.kv, block_table, write=cache.owner)
+        else:
+            q = ops.normed_qkv_write(proj, nh, nkv, d, dv, D, self.q_weight, self.k_weight, self.eps, ctx, cache.kv,
+                                     block_table, has_kv=not self.shares_cache, write=cache.owner and not self.shares_cache,
+                                     position=self.position, query_temperature=self.query_temperature)
+        extra = {"keep_first": self.keep_first} if self.keep_first else {}
         o = ops.paged_attention(q, nh, nkv, D, cache.kv, block_table, ctx, self.scale, self.window,
-                                dist_bias=self.bias_by_distance, sink=self.sink)
+                                dist_bias=self.bias_by_distance, sink=self.sink, **extra)
+        if not self.gate and D == dv:
+            return LazyLinear(o, self.w_o)
         g0 = nh * d + (0 if self.shares_cache else nkv * (d + dv))
         o = ops.head_gate(o, nh, D, dv, proj[:, g0:g0 + nh * dv] if self.gate else None)
         return LazyLinear(o, self.w_o)

@@ -106,12 +106,15 @@ class PagedKV:
     """The mixer keeps a key and a value vector per token, in pages.
     `window`: only the last `window` tokens are ever read (None: all).
     `chunk`: positions are cut into chunks of this many, counted from 0, and a query reads
-    only the keys of its own chunk (None: no such cut)."""
+    only the keys of its own chunk (None: no such cut).
+    `keep_first`: with a window, the first `keep_first` tokens of a request are read by every
+    later query as well."""
 
     num_kv_heads: int
     head_dim: int
     window: int | None = None
     chunk: int | None = None
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)

@@ -8,7 +8,8 @@ from __future__ import annotations
 
 import torch
 
-from .base import Block, LazyNormed, StreamBranch, TensorSpec, branch_args, materialize, register_block
+from .base import (NORMS, Block, LazyLinear, LazyNormed, PartSpec, StreamBranch, TensorSpec, branch_args, make_part,
+                   register_block)
 
 
 @register_block("pre_norm")
@@ -48,6 +49,56 @@ class SandwichNormBlock(Block):
         if not self.feed_forward.accepts_lazy_input:
             h = ctx.ops.materialize(h)
         return x, LazyNormed(self.feed_forward.forward(h, ctx), self.norms["behind_ffn"])
+
+
+@register_block("pre_norm_token_side")
+class TokenSideBlock(PreNormBlock):
+    """A pre-norm layer with an input of its own from the token, after the feed-forward (or, without one, after the mixer):
+
+        g = gelu_tanh(W_gate x) * table[token, offset : offset + dim];   x += rms_norm(W_proj g) * n
+
+    The gate reads the stream itself, without a norm.  `table` is one tensor for all layers, each reading its own part of a
+    row.  The last sum travels as a branch with its norm (`LazyNormed`), so the norm that follows does both norms and the
+    sum in one kernel."""
+
+    def __init__(self, mixer, feed_forward, norms, weights: dict, hidden_size: int, vocab_size: int, dim: int, offset: int,
+                 table_width: int, eps: float):
+        super().__init__(mixer, feed_forward, norms)
+        if not 0 <= offset <= offset + dim <= table_width:
+            raise ValueError(f"columns {offset}..{offset + dim} of a token table of {table_width}")
+        self.hidden_size, self.vocab_size, self.dim, self.offset, self.table_width = hidden_size, vocab_size, dim, offset, table_width
+        self.names = weights
+        self.side_norm = make_part(NORMS, "norm", PartSpec("rms_norm", dict(dim=hidden_size, eps=eps), {"weight": weights["norm"]}))
+        self.w_gate = self.w_proj = self.table = None
+
+    def _parts(self):
+        return super()._parts() + [self.side_norm]
+
+    def tensor_specs(self):
+        out, n = super().tensor_specs(), self.names
+        out[n["table"]] = TensorSpec((self.vocab_size, self.table_width))
+        out[n["gate"]] = TensorSpec((self.dim, self.hidden_size))
+        out[n["proj"]] = TensorSpec((self.hidden_size, self.dim))
+        return out
+
+    def load(self, tensors):
+        super().load(tensors)
+        n = self.names
+        self.side_norm.weight = self.side_norm.weight.float()
+        self.table = tensors[n["table"]].contiguous()
+        gate, proj = tensors[n["gate"]], tensors[n["proj"]]
+        # the inner size filled up with zeros to a multiple of 8: both products then take an aligned form
+        pad = -self.dim % 8
+        self.w_gate = torch.nn.functional.pad(gate, (0, 0, 0, pad)).contiguous()
+        self.w_proj = torch.nn.functional.pad(proj, (0, pad)).contiguous()
+
+    def bytes_read_per_step(self):
+        return super().bytes_read_per_step() + sum(w.numel() * w.element_size() for w in (self.w_gate, self.w_proj))
+
+    def forward(self, x, pending, ctx, cache):
+        x, pending = super().forward(x, pending, ctx, cache)
+        g = ctx.ops.token_side_gate(x, pending, self.w_gate, self.table, self.offset, self.dim, ctx.input_ids)
+        return x, LazyNormed(LazyLinear(g, self.w_proj), self.side_norm)
 
 
 @register_block("hyper_connections")

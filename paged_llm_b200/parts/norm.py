@@ -36,6 +36,10 @@ class RMSNorm(Norm):
     def bytes_read_per_step(self):
         return self.weight.numel() * self.weight.element_size()
 
+    def apply(self, t: torch.Tensor, ops) -> torch.Tensor:
+        """The norm of a tensor that is not the stream (the norm behind a branch), float32."""
+        return ops.normed_branch(t, self.weight, self.eps)
+
     def forward(self, x, ctx):
         return self.add_forward(x, None, ctx)
 
@@ -55,6 +59,10 @@ class RMSNorm(Norm):
             # both norms of the pair, the residual sum and this norm in one kernel
             return ctx.ops.normed_pair_add_rms_norm(x, branch.a, branch.b, branch.weights[0], branch.weights[1],
                                                     branch.scales[0], branch.scales[1], branch.eps, self.weight, self.eps)
+        if isinstance(branch, LazyNormed) and isinstance(branch.norm, RMSNorm) and branch.norm.groups == branch.norm.streams == 1:
+            # the branch's own norm, the residual sum and this norm in one kernel
+            return ctx.ops.normed_add_rms_norm(x, materialize(branch.branch, ctx.ops), branch.norm.weight, branch.norm.eps,
+                                               self.weight, self.eps)
         if isinstance(branch, LazyPair) or (isinstance(branch, LazyLinear) and branch.bias is not None):
             branch = branch.materialize(ctx.ops)
         if isinstance(branch, LazyLinear):

@@ -9,7 +9,11 @@ Options: `scoring` "sigmoid": every expert scores s = sigmoid(z) by itself, the 
 weights are those scores as they are (not renormalised).  `groups` (count, keep): the experts form `count` equal groups
 of neighbours, a group scores the sum of its `group_score_top` largest scores, and only experts of the `keep` best
 groups can be chosen.  `activation` "swish_clamped" with `activation_limit` L: g = min(gate, L), u = clamp(up, -L, L),
-the expert's inner vector is g * sigmoid(1.702 g) * (u + 1).
+the expert's inner vector is g * sigmoid(1.702 g) * (u + 1).  `scoring` "softmax": the scores are the softmax of z over
+all experts.  `correction`: one learned number per expert joins its score for the choice (and in the groups' scores), not
+for the weights.  `renorm`: the chosen scores are divided by their sum (+ 1e-20); `weight_scale` multiplies the weights.
+`gated` False: an expert, and the shared one, is down(act(up h)) with the square of relu ("relu2") as act.  `shared_gate`
+False: the shared expert is added as it is.
 
 The experts' matrices are stacked when the weights are taken ([E, 2F, D] gate over up, and
 [E, D, F]), the shared gate's row rides behind the router's, and the kernel library does the
@@ -24,6 +28,7 @@ from .base import FeedForward, TensorSpec, register_feed_forward
 from .mlp import ACTIVATIONS
 
 EXPERT_ACTIVATIONS = ACTIVATIONS + ("swish_clamped",)
+UNGATED_ACTIVATIONS = ("relu2",)
 
 
 @register_feed_forward("routed_mlp")
@@ -31,24 +36,32 @@ class RoutedMLP(FeedForward):
     def __init__(self, weights: dict[str, str], hidden_size: int, expert_size: int, num_experts: int, top_k: int,
                  activation: str = "silu", shared_size: int | None = None, shared_activation: str | None = None,
                  activation_limit: float | None = None, scoring: str = "softmax_top", groups=None,
-                 group_score_top: int = 2):
+                 group_score_top: int = 2, gated: bool = True, shared_gate: bool = True, correction: bool = False,
+                 renorm: bool = False, weight_scale: float = 1.0):
         if not 1 <= top_k <= num_experts:
             raise ValueError(f"top_k={top_k} of {num_experts} experts")
         for a in (activation, shared_activation or activation):
-            if a not in EXPERT_ACTIVATIONS:
-                raise ValueError(f"activation {a!r} is not implemented ({', '.join(EXPERT_ACTIVATIONS)} only)")
+            known = EXPERT_ACTIVATIONS if gated else UNGATED_ACTIVATIONS
+            if a not in known:
+                raise ValueError(f"activation {a!r} is not implemented ({', '.join(known)} only)")
         if activation == "swish_clamped" and not (activation_limit is not None and activation_limit > 0):
             raise ValueError("the clamped activation needs a positive activation_limit")
-        if shared_size is not None and (shared_activation or activation) not in ACTIVATIONS:
+        if gated and shared_size is not None and (shared_activation or activation) not in ACTIVATIONS:
             raise ValueError(f"a shared expert takes the activations {', '.join(ACTIVATIONS)} only")
-        if scoring not in ("softmax_top", "sigmoid"):
-            raise ValueError(f"scoring {scoring!r} is not implemented (softmax_top and sigmoid only)")
+        if scoring not in ("softmax_top", "sigmoid", "softmax"):
+            raise ValueError(f"scoring {scoring!r} is not implemented (softmax_top, sigmoid and softmax only)")
+        if scoring == "softmax_top" and (correction or renorm or weight_scale != 1.0):
+            raise ValueError("a correction, renormalised weights and their scale go with sigmoid and softmax scores")
+        if shared_size is not None and shared_gate and scoring != "softmax_top":
+            raise ValueError("a shared expert's gate rides with the softmax over the chosen experts only")
+        self.gated, self.shared_gate, self.has_correction = bool(gated), bool(shared_gate), bool(correction)
+        self.renorm, self.weight_scale, self.correction = bool(renorm), float(weight_scale), None
         if groups is not None:
             count, keep = (int(g) for g in groups)
             if count < 1 or num_experts % count or not 1 <= keep <= count or top_k > num_experts // count * keep:
                 raise ValueError(f"{num_experts} experts in {count} groups of which {keep} are kept, top_k={top_k}")
-            if scoring != "sigmoid":
-                raise ValueError("groups of experts are chosen by sigmoid scores")
+            if scoring == "softmax_top":
+                raise ValueError("groups of experts are chosen by sigmoid or softmax scores")
             groups = (count, keep, int(group_score_top))
         self.activation_limit = float(activation_limit) if activation_limit is not None else 0.0
         self.scoring, self.groups = scoring, groups
@@ -57,7 +70,7 @@ class RoutedMLP(FeedForward):
         self.shared_activation = shared_activation or activation
         self.names = weights
         self.w_router = None          # [E (+1) and padding, D]: the router's rows, then the shared expert's gate
-        self.w_gate_up = None         # [E, 2F, D]
+        self.w_gate_up = None         # [E, 2F, D]; without a gate [E, F, D]
         self.w_down = None            # [E, D, F]
         self.shared = None            # (gate over up [2Fs, D], down [D, Fs])
 
@@ -65,26 +78,36 @@ class RoutedMLP(FeedForward):
         d, f = self.hidden_size, self.expert_size
         out = {self.names["router"]: TensorSpec((self.num_experts, d))}
         for e in range(self.num_experts):
-            out[self.names[f"e{e}.gate"]] = TensorSpec((f, d))
+            if self.gated:
+                out[self.names[f"e{e}.gate"]] = TensorSpec((f, d))
             out[self.names[f"e{e}.up"]] = TensorSpec((f, d))
             out[self.names[f"e{e}.down"]] = TensorSpec((d, f))
+        if self.has_correction:
+            out[self.names["correction"]] = TensorSpec((self.num_experts,), role="vector", init="norm_zero")
         if self.shared_size is not None:
             s = self.shared_size
-            out[self.names["shared.gate"]] = TensorSpec((s, d))
+            if self.gated:
+                out[self.names["shared.gate"]] = TensorSpec((s, d))
             out[self.names["shared.up"]] = TensorSpec((s, d))
             out[self.names["shared.down"]] = TensorSpec((d, s))
-            out[self.names["shared.sg"]] = TensorSpec((1, d))
+            if self.shared_gate:
+                out[self.names["shared.sg"]] = TensorSpec((1, d))
         return out
 
     def load(self, tensors):
         t, n, E = tensors, self.names, self.num_experts
-        self.w_gate_up = torch.stack([torch.cat([t[n[f"e{e}.gate"]], t[n[f"e{e}.up"]]], dim=0) for e in range(E)]).contiguous()
+        def first(prefix):          # what stands in front of the activation: gate over up, or up alone
+            return torch.cat([t[n[prefix + "gate"]], t[n[prefix + "up"]]], dim=0) if self.gated else t[n[prefix + "up"]]
+
+        self.w_gate_up = torch.stack([first(f"e{e}.") for e in range(E)]).contiguous()
         self.w_down = torch.stack([t[n[f"e{e}.down"]] for e in range(E)]).contiguous()
         router = [t[n["router"]]]
         if self.shared_size is not None:
-            router.append(t[n["shared.sg"]])
-            self.shared = (torch.cat([t[n["shared.gate"]], t[n["shared.up"]]], dim=0).contiguous(),
-                           t[n["shared.down"]].contiguous())
+            if self.shared_gate:
+                router.append(t[n["shared.sg"]])
+            self.shared = (first("shared.").contiguous(), t[n["shared.down"]].contiguous())
+        if self.has_correction:
+            self.correction = t[n["correction"]].float().contiguous()
         rows = sum(r.shape[0] for r in router)
         if rows % 8:
             # rows of zeros up to a multiple of 8: the library's product of the logits then takes an aligned form
@@ -102,4 +125,15 @@ class RoutedMLP(FeedForward):
     def forward(self, h, ctx):
         return ctx.ops.routed_experts(h, self.w_router, self.w_gate_up, self.w_down, self.top_k, self.activation,
                                       shared=self.shared, shared_activation=self.shared_activation,
-                                      activation_limit=self.activation_limit, scoring=self.scoring, groups=self.groups)
+                                      activation_limit=self.activation_limit, scoring=self.scoring, groups=self.groups,
+                                      **self._options())
+
+    def _options(self) -> dict:
+        out = {}
+        if not self.gated:
+            out["gated"] = False
+        if self.shared is not None and not self.shared_gate:
+            out["shared_gate"] = False
+        if self.scoring != "softmax_top" and (self.correction is not None or self.renorm or self.weight_scale != 1.0):
+            out.update(correction=self.correction, renorm=self.renorm, weight_scale=self.weight_scale)
+        return out

@@ -33,6 +33,34 @@ class TorchOps:
         self._count("embedding")
         return (table[ids.long()].float() * scale).repeat(1, copies)
 
+    def embedding_sinusoid(self, table, ids, scale, turns, positions):
+        self._count("embedding_sinusoid")
+        W = table.shape[1]
+        ang = 2.0 * np.pi * positions.double()[:, None] * turns[None, :]
+        vec = torch.stack([torch.sin(ang), torch.cos(ang)], dim=-1).reshape(len(ids), -1)[:, :W]
+        return table[ids.long()].float() * scale + vec.float()
+
+    def softcap(self, logits, cap):
+        self._count("softcap")
+        return cap * torch.tanh(logits / cap)
+
+    def token_side_gate(self, x, branch, w_gate, table, offset, dim, ids):
+        self._count("token_side_gate")
+        if hasattr(branch, "materialize"):
+            branch = branch.materialize(self)
+        x += branch.float()
+        z = torch.nn.functional.gelu(self.linear(x.to(self.compute_dtype), w_gate).float(), approximate="tanh")
+        out = torch.zeros_like(z)
+        out[:, :dim] = z[:, :dim] * table[ids.long()][:, offset:offset + dim].float()
+        return out.to(self.compute_dtype)
+
+    def tanh_columns(self, x, col0, n):
+        self._count("tanh_columns")
+        return torch.tanh(x[:, col0:col0 + n].float()).to(self.compute_dtype)
+
+    def relu2_linear(self, h, w):
+        return (self.linear(h, w).float().clamp(min=0.0) ** 2).to(self.compute_dtype)
+
     def stream_norm(self, x, streams, branch, mix, out, w_in, norm_w, groups, eps, branch2=None, scales=None, biases=None):
         self._count("stream_norm")
         rows, width = x.shape[0], x.shape[1] // streams
@@ -128,21 +156,25 @@ class TorchOps:
         return self.act_mul(self.linear(h, w_gate_up), activation)
 
     def routed_experts(self, h, w_router, w_gate_up, w_down, top_k, activation="silu", shared=None,
-                       shared_activation="silu", activation_limit=0.0, scoring="softmax_top", groups=None):
+                       shared_activation="silu", activation_limit=0.0, scoring="softmax_top", groups=None, gated=True,
+                       shared_gate=True, correction=None, renorm=False, weight_scale=1.0):
         self._count("routed_experts")
         E = w_gate_up.shape[0]
         z = h.float() @ w_router.float().T              # (rows behind the experts' and the gate's are padding)
-        if scoring == "sigmoid":
-            sc = torch.sigmoid(z[:, :E])
-            pick = sc
+        if scoring in ("sigmoid", "softmax"):
+            sc = torch.sigmoid(z[:, :E]) if scoring == "sigmoid" else torch.softmax(z[:, :E], dim=-1)
+            pick = sc if correction is None else sc + correction
             if groups is not None:
                 count, keep, best = groups
-                per = sc.view(-1, count, E // count)
+                per = pick.view(-1, count, E // count)
                 group_score = per.topk(min(best, E // count), dim=-1).values.sum(-1)
                 kept = torch.zeros_like(group_score, dtype=torch.bool).scatter_(1, group_score.topk(keep, dim=-1).indices, True)
-                pick = sc.masked_fill(~kept[:, :, None].expand_as(per).reshape(-1, E), -1.0)
+                pick = pick.masked_fill(~kept[:, :, None].expand_as(per).reshape(-1, E), float("-inf"))
             idx = torch.topk(pick, top_k, dim=-1).indices
             wt = sc.gather(1, idx)
+            if renorm:
+                wt = wt / (wt.sum(-1, keepdim=True) + 1e-20)
+            wt = wt * weight_scale
         else:
             top, idx = torch.topk(z[:, :E], top_k, dim=-1)
             wt = torch.softmax(top, dim=-1)
@@ -150,11 +182,13 @@ class TorchOps:
         for t in range(h.shape[0]):
             for j in range(top_k):
                 e = int(idx[t, j])
-                inter = self.act_mul(self.linear(h[t:t + 1], w_gate_up[e]), activation, activation_limit)
+                inter = (self.act_mul(self.linear(h[t:t + 1], w_gate_up[e]), activation, activation_limit) if gated
+                         else self.relu2_linear(h[t:t + 1], w_gate_up[e]))
                 y[t] += wt[t, j] * self.linear(inter, w_down[e]).float()[0]
         if shared is not None:
-            s = self.linear(self.gated_act_linear(h, shared[0], shared_activation), shared[1]).float()
-            y += torch.sigmoid(z[:, E:E + 1]) * s
+            inner = self.gated_act_linear(h, shared[0], shared_activation) if gated else self.relu2_linear(h, shared[0])
+            s = self.linear(inner, shared[1]).float()
+            y += torch.sigmoid(z[:, E:E + 1]) * s if shared_gate else s
         return y
 
     def materialize(self, h):
@@ -219,15 +253,16 @@ class TorchOps:
                 kv[page, 1, :, p % ps, :] = v[t].to(kv.dtype)
 
     # ---- attention -------------------------------------------------------------
-    def plan_attention(self, q_lens, k_lens, group_size, num_kv_heads, window, head_dim, chunk=None, pad_requests=None,
-                       fixed_capacity=False, pad_tokens=None):
-        return plan_attention(q_lens, k_lens, group_size, num_kv_heads, window, chunk=chunk, small_rows=16, large_rows=64,
+    def plan_attention(self, q_lens, k_lens, group_size, num_kv_heads, window, head_dim, chunk=None, keep_first=None,
+                       pad_requests=None, fixed_capacity=False, pad_tokens=None):
+        return plan_attention(q_lens, k_lens, group_size, num_kv_heads, window, chunk=chunk, keep_first=keep_first, small_rows=16, large_rows=64,
                               min_split_keys=128, num_sms=4, pad_requests=pad_requests, fixed_capacity=fixed_capacity,
                               pad_tokens=pad_tokens)
 
     def paged_attention(self, qkv, nh, nkv, d, kv, block_table, ctx, scale, window, softcap=None, slopes=None,
-                        chunk=None, dist_bias=None, sink=None):
+                        chunk=None, dist_bias=None, sink=None, keep_first=0):
         self._count("paged_attention")
+        keep_first = keep_first if window else 0
         T = ctx.num_tokens
         q = qkv[:, :nh * d].view(T, nh, d).float()
         out = torch.zeros(T, nh * d, dtype=self.compute_dtype, device=qkv.device)
@@ -240,6 +275,8 @@ class TorchOps:
             if chunk:
                 lo = max(lo, first - first % chunk)
             idx = torch.arange(lo, lk)
+            if keep_first:
+                idx = torch.cat([torch.arange(min(lo, keep_first)), idx])
             pages = block_table[s, (idx // ps)].long()
             assert (pages >= 0).all(), "read of a page that was given back"
             k = kv[pages, 0, :, idx % ps, :].float()       # [n, nkv, d]
@@ -258,7 +295,7 @@ class TorchOps:
                 scores = scores + dist_bias.float().cpu()[:, dist]
             hidden = idx[None, :] > qpos[:, None]
             if window:
-                hidden |= idx[None, :] <= qpos[:, None] - window
+                hidden |= (idx[None, :] <= qpos[:, None] - window) & (idx[None, :] >= keep_first)
             if chunk:
                 hidden |= idx[None, :] < (qpos - qpos % chunk)[:, None]
             scores = scores.masked_fill(hidden[None], float("-inf"))
@@ -397,6 +434,55 @@ class TorchOps:
                     out[t, h] = Sh @ qt
         return out.reshape(T, H * dv)
 
+    def residual_conv(self, h, conv_w, state, ctx):
+        self._count("residual_conv")
+        taps, C = conv_w.shape
+        hist = taps - 1
+        out = torch.zeros(h.shape, dtype=torch.float32)
+        cu = ctx.host.cu
+        for s, slot in enumerate(ctx.host.state_slots):
+            rows = h[cu[s]:cu[s + 1]].float()
+            nq = rows.shape[0]
+            seq = rows
+            if hist:
+                assert slot >= 0, "a request of a model with state must own a slot"
+                seq = torch.cat([state[slot].view(hist, C), rows], dim=0)
+            y = rows.clone()
+            for j in range(taps):
+                y = y + conv_w[j] * seq[j:j + nq]
+            out[cu[s]:cu[s + 1]] = y
+            if hist:
+                state[slot] = seq[nq:].reshape(-1).clone()
+        return out.to(self.compute_dtype)
+
+    def general_delta_scan(self, proj, a_col0, z, w0, a_bias, H, d, decay_scale, unit_eps, state, ctx):
+        self._count("general_delta_scan")
+        T, C = proj.shape[0], H * d
+        pf = proj.float()
+        r, k, v = (pf[:, i * C:(i + 1) * C].view(T, H, d) for i in range(3))
+        a = torch.sigmoid(pf[:, a_col0:a_col0 + C] + a_bias).view(T, H, d)
+        w = torch.exp(decay_scale * torch.sigmoid(z + w0)).view(T, H, d)
+        u = k * torch.rsqrt((k * k).sum(-1, keepdim=True) + unit_eps)
+        out = torch.zeros(T, H, d)
+        cu = ctx.host.cu
+        for s, slot in enumerate(ctx.host.state_slots):
+            assert slot >= 0, "a request of a model with state must own a slot"
+            S = state[slot].view(H, d, d)                       # column j of head h: S[h, j, :]
+            for t in range(cu[s], cu[s + 1]):
+                along = torch.einsum("hji,hi->hj", S, u[t])
+                S.copy_(S * w[t][:, None, :] - along[:, :, None] * (a[t] * u[t])[:, None, :] + v[t][:, :, None] * k[t][:, None, :])
+                out[t] = torch.einsum("hji,hi->hj", S, r[t])
+        return out.reshape(T, C)
+
+    def normed_branch(self, a, wa, eps):
+        self._count("normed_branch")
+        a = a.float()
+        return a * torch.rsqrt((a * a).mean(-1, keepdim=True) + eps) * wa.float()
+
+    def normed_add_rms_norm(self, x, a, wa, branch_eps, norm_w, eps):
+        x += self.normed_branch(a, wa, branch_eps)
+        return self.rms_norm(x, norm_w, eps)
+
     def normed_pair_sum(self, a, b, wa, wb, sa, sb, eps):
         self._count("normed_pair_sum")
 
@@ -448,13 +534,32 @@ class TorchOps:
                 out[t] = torch.einsum("hvd,hd->hv", S, q[t]).reshape(H * dv)
         return out
 
-    def head_norm_gate(self, o, proj, g_col0, H, dv, norm_w, eps):
+    def head_norm_gate(self, o, proj, g_col0, H, dv, norm_w, eps, gate="silu"):
         self._count("head_norm_gate")
         T = o.shape[0]
         v = o.view(T, H, dv)
-        v = v * torch.rsqrt((v * v).mean(-1, keepdim=True) + eps) * norm_w[None, None, :]
+        v = v * torch.rsqrt((v * v).mean(-1, keepdim=True) + eps) * norm_w.view(1, -1, dv)
         g = proj[:, g_col0:g_col0 + H * dv].float()
-        return (v.reshape(T, H * dv) * (g * torch.sigmoid(g))).to(self.compute_dtype)
+        g = g * torch.sigmoid(g) if gate == "silu" else torch.sigmoid(g)
+        return (v.reshape(T, H * dv) * g).to(self.compute_dtype)
+
+    def unit_qkv_write(self, proj, bias, nh, nkv, d, dv, D, eps, ctx, kv, block_table, write=True):
+        self._count("unit_qkv_write")
+        T = proj.shape[0]
+        pf = proj[:, :nh * d + nkv * (d + dv)].float()
+        if bias is not None:
+            pf = pf + bias
+
+        def unit(x):
+            return x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps)
+
+        q, k, v = torch.zeros(T, nh, D), torch.zeros(T, nkv, D), torch.zeros(T, nkv, D)
+        q[:, :, :d] = unit(pf[:, :nh * d].view(T, nh, d))
+        k[:, :, :d] = unit(pf[:, nh * d:(nh + nkv) * d].view(T, nkv, d))
+        v[:, :, :dv] = pf[:, (nh + nkv) * d:].view(T, nkv, dv)
+        if write:
+            self._write_slots(ctx, kv, block_table, k, v)
+        return q.reshape(T, nh * D).to(self.compute_dtype)
 
     def normed_qkv_write(self, proj, nh, nkv, d, dv, D, q_weight, k_weight, eps, ctx, kv, block_table, has_kv=True,
                          write=True, position=None, query_temperature=None):
