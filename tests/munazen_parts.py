@@ -57,6 +57,8 @@ def _cache_for(req, n_req, lens, ps, dtype, device, seed):
         for view, ts in parts:
             views.append(view)
         return LayerCache("parts", -1, True, parts=tuple(views)), tables
+    if req is None:
+        return None, []
     if isinstance(req, FixedState):
         return LayerCache("fixed_state", -1, True, state=torch.zeros((n_req, *req.shape), device=device)), []
     assert isinstance(req, PagedKV)
