@@ -107,6 +107,21 @@ PIRERAX_SIZES = {
     "x-tiny": dict(vocab=256, width=128, heads=4, kv_heads=2, dim=32, rot_dim=16, kv_rank=32, delta_heads=4, delta_kv=2,
                    delta_dim=16, delta_vdim=32, conv=3, experts=8, top=2, groups=(4, 2), expert_ff=64),
 }
+# Tagelorn at the layer sizes of a 2k- and a 4k-wide model: windowed attention with kept tokens, a bias table and a sink, the
+# generalized delta rule, routed experts of one matrix in front of the activation beside a shared one (the Pirerax beside it
+# gets the same widths, heads, delta-rule heads and experts)
+TAGELORN_SIZES = {
+    "t-2k": dict(vocab=32000, width=2048, heads=16, kv_heads=4, dim=128, window=1024, keep_first=4, delta_heads=16, delta_dim=128,
+                 ff=8192, experts=32, top=4, groups=(8, 4), expert_ff=1024, shared_ff=1024, taps=3, side_dim=128),
+    "t-4k": dict(vocab=32000, width=4096, heads=32, kv_heads=8, dim=128, window=1024, keep_first=4, delta_heads=32, delta_dim=128,
+                 ff=14336, experts=64, top=6, groups=(8, 4), expert_ff=1408, shared_ff=1408, taps=3, side_dim=256),
+    # heads of 64 in both mixers
+    "t-2k-64": dict(vocab=32000, width=2048, heads=32, kv_heads=8, dim=64, window=1024, keep_first=4, delta_heads=32, delta_dim=64,
+                    ff=8192, experts=32, top=4, groups=(8, 4), expert_ff=1024, shared_ff=1024, taps=3, side_dim=128),
+    # for trying the option out quickly; never a result
+    "t-tiny": dict(vocab=256, width=128, heads=4, kv_heads=2, dim=32, window=64, keep_first=4, delta_heads=4, delta_dim=16, ff=256,
+                   experts=8, top=2, groups=(4, 2), expert_ff=64, shared_ff=64, taps=3, side_dim=24),
+}
 PROMPT_LEN, DECODE_LEN, PREFILL_TOKENS, BLOCK_SIZE = 512, 256, 2048, 16
 RAGGED_PROMPTS, RAGGED_OUTPUTS = (128, 4096), (64, 512)      # the ragged serving workload: lengths drawn uniformly
 
@@ -689,9 +704,31 @@ def pirerax_configs(name: str):
     return pir, llama, len(order)
 
 
-def compare_with_llama(args, label: str, size: str, sizes: dict, model: dict, llama: dict, runs: int) -> dict:
+def tagelorn_configs(name: str):
+    """(Tagelorn configuration dict, Pirerax configuration dict of equal size, number of layers)."""
+    s = TAGELORN_SIZES[name]
+    heads = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5}
+    attention = dict(heads, bias_max=float(s["window"]), mask={"size": s["window"], "keep_first": s["keep_first"]})
+    delta = {"heads": s["delta_heads"], "dim": s["delta_dim"]}
+    groups = {"count": s["groups"][0], "keep": s["groups"][1]}
+    moe = {"kind": "moe", "expert": {"ff": s["expert_ff"]}, "router": {"experts": s["experts"], "top": s["top"], "scale": 2.0, "groups": groups},
+           "shared": {"ff": s["shared_ff"]}}
+    order = [("attention", attention, {"kind": "dense", "ff": s["ff"]}), ("general_delta", delta, moe), ("attention", attention, moe),
+             ("general_delta", delta, moe), ("attention", attention, moe), ("general_delta", delta, moe)]
+    tag = {"architecture": "Tagelorn", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6},
+           "embedding": {"scale": s["width"] ** 0.5}, "canon": {"taps": s["taps"]}, "token_side": {"dim": s["side_dim"]},
+           "logit_softcap": 30.0, "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in order]}
+    par = {"left": dict(heads, rot={"dims": s["dim"] // 2, "base": 500000.0}),
+           "right": {"heads": s["delta_heads"], "kv_heads": s["delta_heads"], "dim": s["delta_dim"], "vdim": s["delta_dim"], "conv": s["taps"]}}
+    pmoe = {"kind": "moe", "expert": {"ff": s["expert_ff"], "limit": 7.0}, "router": {"experts": s["experts"], "top": s["top"], "groups": groups}}
+    pir = {"architecture": "Pirerax", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6},
+           "layers": [{"type": t, "mixer": m, "mlp": pmoe} for t, m in [("attention", heads), ("parallel", par)] * 3]}
+    return tag, pir, len(order)
+
+
+def compare_with_llama(args, label: str, size: str, sizes: dict, model: dict, llama: dict, runs: int, beside: str = "llama") -> dict:
     """Prefill and decode of another decoder at layer sizes of a real model (random weights drawn on the
-    device) beside a Llama of equal width, heads and layer runs: device-timed with CUDA events, with the device
+    device) beside a Llama (or the model named by `beside`) of equal width, heads and layer runs: device-timed with CUDA events, with the device
     time of every kernel inside the steps for the roofline of each."""
     import torch
     from paged_llm_b200 import EngineConfig, LLMEngine
@@ -705,7 +742,7 @@ def compare_with_llama(args, label: str, size: str, sizes: dict, model: dict, ll
     max_len = max(ctx_len + steps + args.warmup + 16, pre) + 64
     out = {"only": label, "size": size, "layer_runs": runs, "prefill_tokens": pre, "context": ctx_len,
            "sizes": sizes, "peaks": load_peaks()}
-    for arm, hf in ((label, model), ("llama", llama)):
+    for arm, hf in ((label, model), (beside, llama)):
         with tempfile.TemporaryDirectory() as folder:
             _, cfg = parse_model_config(hf)
             write_random_stub(folder, cfg, seed=0, std=0.02, dtype="bfloat16")
@@ -753,6 +790,11 @@ def pirerax_compare(args) -> dict:
     return compare_with_llama(args, "pirerax", args.pirerax_size, PIRERAX_SIZES[args.pirerax_size], pir, llama, runs)
 
 
+def tagelorn_compare(args) -> dict:
+    tag, pir, runs = tagelorn_configs(args.tagelorn_size)
+    return compare_with_llama(args, "tagelorn", args.tagelorn_size, TAGELORN_SIZES[args.tagelorn_size], tag, pir, runs, beside="pirerax")
+
+
 def run_ours(args) -> dict:
     import torch
     from paged_llm_b200 import EngineConfig, LLMEngine
@@ -766,6 +808,8 @@ def run_ours(args) -> dict:
         return munazen_compare(args)
     if args.only == "pirerax":
         return pirerax_compare(args)
+    if args.only == "tagelorn":
+        return tagelorn_compare(args)
     if args.only == "validate":
         return validate(args)
     if args.only == "sample":
@@ -966,13 +1010,16 @@ def main() -> int:
                     help="with --only munazen: the layer sizes (the Llama beside it gets the same)")
     ap.add_argument("--pirerax-size", choices=sorted(PIRERAX_SIZES), default="x-2k",
                     help="with --only pirerax: the layer sizes (the Llama beside it gets the same)")
+    ap.add_argument("--tagelorn-size", choices=sorted(TAGELORN_SIZES), default="t-2k",
+                    help="with --only tagelorn: the layer sizes (the Pirerax beside it gets the same)")
     ap.add_argument("--only", choices=["decode", "prefill", "ragged", "mixed", "validate", "sample", "pomisun", "rokarax", "munazen",
-                                       "pirerax"], default=None,
+                                       "pirerax", "tagelorn"], default=None,
                     help="run only the decode loop, only the prefill step, the ragged serving workload through "
                          "LLMEngine.generate, one mixed step (--batch decoding requests of --context tokens beside one "
                          "portion of --prefill-tokens), the float32 validation run, the sampler's kernels on --batch rows, or "
                          "prefill and decode of the Pomisun, the Rokarax, the Munazen or the Pirerax decoder beside a Llama of equal size "
-                         "(--pomisun-size, --rokarax-size, --munazen-size, --pirerax-size), and print "
+                         "(--pomisun-size, --rokarax-size, --munazen-size, --pirerax-size), or of the Tagelorn decoder beside a Pirerax of "
+                         "equal size (--tagelorn-size), and print "
                          "a short line")
     args = ap.parse_args()
     if args.gpus != 1 or int(os.environ.get("WORLD_SIZE", "1")) > 1:

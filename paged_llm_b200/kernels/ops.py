@@ -294,10 +294,6 @@ class CudaOps:
         self.launches += 1
         return out
 
-    def tanh_columns(self, x: torch.Tensor, col0: int, n: int) -> torch.Tensor:
-        """tanh(x[:, col0 : col0 + n]) as a tensor of its own."""
-        return self._act_columns(x, col0, n, ACT_TANH)
-
     def relu2_linear(self, h, w: torch.Tensor) -> torch.Tensor:
         """relu(h @ w^T)^2: the activation sits in the product's epilogue where the product is this package's own."""
         M, K = h.shape
@@ -837,30 +833,43 @@ class CudaOps:
         self.launches += 1
         return out
 
-    def general_delta_scan(self, proj, a_col0, z, w0, a_bias, H, d, decay_scale, unit_eps, state, ctx) -> torch.Tensor:
-        """The generalized delta rule's recurrence.  proj rows [r: C | k: C | v: C | ...] with the removal rates' input at
-        columns [a_col0, + C), C = H*d; z float32 [T, C] the decay's input.  Per head, with w = exp(decay_scale *
-        sigmoid(z + w0)), a = sigmoid(removal + a_bias), u = k / sqrt(sum k^2 + unit_eps):
-        S <- diag(w) S - (a u)(u^T S) + k v^T, o = S^T r.  state: [slots, H*d*d] float32 (a head's columns one after the
-        other), updated in place.  Returns o float32 [T, C]."""
+    GENERAL_DELTA_STEP_TOKENS = 8        # requests that bring no more than this run token by token in one kernel
+
+    def general_delta_mix(self, proj, rank, w_decay, w0, a_bias, H, d, decay_scale, unit_eps, norm_w, eps, state, ctx) -> torch.Tensor:
+        """The generalized delta rule between its two projections.  proj rows [r: C | k: C | v: C | g: C | removal: C |
+        decay: rank], C = H*d.  Per head, with w = exp(decay_scale * sigmoid(w_decay tanh(decay) + w0)), a = sigmoid(removal +
+        a_bias), u = k / sqrt(sum k^2 + unit_eps): S <- diag(w) S - (a u)(u^T S) + k v^T, o = S^T r; returns
+        rms_norm(o per head) * norm_w * sigmoid(g) in the compute dtype.  state: [slots, H*d*d] float32 (a head's columns one
+        after the other), updated in place.  A step of few tokens per request is one kernel; longer portions run in chunks:
+        everything that does not depend on the state first, for all chunks at once, then a request's chunks in order."""
         lib = load_module("general_delta")
         T, ld = proj.shape
         C = H * d
-        assert proj.is_contiguous() and z.dtype == torch.float32 and z.is_contiguous() and z.shape == (T, C)
-        assert w0.dtype == torch.float32 and a_bias.dtype == torch.float32 and w0.numel() == C and a_bias.numel() == C
+        assert proj.is_contiguous() and w_decay.is_contiguous() and w_decay.shape == (C, rank) and w_decay.dtype == proj.dtype
+        for t in (w0, a_bias, norm_w):
+            assert t.dtype == torch.float32 and t.numel() == C and t.is_contiguous()
         assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] == C * d
+        code = self._code(proj)
+        if (int(ctx.max_q_len) <= self.GENERAL_DELTA_STEP_TOKENS and not getattr(ctx, "padded", False) and d <= 128
+                and rank % 8 == 0 and rank <= 256):
+            out = torch.empty((T, C), dtype=proj.dtype, device=self.device)
+            _check(lib, lib.pl_general_delta_step(self._p(proj), code, ld, self._p(w_decay), rank, self._p(w0), self._p(a_bias), H, d,
+                                                  c_float(decay_scale), c_float(unit_eps), self._p(norm_w), c_float(eps), self._p(state),
+                                                  c_longlong(state.shape[1]), self._p(ctx.cu_seqlens_q), self._p(ctx.state_slots),
+                                                  ctx.num_seqs, self._p(out), self._stream))
+            self.launches += 1
+            return out
+        z = self.linear(self._act_columns(proj, 5 * C, rank, ACT_TANH), w_decay, out_float32=True)
         o = torch.empty((T, C), dtype=torch.float32, device=self.device)
-        vec = scal = None
-        if int(ctx.max_q_len) > 4 or getattr(ctx, "padded", False):
-            # longer portions: what does not depend on the state is formed for all tokens at once in front
-            vec = torch.empty((T, H, 6, d), dtype=torch.float32, device=self.device)
-            scal = torch.empty((T, H, 2), dtype=torch.float32, device=self.device)
-        _check(lib, lib.pl_general_delta(self._p(proj), self._code(proj), ld, a_col0, self._p(z), self._p(w0), self._p(a_bias), H, d,
-                                         c_float(decay_scale), c_float(unit_eps), self._p(vec), self._p(scal), self._p(state),
-                                         c_longlong(state.shape[1]), self._p(ctx.cu_seqlens_q), self._p(ctx.state_slots),
-                                         ctx.num_seqs, c_longlong(T), self._p(o), self._stream))
-        self.launches += 1 if vec is None else 2
-        return o
+        lib.pl_general_delta_chunk_floats.restype = c_longlong
+        chunks = T // lib.pl_general_delta_chunk() + ctx.num_seqs
+        buf = torch.empty(chunks * H * lib.pl_general_delta_chunk_floats(d), dtype=torch.float32, device=self.device)
+        _check(lib, lib.pl_general_delta_chunks(self._p(proj), code, ld, self._p(z), self._p(w0), self._p(a_bias), H, d,
+                                                c_float(decay_scale), c_float(unit_eps), self._p(buf), chunks, self._p(state),
+                                                c_longlong(state.shape[1]), self._p(ctx.cu_seqlens_q), self._p(ctx.state_slots),
+                                                ctx.num_seqs, self._p(o), self._stream))
+        self.launches += 2
+        return self.head_norm_gate(o, proj, 3 * C, H, d, norm_w, eps, gate="sigmoid")
 
     # ---- two branches that are normed before they meet ---------------------------------
     def normed_pair_sum(self, a, b, wa, wb, sa, sb, eps) -> torch.Tensor:

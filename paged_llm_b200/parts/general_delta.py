@@ -39,6 +39,8 @@ class GeneralDeltaRule(Mixer):
         if head_dim > 256:
             raise ValueError(f"heads of {head_dim}: the recurrence's kernels take at most 256")
         self.hidden_size, self.num_heads, self.head_dim, self.eps = hidden_size, num_heads, head_dim, float(eps)
+        if not -4.0 <= decay_scale <= 0.0:
+            raise ValueError(f"decay_scale={decay_scale}: the kernels for prompts take -4 to 0")
         self.decay_scale, self.unit_eps = float(decay_scale), float(unit_eps)
         self.decay_rank = int(decay_rank)           # what random weights are drawn with; a checkpoint's own shape rules
         self.names = weights
@@ -88,11 +90,7 @@ class GeneralDeltaRule(Mixer):
         if any(slot < 0 for slot in ctx.host.state_slots):
             raise RuntimeError("a request of a model with per-request state runs without a state slot "
                                "(CacheManager.acquire_state_slot at its admission)")
-        H, d = self.num_heads, self.head_dim
-        C = H * d
         proj = ops.linear(h, self.w_in)                                       # [T, r | k | v | g | removal | decay | padding]
-        z = ops.linear(ops.tanh_columns(proj, 5 * C, self.rank), self.w_decay, out_float32=True)
-        o = ops.general_delta_scan(proj, 4 * C, z, self.decay_bias, self.removal_bias, H, d, self.decay_scale, self.unit_eps,
-                                   cache.state, ctx)                          # float32 [T, C]
-        out = ops.head_norm_gate(o, proj, 3 * C, H, d, self.norm_w, self.eps, gate="sigmoid")
+        out = ops.general_delta_mix(proj, self.rank, self.w_decay, self.decay_bias, self.removal_bias, self.num_heads, self.head_dim,
+                                    self.decay_scale, self.unit_eps, self.norm_w, self.eps, cache.state, ctx)
         return LazyLinear(out, self.w_o)

@@ -54,10 +54,6 @@ class TorchOps:
         out[:, :dim] = z[:, :dim] * table[ids.long()][:, offset:offset + dim].float()
         return out.to(self.compute_dtype)
 
-    def tanh_columns(self, x, col0, n):
-        self._count("tanh_columns")
-        return torch.tanh(x[:, col0:col0 + n].float()).to(self.compute_dtype)
-
     def relu2_linear(self, h, w):
         return (self.linear(h, w).float().clamp(min=0.0) ** 2).to(self.compute_dtype)
 
@@ -455,12 +451,13 @@ class TorchOps:
                 state[slot] = seq[nq:].reshape(-1).clone()
         return out.to(self.compute_dtype)
 
-    def general_delta_scan(self, proj, a_col0, z, w0, a_bias, H, d, decay_scale, unit_eps, state, ctx):
-        self._count("general_delta_scan")
+    def general_delta_mix(self, proj, rank, w_decay, w0, a_bias, H, d, decay_scale, unit_eps, norm_w, eps, state, ctx):
+        self._count("general_delta_mix")
         T, C = proj.shape[0], H * d
         pf = proj.float()
+        z = self.linear(torch.tanh(pf[:, 5 * C:5 * C + rank]).to(self.compute_dtype), w_decay, out_float32=True)
         r, k, v = (pf[:, i * C:(i + 1) * C].view(T, H, d) for i in range(3))
-        a = torch.sigmoid(pf[:, a_col0:a_col0 + C] + a_bias).view(T, H, d)
+        a = torch.sigmoid(pf[:, 4 * C:5 * C] + a_bias).view(T, H, d)
         w = torch.exp(decay_scale * torch.sigmoid(z + w0)).view(T, H, d)
         u = k * torch.rsqrt((k * k).sum(-1, keepdim=True) + unit_eps)
         out = torch.zeros(T, H, d)
@@ -472,7 +469,7 @@ class TorchOps:
                 along = torch.einsum("hji,hi->hj", S, u[t])
                 S.copy_(S * w[t][:, None, :] - along[:, :, None] * (a[t] * u[t])[:, None, :] + v[t][:, :, None] * k[t][:, None, :])
                 out[t] = torch.einsum("hji,hi->hj", S, r[t])
-        return out.reshape(T, C)
+        return self.head_norm_gate(out.reshape(T, C), proj, 3 * C, H, d, norm_w, eps, gate="sigmoid")
 
     def normed_branch(self, a, wa, eps):
         self._count("normed_branch")
