@@ -116,34 +116,6 @@ struct GdIn {
     float decay_scale, unit_eps;
 };
 
-// Per token and head, what does not depend on the state: w, u, a u, k, r w, v and the numbers r . (a u) and r . k.  A warp
-// computes one (token, head); `lane` takes channels lane, lane + 32, ...; z: the head's d decay inputs in front of their bias.
-template <typename T>
-__device__ __forceinline__ void gd_prepare(const GdIn& in, long long t, int h, int lane, const float* z, float* w, float* u, float* au,
-                                           float* k, float* rw, float* v, float* scal) {
-    const int d = in.d, C = in.H * d, c0 = h * d;
-    const T* row = (const T*)in.proj + (size_t)t * in.ld + c0;
-    float sq = 0.f;
-    for (int i = lane; i < d; i += 32) {
-        const float kv = to_float(row[C + i]);
-        sq = fmaf(kv, kv, sq);
-    }
-    const float f = 1.0f / sqrtf(warp_sum(sq) + in.unit_eps);
-    float rau = 0.f, rk = 0.f;
-    for (int i = lane; i < d; i += 32) {
-        const float rv = to_float(row[i]), kv = to_float(row[C + i]);
-        const float a = sigmoid_f(to_float(row[4 * C + i]) + __ldg(in.a_bias + c0 + i));
-        const float wv = expf(in.decay_scale * sigmoid_f(z[i] + __ldg(in.w0 + c0 + i)));
-        const float uv = kv * f, auv = a * uv;
-        w[i] = wv, u[i] = uv, au[i] = auv, k[i] = kv, rw[i] = rv * wv, v[i] = to_float(row[2 * C + i]);
-        rau = fmaf(rv, auv, rau);
-        rk = fmaf(rv, kv, rk);
-    }
-    rau = warp_sum(rau);
-    rk = warp_sum(rk);
-    if (lane == 0) scal[0] = rau, scal[1] = rk;
-}
-
 // ------------------------------------------------------------------ few tokens per request (decoding)
 // A block per (request, head) does the whole mixer between its two projections: the decay's low rank
 // (tanh, product), gates and unit norm, the recurrence, the norm of the head's output and the output gate.  The head's state
@@ -156,7 +128,7 @@ struct GdTail {
     const float* norm_w;        // [C]
     float eps;
 };
-constexpr int GD_MAX_RANK = 256, GS_TOK = 4, GS_THREADS = 256, GS_LANES = 8;
+constexpr int GD_MAX_RANK = 256, GS_THREADS = 256, GS_LANES = 8;
 
 __device__ __forceinline__ void gs_load8(const float* p, float (&v)[8]) {
     const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
@@ -173,23 +145,45 @@ __device__ __forceinline__ void gd_cp16(float* dst, const float* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src));
 }
 
-__host__ __device__ constexpr int gs_smem(int DP) { return (DP * DP + GS_TOK * (6 * DP + 4) + GS_TOK * DP + GS_TOK * GD_MAX_RANK) * (int)sizeof(float); }
+// Tokens of a request worked on at a time: a thread prepares one channel of one token.
+__host__ __device__ constexpr int gs_tokens(int DP) { return GS_THREADS / DP; }
+__host__ __device__ constexpr int gs_row(int DP) { return 6 * DP + 4; }
+__host__ __device__ constexpr int gs_smem(int DP) {
+    return (DP * DP + gs_tokens(DP) * (gs_row(DP) + DP + GD_MAX_RANK)) * (int)sizeof(float);
+}
+
+// The sum over a token's DP channels of two numbers per thread, in a fixed order, for all of the token's threads.
+// red: [2][GS_THREADS / 32]; all threads of the block take part.
+template <int DP>
+__device__ __forceinline__ float2 gs_token_sum(float a, float b, float* red, int tid) {
+    a = warp_sum(a), b = warp_sum(b);
+    if (DP == 32) return make_float2(a, b);
+    constexpr int W = DP / 32, NW = GS_THREADS / 32;
+    if ((tid & 31) == 0) red[tid >> 5] = a, red[NW + (tid >> 5)] = b;
+    __syncthreads();
+    const int w0 = (tid >> 5) / W * W;
+    float2 s = make_float2(red[w0], red[NW + w0]);
+#pragma unroll
+    for (int i = 1; i < W; ++i) s.x += red[w0 + i], s.y += red[NW + w0 + i];
+    return s;
+}
 
 template <typename T, int NPER>
-__global__ void __launch_bounds__(GS_THREADS) gd_step_kernel(GdIn in, GdTail tail, float* __restrict__ state, long long state_stride,
-                                                             const int* __restrict__ cu_q, const int* __restrict__ slots,
-                                                             T* __restrict__ out, int vec) {
-    constexpr int DP = NPER * GS_LANES, ROW = 6 * DP + 4;
+__global__ void __launch_bounds__(GS_THREADS, 3) gd_step_kernel(GdIn in, GdTail tail, float* __restrict__ state, long long state_stride,
+                                                                const int* __restrict__ cu_q, const int* __restrict__ slots,
+                                                                T* __restrict__ out, int vec) {
+    constexpr int DP = NPER * GS_LANES, ROW = gs_row(DP), TOK = gs_tokens(DP), NW = GS_THREADS / 32;
     extern __shared__ __align__(16) float gs_raw[];
     float* Ss = gs_raw;                                 // [DP columns][DP]: the head's state
-    float* rows = Ss + DP * DP;                         // [GS_TOK][ROW]
-    float* zs = rows + GS_TOK * ROW;                    // [GS_TOK][DP]: the decay's inputs, then the head's outputs
-    float* th = zs + GS_TOK * DP;                       // [GS_TOK][GD_MAX_RANK]
+    float* rows = Ss + DP * DP;                         // [TOK][ROW]: w, u, a u, k, r w, v, r . (a u), r . k
+    float* os = rows + TOK * ROW;                       // [TOK][DP]: the head's outputs
+    float* th = os + TOK * DP;                          // [TOK][GD_MAX_RANK]
+    __shared__ float red[3][2 * NW];
     pdl_launch_dependents();
     const int s = blockIdx.x / in.H, h = blockIdx.x - s * in.H, d = in.d, C = in.H * d, c0 = h * d;
     const int slot = slots[s];
     const int q0 = cu_q[s], nq = cu_q[s + 1] - q0;
-    const int tid = threadIdx.x, lane = tid % GS_LANES, col = tid / GS_LANES, wlane = tid & 31, warp = tid >> 5;
+    const int tid = threadIdx.x, lane = tid % GS_LANES, col = tid / GS_LANES, wlane = tid & 31;
     if (slot < 0 || nq <= 0) {
         pdl_wait();
         return;
@@ -209,37 +203,42 @@ __global__ void __launch_bounds__(GS_THREADS) gd_step_kernel(GdIn in, GdTail tai
         }
     }
     asm volatile("cp.async.commit_group;\n" ::);
-    pdl_wait();
-    if (d < DP)
-        for (int e = tid; e < GS_TOK * ROW; e += GS_THREADS) rows[e] = 0.f;          // channels that pad a row stay zero
+    // this thread's channel of its token: what is weights
+    const int tt = tid / DP, i = tid - tt * DP;
+    const bool real = i < d;
+    const float w0 = real ? __ldg(in.w0 + c0 + i) : 0.f, ab = real ? __ldg(in.a_bias + c0 + i) : 0.f, nw = real ? __ldg(tail.norm_w + c0 + i) : 0.f;
+    const T* w2 = (const T*)tail.w_decay + (size_t)(c0 + (real ? i : 0)) * tail.rank;
     const T* proj = (const T*)in.proj;
-    for (int t0 = 0; t0 < nq; t0 += GS_TOK) {
-        const int nt = min(GS_TOK, nq - t0);
-        const bool last = t0 + GS_TOK >= nq;
+    pdl_wait();
+    for (int t0 = 0; t0 < nq; t0 += TOK) {
+        const int nt = min(TOK, nq - t0);
+        const bool last = t0 + TOK >= nq, live = real && tt < nt;
+        const T* row_in = proj + (size_t)(q0 + t0 + (tt < nt ? tt : 0)) * in.ld + c0 + (real ? i : 0);
+        const float r = live ? to_float(row_in[0]) : 0.f, k = live ? to_float(row_in[C]) : 0.f, v = live ? to_float(row_in[2 * C]) : 0.f;
+        const float g = to_float(row_in[3 * C]), rem = to_float(row_in[4 * C]);
         for (int e = tid; e < nt * tail.rank; e += GS_THREADS) {
-            const int tt = e / tail.rank, r = e - tt * tail.rank;
+            const int t = e / tail.rank, q = e - t * tail.rank;
             // (rounded as the activations of a product are)
-            th[tt * GD_MAX_RANK + r] = to_float(from_float<T>(tanhf(to_float(proj[(size_t)(q0 + t0 + tt) * in.ld + 5 * C + r]))));
+            th[t * GD_MAX_RANK + q] = to_float(from_float<T>(tanhf(to_float(proj[(size_t)(q0 + t0 + t) * in.ld + 5 * C + q]))));
         }
+        const float unit = 1.0f / sqrtf(gs_token_sum<DP>(k * k, 0.f, red[0], tid).x + in.unit_eps);
         __syncthreads();
-        for (int e = tid; e < nt * d; e += GS_THREADS) {
-            const int tt = e / d, i = e - tt * d;
-            const T* w2 = (const T*)tail.w_decay + (size_t)(c0 + i) * tail.rank;
-            float acc = 0.f;
+        float z = 0.f;
+        if (live) {
 #pragma unroll 4
-            for (int r = 0; r < tail.rank; r += 8) {
+            for (int q = 0; q < tail.rank; q += 8) {
                 float w8[8];
-                gs_load8(w2 + r, w8);
-#pragma unroll
-                for (int q = 0; q < 8; ++q) acc = fmaf(th[tt * GD_MAX_RANK + r + q], w8[q], acc);
+                gs_load8(w2 + q, w8);
+                const float4 a4 = *reinterpret_cast<const float4*>(th + tt * GD_MAX_RANK + q), b4 = *reinterpret_cast<const float4*>(th + tt * GD_MAX_RANK + q + 4);
+                z = fmaf(a4.x, w8[0], z), z = fmaf(a4.y, w8[1], z), z = fmaf(a4.z, w8[2], z), z = fmaf(a4.w, w8[3], z);
+                z = fmaf(b4.x, w8[4], z), z = fmaf(b4.y, w8[5], z), z = fmaf(b4.z, w8[6], z), z = fmaf(b4.w, w8[7], z);
             }
-            zs[tt * DP + i] = acc;
         }
-        __syncthreads();
-        if (warp < nt) {
-            float* o = rows + warp * ROW;
-            gd_prepare<T>(in, q0 + t0 + warp, h, wlane, zs + warp * DP, o, o + DP, o + 2 * DP, o + 3 * DP, o + 4 * DP, o + 5 * DP, o + 6 * DP);
-        }
+        const float w = expf(in.decay_scale * sigmoid_f(z + w0)), u = k * unit, au = sigmoid_f(rem + ab) * u;
+        float* row = rows + tt * ROW;                   // (channels that pad a row: everything but w is zero, and so is S)
+        row[i] = w, row[DP + i] = u, row[2 * DP + i] = au, row[3 * DP + i] = k, row[4 * DP + i] = r * w, row[5 * DP + i] = v;
+        const float2 dots = gs_token_sum<DP>(r * au, r * k, red[1], tid);
+        if (i == 0) row[6 * DP] = dots.x, row[6 * DP + 1] = dots.y;
         asm volatile("cp.async.wait_group 0;\n" ::);
         __syncthreads();
 #pragma unroll 2
@@ -248,17 +247,17 @@ __global__ void __launch_bounds__(GS_THREADS) gd_step_kernel(GdIn in, GdTail tai
             const int jr = j < d ? j : 0;
 #pragma unroll
             for (int m = 0; m < NPER / 4; ++m) {
-                const float4 v = *reinterpret_cast<const float4*>(Ss + jr * DP + m * 32 + lane * 4);
-                S[4 * m] = v.x, S[4 * m + 1] = v.y, S[4 * m + 2] = v.z, S[4 * m + 3] = v.w;
+                const float4 x = *reinterpret_cast<const float4*>(Ss + jr * DP + m * 32 + lane * 4);
+                S[4 * m] = x.x, S[4 * m + 1] = x.y, S[4 * m + 2] = x.z, S[4 * m + 3] = x.w;
             }
-            for (int tt = 0; tt < nt; ++tt) {
-                const float* row = rows + tt * ROW;
-                const float rau = row[6 * DP], rk = row[6 * DP + 1], v = row[5 * DP + jr];
+            for (int t = 0; t < nt; ++t) {
+                const float* ro = rows + t * ROW;
+                const float rau = ro[6 * DP], rk = ro[6 * DP + 1], vj = ro[5 * DP + jr];
                 float c4[4] = {0.f, 0.f, 0.f, 0.f}, e4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
                 for (int m = 0; m < NPER / 4; ++m) {
-                    const float4 u4 = *reinterpret_cast<const float4*>(row + DP + m * 32 + lane * 4);
-                    const float4 q4 = *reinterpret_cast<const float4*>(row + 4 * DP + m * 32 + lane * 4);
+                    const float4 u4 = *reinterpret_cast<const float4*>(ro + DP + m * 32 + lane * 4);
+                    const float4 q4 = *reinterpret_cast<const float4*>(ro + 4 * DP + m * 32 + lane * 4);
                     c4[0] = fmaf(S[4 * m], u4.x, c4[0]), c4[1] = fmaf(S[4 * m + 1], u4.y, c4[1]);
                     c4[2] = fmaf(S[4 * m + 2], u4.z, c4[2]), c4[3] = fmaf(S[4 * m + 3], u4.w, c4[3]);
                     e4[0] = fmaf(S[4 * m], q4.x, e4[0]), e4[1] = fmaf(S[4 * m + 1], q4.y, e4[1]);
@@ -276,24 +275,24 @@ __global__ void __launch_bounds__(GS_THREADS) gd_step_kernel(GdIn in, GdTail tai
                 c = __shfl_sync(0xffffffffu, x, wlane & ~(GS_LANES - 1));
 #pragma unroll
                 for (int m = 0; m < NPER / 4; ++m) {
-                    const float4 w4 = *reinterpret_cast<const float4*>(row + m * 32 + lane * 4);
-                    const float4 a4 = *reinterpret_cast<const float4*>(row + 2 * DP + m * 32 + lane * 4);
-                    const float4 k4 = *reinterpret_cast<const float4*>(row + 3 * DP + m * 32 + lane * 4);
-                    S[4 * m] = fmaf(-a4.x, c, fmaf(w4.x, S[4 * m], k4.x * v));
-                    S[4 * m + 1] = fmaf(-a4.y, c, fmaf(w4.y, S[4 * m + 1], k4.y * v));
-                    S[4 * m + 2] = fmaf(-a4.z, c, fmaf(w4.z, S[4 * m + 2], k4.z * v));
-                    S[4 * m + 3] = fmaf(-a4.w, c, fmaf(w4.w, S[4 * m + 3], k4.w * v));
+                    const float4 w4 = *reinterpret_cast<const float4*>(ro + m * 32 + lane * 4);
+                    const float4 a4 = *reinterpret_cast<const float4*>(ro + 2 * DP + m * 32 + lane * 4);
+                    const float4 k4 = *reinterpret_cast<const float4*>(ro + 3 * DP + m * 32 + lane * 4);
+                    S[4 * m] = fmaf(-a4.x, c, fmaf(w4.x, S[4 * m], k4.x * vj));
+                    S[4 * m + 1] = fmaf(-a4.y, c, fmaf(w4.y, S[4 * m + 1], k4.y * vj));
+                    S[4 * m + 2] = fmaf(-a4.z, c, fmaf(w4.z, S[4 * m + 2], k4.z * vj));
+                    S[4 * m + 3] = fmaf(-a4.w, c, fmaf(w4.w, S[4 * m + 3], k4.w * vj));
                 }
-                if (j < d && lane == GS_LANES / 2) zs[tt * DP + j] = fmaf(rk, v, fmaf(-rau, c, x));
+                if (lane == GS_LANES / 2) os[t * DP + j] = j < d ? fmaf(rk, vj, fmaf(-rau, c, x)) : 0.f;
             }
             if (j < d) {
 #pragma unroll
                 for (int m = 0; m < NPER / 4; ++m) {
                     const int ch = m * 32 + lane * 4;
-                    const float4 v = make_float4(S[4 * m], S[4 * m + 1], S[4 * m + 2], S[4 * m + 3]);
-                    if (!last) *reinterpret_cast<float4*>(Ss + j * DP + ch) = v;
+                    const float4 x = make_float4(S[4 * m], S[4 * m + 1], S[4 * m + 2], S[4 * m + 3]);
+                    if (!last) *reinterpret_cast<float4*>(Ss + j * DP + ch) = x;
                     else if (vec) {
-                        if (ch < d) *reinterpret_cast<float4*>(sp + (size_t)j * d + ch) = v;
+                        if (ch < d) *reinterpret_cast<float4*>(sp + (size_t)j * d + ch) = x;
                     } else {
 #pragma unroll
                         for (int q = 0; q < 4; ++q)
@@ -303,16 +302,10 @@ __global__ void __launch_bounds__(GS_THREADS) gd_step_kernel(GdIn in, GdTail tai
             }
         }
         __syncthreads();
-        if (warp < nt) {
-            const float* o = zs + warp * DP;
-            float sq = 0.f;
-            for (int i = wlane; i < d; i += 32) sq = fmaf(o[i], o[i], sq);
-            const float f = 1.0f / sqrtf(warp_sum(sq) / (float)d + tail.eps);
-            const T* g = proj + (size_t)(q0 + t0 + warp) * in.ld + 3 * C + c0;
-            T* dst = out + (size_t)(q0 + t0 + warp) * C + c0;
-            for (int i = wlane; i < d; i += 32) dst[i] = from_float<T>(o[i] * f * __ldg(tail.norm_w + c0 + i) * sigmoid_f(to_float(g[i])));
-        }
-        __syncthreads();
+        const float o = tt < nt ? os[tt * DP + i] : 0.f;
+        const float f = 1.0f / sqrtf(gs_token_sum<DP>(o * o, 0.f, red[2], tid).x / (float)d + tail.eps);
+        if (live) out[(size_t)(q0 + t0 + tt) * C + c0 + i] = from_float<T>(o * f * nw * sigmoid_f(g));
+        if (!last) __syncthreads();
     }
 }
 
@@ -353,18 +346,22 @@ int launch_gd_step(const GdIn& in, const GdTail& tail, float* state, long long s
 // The chunks of request s are numbered from cu_q[s] / GC + s; the numbers of different requests do not meet.
 constexpr int GC = 16, GC_THREADS = 256, GC_COLS = 16;
 
-// Floats of a (chunk, head): [DP + GC][2 GC] the matrix above, transposed; [2 GC][DP] what is added to the state per value and
-// per c; [DP] P_end; [GC][DP] the values.
-__host__ __device__ constexpr size_t gc_floats(int DP) { return (size_t)(DP + GC) * 2 * GC + 2 * GC * DP + DP + GC * DP; }
+// A (chunk, head) in memory, in floats: the matrix above, row-major, a row GC_LD(DP) long (4 floats more than it needs, so that
+// the second kernel's reads of eight rows meet no bank of shared memory twice); [2 GC][DP] what is added to the state per value
+// and per c; [DP] P_end; the values, by blocks of 16 columns, [DP / 16][GC][16].
+__host__ __device__ constexpr int gc_ld(int DP) { return DP + GC + 4; }
+__host__ __device__ constexpr int gc_fixed(int DP) { return 2 * GC * gc_ld(DP) + 2 * GC * DP + DP; }
+__host__ __device__ constexpr size_t gc_floats(int DP) { return (size_t)gc_fixed(DP) + GC * DP; }
 __host__ __device__ constexpr int gc_prepare_smem(int DP) { return (4 * GC * (DP + 4) + 4 * GC * GC + GC) * (int)sizeof(float); }
 
 template <typename T, int DP>
 __global__ void __launch_bounds__(GC_THREADS) gd_chunk_prepare_kernel(GdIn in, const float* __restrict__ z, const int* __restrict__ cu_q,
                                                                       const int* __restrict__ slots, int num_seqs, float* __restrict__ buf) {
     constexpr int LD = DP + 4;                          // rows 4 floats longer: 16-byte reads of eight rows meet no bank twice
+    constexpr int PARTS = GC_THREADS / DP, TP = GC / PARTS;          // threads per channel, tokens of each
     extern __shared__ __align__(16) float gc_smem[];
-    float *xs = gc_smem, *bs = xs + GC * LD, *ks = bs + GC * LD, *ys = ks + GC * LD;      // first w, a; then x, b, k~, y
-    float* gram = ys + GC * LD;                         // [x . k~ | x . b | y . k~ | y . b][GC][GC]
+    float *xs = gc_smem, *bs = xs + GC * LD, *ks = bs + GC * LD, *ys = ks + GC * LD;      // first w, a, k, r; then x, b, k~, y
+    float* gram = ys + GC * LD;                         // [x . k~ | x . b | y . k~ | y . b][s][t]: a column of each in a row
     float* unit = gram + 4 * GC * GC;                   // [GC]
     const int chunk = blockIdx.x, h = blockIdx.y, d = in.d, C = in.H * d, c0 = h * d;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -380,61 +377,68 @@ __global__ void __launch_bounds__(GC_THREADS) gd_chunk_prepare_kernel(GdIn in, c
     const int nt = min(GC, nq - t0);
     const T* row0 = (const T*)in.proj + (size_t)(q0 + t0) * in.ld + c0;
     const float* z0 = z + (size_t)(q0 + t0) * C + c0;
-    for (int t = warp; t < nt; t += GC_THREADS / 32) {
-        float sq = 0.f;
-        for (int i = lane; i < d; i += 32) {
-            const float kv = to_float(row0[(size_t)t * in.ld + C + i]);
-            sq = fmaf(kv, kv, sq);
+    float* M = buf + ((size_t)chunk * in.H + h) * gc_floats(DP);
+    float* W = M + 2 * GC * gc_ld(DP);
+    float* Pend = W + 2 * GC * DP;
+    float* V = Pend + DP;
+    // a thread per channel and PARTS apart in the tokens, all loads of a token independent of each other
+    {
+        const int i = tid % DP;
+        const bool real = i < d;
+        const float w0 = real ? __ldg(in.w0 + c0 + i) : 0.f, ab = real ? __ldg(in.a_bias + c0 + i) : 0.f;
+#pragma unroll 4
+        for (int t = tid / DP; t < GC; t += PARTS) {
+            float w = 1.f, a = 0.f, k = 0.f, r = 0.f, v = 0.f;
+            if (t < nt && real) {
+                const T* row = row0 + (size_t)t * in.ld + i;
+                r = to_float(row[0]), k = to_float(row[C]), v = to_float(row[2 * C]);
+                w = expf(in.decay_scale * sigmoid_f(z0[(size_t)t * C + i] + w0));
+                a = sigmoid_f(to_float(row[4 * C]) + ab);
+            }
+            xs[t * LD + i] = w, bs[t * LD + i] = a, ks[t * LD + i] = k, ys[t * LD + i] = r;
+            V[(i >> 4) * (GC * 16) + t * 16 + (i & 15)] = v;
         }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int t = warp; t < GC; t += GC_THREADS / 32) {
+        float sq = 0.f;
+#pragma unroll
+        for (int i = lane; i < DP; i += 32) sq = fmaf(ks[t * LD + i], ks[t * LD + i], sq);
         sq = warp_sum(sq);
         if (lane == 0) unit[t] = 1.0f / sqrtf(sq + in.unit_eps);
     }
-    for (int e = tid; e < GC * DP; e += GC_THREADS) {
-        const int t = e / DP, i = e - t * DP;
-        float w = 1.f, a = 0.f;
-        if (t < nt && i < d) {
-            w = expf(in.decay_scale * sigmoid_f(z0[(size_t)t * C + i] + __ldg(in.w0 + c0 + i)));
-            a = sigmoid_f(to_float(row0[(size_t)t * in.ld + 4 * C + i]) + __ldg(in.a_bias + c0 + i));
-        }
-        xs[t * LD + i] = w;
-        bs[t * LD + i] = a;
+    float P = 1.f, total = 1.f, ws[TP];
+    const int ci = tid % DP, ct0 = tid / DP * TP;
+#pragma unroll
+    for (int t = 0; t < GC; ++t) {
+        const float w = xs[t * LD + ci];
+        if (t == ct0) P = total;
+        total *= w;
     }
-    __syncthreads();
-    float* M = buf + ((size_t)chunk * in.H + h) * gc_floats(DP);
-    float* W = M + (size_t)(DP + GC) * 2 * GC;
-    float* Pend = W + 2 * GC * DP;
-    float* V = Pend + DP;
-    for (int i = tid; i < DP; i += GC_THREADS) {
-        float P = 1.f, invs[GC], kk[GC], ab[GC];
 #pragma unroll
-        for (int t = 0; t < GC; ++t) {
-            float r = 0.f, k = 0.f, v = 0.f, f = 0.f;
-            if (t < nt && i < d) {
-                const T* row = row0 + (size_t)t * in.ld + i;
-                r = to_float(row[0]), k = to_float(row[C]), v = to_float(row[2 * C]), f = unit[t];
-            }
-            const float u = k * f, au = bs[t * LD + i] * u, w = xs[t * LD + i];
-            xs[t * LD + i] = P * u;
-            P *= w;
-            const float inv = 1.0f / P;
-            invs[t] = inv, kk[t] = k * inv, ab[t] = au * inv;
-            bs[t * LD + i] = ab[t];
-            ks[t * LD + i] = kk[t];
-            ys[t * LD + i] = P * r;
-            V[t * DP + i] = v;
-        }
-        Pend[i] = P;
+    for (int t = 0; t < TP; ++t) ws[t] = xs[(ct0 + t) * LD + ci];
+    __syncthreads();                                    // (`unit`, and every w is read)
+    if (ct0 == 0) Pend[ci] = total;
 #pragma unroll
-        for (int t = 0; t < GC; ++t) {
-            W[t * DP + i] = kk[t] * P;
-            W[(GC + t) * DP + i] = -ab[t] * P;
-        }
+    for (int q = 0; q < TP; ++q) {
+        const int t = ct0 + q;
+        const float k = ks[t * LD + ci], u = k * unit[t], au = bs[t * LD + ci] * u;
+        xs[t * LD + ci] = P * u;
+        P *= ws[q];
+        const float inv = 1.0f / P, kk = k * inv, b = au * inv;
+        bs[t * LD + ci] = b;
+        ks[t * LD + ci] = kk;
+        ys[t * LD + ci] *= P;
+        W[t * DP + ci] = kk * total;
+        W[(GC + t) * DP + ci] = -b * total;
     }
     __syncthreads();
     {
         // a thread per pair (t, s): four dots
-        const int t = tid / GC, q = tid - t * GC;
+        const int q = tid / GC, t = tid - q * GC;
         float xk = 0.f, xb = 0.f, yk = 0.f, yb = 0.f;
+#pragma unroll 4
         for (int i = 0; i < DP; i += 4) {
             const float4 x = *reinterpret_cast<const float4*>(xs + t * LD + i), y = *reinterpret_cast<const float4*>(ys + t * LD + i);
             const float4 k = *reinterpret_cast<const float4*>(ks + q * LD + i), b = *reinterpret_cast<const float4*>(bs + q * LD + i);
@@ -443,56 +447,84 @@ __global__ void __launch_bounds__(GC_THREADS) gd_chunk_prepare_kernel(GdIn in, c
             yk = fmaf(y.x, k.x, fmaf(y.y, k.y, fmaf(y.z, k.z, fmaf(y.w, k.w, yk))));
             yb = fmaf(y.x, b.x, fmaf(y.y, b.y, fmaf(y.z, b.z, fmaf(y.w, b.w, yb))));
         }
-        gram[t * GC + q] = q < t ? xk : 0.f;
-        gram[GC * GC + t * GC + q] = q < t ? xb : 0.f;
-        gram[2 * GC * GC + t * GC + q] = q <= t ? yk : 0.f;
-        gram[3 * GC * GC + t * GC + q] = q <= t ? yb : 0.f;
+        gram[q * GC + t] = q < t ? xk : 0.f;
+        gram[GC * GC + q * GC + t] = q < t ? xb : 0.f;
+        gram[2 * GC * GC + q * GC + t] = q <= t ? yk : 0.f;
+        gram[3 * GC * GC + q * GC + t] = q <= t ? yb : 0.f;
     }
     __syncthreads();
-    // forward substitution, a thread per column of [X | G], then the same column of [Y | H]
+    // forward substitution, a thread per column of [X | G] and the same column of [Y | H]: row by row, each solved entry is
+    // taken out of all entries behind it
     for (int c = tid; c < DP + GC; c += GC_THREADS) {
-        float x[GC];
+        float x[GC], y[GC];
 #pragma unroll
         for (int t = 0; t < GC; ++t) {
-            float acc = c < DP ? xs[t * LD + c] : gram[t * GC + c - DP];
-#pragma unroll
-            for (int q = 0; q < t; ++q) acc = fmaf(-gram[GC * GC + t * GC + q], x[q], acc);
-            x[t] = acc;
+            x[t] = c < DP ? xs[t * LD + c] : gram[(c - DP) * GC + t];
+            y[t] = c < DP ? ys[t * LD + c] : gram[2 * GC * GC + (c - DP) * GC + t];
         }
-        float* m = M + (size_t)c * 2 * GC;
 #pragma unroll
-        for (int t = 0; t < GC; t += 4) *reinterpret_cast<float4*>(m + t) = make_float4(x[t], x[t + 1], x[t + 2], x[t + 3]);
-        float o[4];
+        for (int q = 0; q < GC; ++q) {
+            const float* xb = gram + GC * GC + q * GC;
+            const float* yb = gram + 3 * GC * GC + q * GC;
+#pragma unroll
+            for (int t4 = q / 4 * 4; t4 < GC; t4 += 4) {
+                const float4 a = *reinterpret_cast<const float4*>(xb + t4), b = *reinterpret_cast<const float4*>(yb + t4);
+                if (t4 + 0 > q) x[t4 + 0] = fmaf(-a.x, x[q], x[t4 + 0]);
+                if (t4 + 1 > q) x[t4 + 1] = fmaf(-a.y, x[q], x[t4 + 1]);
+                if (t4 + 2 > q) x[t4 + 2] = fmaf(-a.z, x[q], x[t4 + 2]);
+                if (t4 + 3 > q) x[t4 + 3] = fmaf(-a.w, x[q], x[t4 + 3]);
+                if (t4 + 0 >= q) y[t4 + 0] = fmaf(-b.x, x[q], y[t4 + 0]);
+                if (t4 + 1 >= q) y[t4 + 1] = fmaf(-b.y, x[q], y[t4 + 1]);
+                if (t4 + 2 >= q) y[t4 + 2] = fmaf(-b.z, x[q], y[t4 + 2]);
+                if (t4 + 3 >= q) y[t4 + 3] = fmaf(-b.w, x[q], y[t4 + 3]);
+            }
+        }
 #pragma unroll
         for (int t = 0; t < GC; ++t) {
-            float acc = c < DP ? ys[t * LD + c] : gram[2 * GC * GC + t * GC + c - DP];
-#pragma unroll
-            for (int q = 0; q <= t; ++q) acc = fmaf(-gram[3 * GC * GC + t * GC + q], x[q], acc);
-            o[t & 3] = acc;
-            if ((t & 3) == 3) *reinterpret_cast<float4*>(m + GC + t - 3) = make_float4(o[0], o[1], o[2], o[3]);
+            M[(size_t)t * gc_ld(DP) + c] = x[t];
+            M[(size_t)(GC + t) * gc_ld(DP) + c] = y[t];
         }
     }
 }
 
-// Shared floats of the second kernel: two stages of [matrix | additions | P_end | a block of the values], the state's block
-// of columns, c, and the partial sums of eight warps.
-__host__ __device__ constexpr int gc_stage_floats(int DP) { return (DP + GC) * 2 * GC + 2 * GC * DP + DP + GC * GC_COLS; }
+// The second kernel's tiles: a thread owns GC_R rows x 4 columns of the state's block; the block's rows are so far apart that
+// the reads of a warp's tiles meet no bank twice.
+__host__ __device__ constexpr int gc_r(int DP) { return DP >= 64 ? DP / 64 : 1; }
+__host__ __device__ constexpr int gc_sld(int DP) { return gc_r(DP) == 1 ? 16 : gc_r(DP) == 2 ? 24 : 20; }
+// Its shared floats: two stages of [matrix | additions | P_end | a block of the values], the state's block of columns, c, and
+// the partial sums of eight warps.
+__host__ __device__ constexpr int gc_stage_floats(int DP) { return gc_fixed(DP) + GC * GC_COLS; }
 __host__ __device__ constexpr int gc_scan_smem(int DP) {
-    return (2 * gc_stage_floats(DP) + DP * GC_COLS + GC * GC_COLS + 8 * 2 * GC * GC_COLS) * (int)sizeof(float);
+    return (2 * gc_stage_floats(DP) + DP * gc_sld(DP) + GC * GC_COLS + 8 * 2 * GC * GC_COLS) * (int)sizeof(float);
+}
+
+template <int R>
+__device__ __forceinline__ void gc_rows(const float* p, float (&w)[R]) {
+    if (R == 2) {
+        const float2 v = *reinterpret_cast<const float2*>(p);
+        w[0] = v.x, w[R > 1 ? 1 : 0] = v.y;
+    } else if (R == 4) {
+        const float4 v = *reinterpret_cast<const float4*>(p);
+        w[0] = v.x, w[R > 1 ? 1 : 0] = v.y, w[R > 2 ? 2 : 0] = v.z, w[R > 3 ? 3 : 0] = v.w;
+    } else {
+        w[0] = p[0];
+    }
 }
 
 // grid: (requests, heads, blocks of 16 columns); 256 threads.  Per chunk: the 2 GC x 16 product over the DP + GC rows of state
-// and values, cut between the eight warps (tiles of 4 x 4 per thread) and summed in a fixed order; then the state's update.
+// and values, cut between the eight warps (tiles of 4 x 4 per thread) and summed in a fixed order; then the state's update,
+// whose part that does not wait for the sums runs in front of them.
 template <int DP>
 __global__ void __launch_bounds__(GC_THREADS) gd_chunk_scan_kernel(int H, int d, const float* __restrict__ buf, float* __restrict__ state,
                                                                    long long state_stride, const int* __restrict__ cu_q,
                                                                    const int* __restrict__ slots, float* __restrict__ out) {
-    constexpr int STAGE = gc_stage_floats(DP), KW = (DP + GC) / 8, MF = (DP + GC) * 2 * GC + 2 * GC * DP + DP;
-    static_assert((DP + GC) % 8 == 0 && MF % 4 == 0, "");
+    constexpr int STAGE = gc_stage_floats(DP), FIXED = gc_fixed(DP), LDM = gc_ld(DP), SLD = gc_sld(DP), R = gc_r(DP);
+    constexpr int QUADS = (DP + GC) / 4, BASE = QUADS / 8;           // quads of k: the first four warps take one more
+    static_assert(QUADS == 8 * BASE + 4 && FIXED % 4 == 0, "");
     extern __shared__ __align__(16) float gc_smem_raw[];
-    float* Ss = gc_smem_raw + 2 * STAGE;                // [DP][16]
-    float* Cs = Ss + DP * GC_COLS;                      // [GC][16]
-    float* part = Cs + GC * GC_COLS;                    // [8][2 GC][16]
+    float* Ss = gc_smem_raw + 2 * STAGE;                // [DP][SLD]
+    float* Cs = Ss + DP * SLD;                          // [GC][16]
+    float* part = Cs + GC * GC_COLS;                    // [8 warps][4][32 lanes][4]
     const int s = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * GC_COLS;
     const int slot = slots[s];
     const int q0 = cu_q[s], nq = cu_q[s + 1] - q0;
@@ -505,19 +537,18 @@ __global__ void __launch_bounds__(GC_THREADS) gd_chunk_scan_kernel(int H, int d,
     auto stage = [&](int c, int b) {
         float* dst = gc_smem_raw + b * STAGE;
         const float* src = src0 + (size_t)c * H * per;
-        for (int e = tid; e < MF / 4; e += GC_THREADS) gd_cp16(dst + e * 4, src + e * 4);
-        const float* v = src + MF + j0;                 // the values' columns j0 .. j0 + 15 (DP is a multiple of 16)
-        if (tid < GC * GC_COLS / 4) gd_cp16(dst + MF + tid * 4, v + (tid >> 2) * DP + (tid & 3) * 4);
+        for (int e = tid; e < FIXED / 4; e += GC_THREADS) gd_cp16(dst + e * 4, src + e * 4);
+        if (tid < GC * GC_COLS / 4) gd_cp16(dst + FIXED + tid * 4, src + FIXED + (size_t)blockIdx.z * GC * GC_COLS + tid * 4);
         asm volatile("cp.async.commit_group;\n" ::);
     };
     stage(0, 0);
     for (int e = tid; e < GC_COLS * DP; e += GC_THREADS) {
         const int j = e / DP, k = e - j * DP;
-        Ss[k * GC_COLS + j] = j0 + j < d && k < d ? sp[(size_t)(j0 + j) * d + k] : 0.f;
+        Ss[k * SLD + j] = j0 + j < d && k < d ? sp[(size_t)(j0 + j) * d + k] : 0.f;
     }
-    const int rt = (lane >> 2) * 4, ct = (lane & 3) * 4;             // the product's tile of this thread
-    constexpr int R = DP >= 64 ? DP / 64 : 1;                        // rows of the state's tile
-    const int sr = (tid >> 2) * R, sc = (tid & 3) * 4;
+    const int rg = lane >> 2, ct = (lane & 3) * 4;                   // rows rg, rg + 8, .. of the product, columns ct .. ct + 3
+    const int g_lo = warp * BASE + min(warp, 4), g_hi = g_lo + BASE + (warp < 4 ? 1 : 0);
+    const int sr = (tid >> 2) * R, sc = ct;
     const bool owns = sr < DP;
     for (int c = 0; c < chunks; ++c) {
         const int b = c & 1, nt = min(GC, nq - c * GC);
@@ -525,7 +556,7 @@ __global__ void __launch_bounds__(GC_THREADS) gd_chunk_scan_kernel(int H, int d,
         __syncthreads();
         if (c + 1 < chunks) stage(c + 1, b ^ 1);
         const float* M = gc_smem_raw + b * STAGE;
-        const float* W = M + (DP + GC) * 2 * GC;
+        const float* W = M + 2 * GC * LDM;
         const float* Pend = W + 2 * GC * DP;
         const float* V = Pend + DP;
         float acc[4][4];
@@ -533,47 +564,61 @@ __global__ void __launch_bounds__(GC_THREADS) gd_chunk_scan_kernel(int H, int d,
         for (int i = 0; i < 4; ++i)
 #pragma unroll
             for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
-#pragma unroll 6
-        for (int kk = 0; kk < KW; ++kk) {
-            const int k = warp * KW + kk;
-            const float4 m = *reinterpret_cast<const float4*>(M + k * 2 * GC + rt);
-            const float4 x = *reinterpret_cast<const float4*>((k < DP ? Ss + k * GC_COLS : V + (k - DP) * GC_COLS) + ct);
-            const float mm[4] = {m.x, m.y, m.z, m.w}, xx[4] = {x.x, x.y, x.z, x.w};
 #pragma unroll
-            for (int i = 0; i < 4; ++i)
+        for (int gi = 0; gi < BASE + 1; ++gi) {
+            const int k4 = (g_lo + gi) * 4;
+            if (gi == BASE && g_lo + gi >= g_hi) break;              // uniform per warp
+            const float* xp = k4 < DP ? Ss + k4 * SLD + ct : V + (k4 - DP) * GC_COLS + ct;
+            const int xs = k4 < DP ? SLD : GC_COLS;
+            float4 m[4], x[4];
 #pragma unroll
-                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(mm[i], xx[j], acc[i][j]);
+            for (int i = 0; i < 4; ++i) {
+                m[i] = *reinterpret_cast<const float4*>(M + (rg + 8 * i) * LDM + k4);
+                x[i] = *reinterpret_cast<const float4*>(xp + i * xs);
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float mm[4] = {m[i].x, m[i].y, m[i].z, m[i].w};
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    acc[i][0] = fmaf(mm[k], x[k].x, acc[i][0]), acc[i][1] = fmaf(mm[k], x[k].y, acc[i][1]);
+                    acc[i][2] = fmaf(mm[k], x[k].z, acc[i][2]), acc[i][3] = fmaf(mm[k], x[k].w, acc[i][3]);
+                }
+            }
         }
 #pragma unroll
         for (int i = 0; i < 4; ++i)
-            *reinterpret_cast<float4*>(part + (warp * 2 * GC + rt + i) * GC_COLS + ct) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+            *reinterpret_cast<float4*>(part + ((warp * 4 + i) * 32 + lane) * 4) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
         // what does not wait for c: the decayed state and the values' part
         float st[R][4];
         if (owns) {
+            float p[R];
+            gc_rows<R>(Pend + sr, p);
 #pragma unroll
             for (int r = 0; r < R; ++r) {
-                const float p = Pend[sr + r];
-                const float4 x = *reinterpret_cast<const float4*>(Ss + (sr + r) * GC_COLS + sc);
-                st[r][0] = p * x.x, st[r][1] = p * x.y, st[r][2] = p * x.z, st[r][3] = p * x.w;
+                const float4 x = *reinterpret_cast<const float4*>(Ss + (sr + r) * SLD + sc);
+                st[r][0] = p[r] * x.x, st[r][1] = p[r] * x.y, st[r][2] = p[r] * x.z, st[r][3] = p[r] * x.w;
             }
-#pragma unroll 4
+#pragma unroll 8
             for (int q = 0; q < GC; ++q) {
                 const float4 x = *reinterpret_cast<const float4*>(V + q * GC_COLS + sc);
+                float w[R];
+                gc_rows<R>(W + q * DP + sr, w);
 #pragma unroll
                 for (int r = 0; r < R; ++r) {
-                    const float w = W[q * DP + sr + r];
-                    st[r][0] = fmaf(w, x.x, st[r][0]), st[r][1] = fmaf(w, x.y, st[r][1]);
-                    st[r][2] = fmaf(w, x.z, st[r][2]), st[r][3] = fmaf(w, x.w, st[r][3]);
+                    st[r][0] = fmaf(w[r], x.x, st[r][0]), st[r][1] = fmaf(w[r], x.y, st[r][1]);
+                    st[r][2] = fmaf(w[r], x.z, st[r][2]), st[r][3] = fmaf(w[r], x.w, st[r][3]);
                 }
             }
         }
         __syncthreads();
         {
-            const int row = tid >> 3, col = (tid & 7) * 2;
+            const int i = tid >> 6, l = (tid >> 1) & 31, half = (tid & 1) * 2;
+            const int row = (l >> 2) + 8 * i, col = (l & 3) * 4 + half;
             float a0 = 0.f, a1 = 0.f;
 #pragma unroll
             for (int w = 0; w < 8; ++w) {
-                const float2 x = *reinterpret_cast<const float2*>(part + (w * 2 * GC + row) * GC_COLS + col);
+                const float2 x = *reinterpret_cast<const float2*>(part + ((w * 4 + i) * 32 + l) * 4 + half);
                 a0 += x.x, a1 += x.y;
             }
             if (row < GC) {
@@ -586,25 +631,26 @@ __global__ void __launch_bounds__(GC_THREADS) gd_chunk_scan_kernel(int H, int d,
         }
         __syncthreads();
         if (owns) {
-#pragma unroll 4
+#pragma unroll 8
             for (int q = 0; q < GC; ++q) {
                 const float4 x = *reinterpret_cast<const float4*>(Cs + q * GC_COLS + sc);
+                float w[R];
+                gc_rows<R>(W + (GC + q) * DP + sr, w);
 #pragma unroll
                 for (int r = 0; r < R; ++r) {
-                    const float w = W[(GC + q) * DP + sr + r];
-                    st[r][0] = fmaf(w, x.x, st[r][0]), st[r][1] = fmaf(w, x.y, st[r][1]);
-                    st[r][2] = fmaf(w, x.z, st[r][2]), st[r][3] = fmaf(w, x.w, st[r][3]);
+                    st[r][0] = fmaf(w[r], x.x, st[r][0]), st[r][1] = fmaf(w[r], x.y, st[r][1]);
+                    st[r][2] = fmaf(w[r], x.z, st[r][2]), st[r][3] = fmaf(w[r], x.w, st[r][3]);
                 }
             }
 #pragma unroll
             for (int r = 0; r < R; ++r)
-                *reinterpret_cast<float4*>(Ss + (sr + r) * GC_COLS + sc) = make_float4(st[r][0], st[r][1], st[r][2], st[r][3]);
+                *reinterpret_cast<float4*>(Ss + (sr + r) * SLD + sc) = make_float4(st[r][0], st[r][1], st[r][2], st[r][3]);
         }
     }
     __syncthreads();
     for (int e = tid; e < GC_COLS * DP; e += GC_THREADS) {
         const int j = e / DP, k = e - j * DP;
-        if (j0 + j < d && k < d) sp[(size_t)(j0 + j) * d + k] = Ss[k * GC_COLS + j];
+        if (j0 + j < d && k < d) sp[(size_t)(j0 + j) * d + k] = Ss[k * SLD + j];
     }
 }
 
