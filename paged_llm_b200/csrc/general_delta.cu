@@ -355,7 +355,7 @@ __host__ __device__ constexpr size_t gc_floats(int DP) { return (size_t)gc_fixed
 __host__ __device__ constexpr int gc_prepare_smem(int DP) { return (4 * GC * (DP + 4) + 4 * GC * GC + GC) * (int)sizeof(float); }
 
 template <typename T, int DP>
-__global__ void __launch_bounds__(GC_THREADS) gd_chunk_prepare_kernel(GdIn in, const float* __restrict__ z, const int* __restrict__ cu_q,
+__global__ void __launch_bounds__(GC_THREADS, DP <= 128 ? 4 : 1) gd_chunk_prepare_kernel(GdIn in, const float* __restrict__ z, const int* __restrict__ cu_q,
                                                                       const int* __restrict__ slots, int num_seqs, float* __restrict__ buf) {
     constexpr int LD = DP + 4;                          // rows 4 floats longer: 16-byte reads of eight rows meet no bank twice
     constexpr int PARTS = GC_THREADS / DP, TP = GC / PARTS;          // threads per channel, tokens of each
@@ -660,6 +660,7 @@ int launch_gd_chunks(const GdIn& in, const float* z, float* buf, int slots_of_ch
     static bool opted = false;
     if (!opted) {
         PL_CUDA(cudaFuncSetAttribute(gd_chunk_prepare_kernel<T, DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, gc_prepare_smem(DP)));
+        PL_CUDA(cudaFuncSetAttribute(gd_chunk_prepare_kernel<T, DP>, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared));
         PL_CUDA(cudaFuncSetAttribute(gd_chunk_scan_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, gc_scan_smem(DP)));
         opted = true;
     }

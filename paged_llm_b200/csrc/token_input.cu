@@ -12,22 +12,46 @@
 // ------------------------------------------------------------------ embedding + sinusoidal position
 // out[t, 2i] = table[id, 2i] * scale + sin(2 pi p turns[i]), out[t, 2i+1] the same with cos; p the token's position.
 // `turns` (turns of the circle per position) and the reduction to one turn are double, so that the phase is exact far out.
+__device__ __forceinline__ float4 quad(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 quad(const __nv_bfloat16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&raw.x), b = *reinterpret_cast<const __nv_bfloat162*>(&raw.y);
+    return make_float4(__low2float(a), __high2float(a), __low2float(b), __high2float(b));
+}
+
+__device__ __forceinline__ void sinusoid(double turns, double p, float& sn, float& cs) {
+    const double ph = p * turns;
+    sincospif(2.0f * (float)(ph - rint(ph)), &sn, &cs);
+}
+
+// grid: (blocks of a row, tokens).  vec: four elements per thread (H % 4 == 0, 16-byte aligned rows).
 template <typename TW>
 __global__ void __launch_bounds__(128) embedding_sinusoid_kernel(const TW* __restrict__ table, const int* __restrict__ ids,
                                                                  const int* __restrict__ positions, const double* __restrict__ turns,
-                                                                 float* __restrict__ out, int H, int V, float scale) {
+                                                                 float* __restrict__ out, int H, int V, float scale, int vec) {
     pdl_launch_dependents();
-    pdl_wait();
+    const int first = blockIdx.x * blockDim.x + threadIdx.x, stride = gridDim.x * blockDim.x;
     const int t = blockIdx.y;
+    pdl_wait();
     const int id = ids[t];
     const double p = (double)positions[t];
     const bool valid = id >= 0 && id < V;
     const TW* row = table + (size_t)(valid ? id : 0) * H;
     float* o = out + (size_t)t * H;
-    for (int i = blockIdx.x * blockDim.x + threadIdx.x; 2 * i < H; i += gridDim.x * blockDim.x) {
-        const double ph = p * turns[i];
+    if (vec) {
+        for (int c = first * 4; c < H; c += stride * 4) {
+            const double2 tu = *reinterpret_cast<const double2*>(turns + c / 2);
+            float4 v = quad(row + c), e;
+            if (!valid) v = make_float4(0.f, 0.f, 0.f, 0.f);
+            sinusoid(tu.x, p, e.x, e.y);
+            sinusoid(tu.y, p, e.z, e.w);
+            *reinterpret_cast<float4*>(o + c) = make_float4(fmaf(v.x, scale, e.x), fmaf(v.y, scale, e.y), fmaf(v.z, scale, e.z), fmaf(v.w, scale, e.w));
+        }
+        return;
+    }
+    for (int i = first; 2 * i < H; i += stride) {
         float sn, cs;
-        sincospif(2.0f * (float)(ph - rint(ph)), &sn, &cs);
+        sinusoid(turns[i], p, sn, cs);
         o[2 * i] = (valid ? to_float(row[2 * i]) * scale : 0.f) + sn;
         if (2 * i + 1 < H) o[2 * i + 1] = (valid ? to_float(row[2 * i + 1]) * scale : 0.f) + cs;
     }
@@ -38,15 +62,16 @@ PL_EXPORT int pl_embedding_sinusoid(const void* table, int table_dtype, const in
     if (T == 0) return 0;
     PL_REQUIRE(T > 0 && H > 0 && V > 0, "embedding_sinusoid: bad sizes T=%d H=%d V=%d", T, H, V);
     PL_REQUIRE(T <= 65535 * 32, "embedding_sinusoid: %d tokens", T);
-    const int bx = (H / 2 + 127) / 128 > 0 ? (H / 2 + 127) / 128 : 1;
+    const int vec = H % 4 == 0 && (((uintptr_t)table | (uintptr_t)out | (uintptr_t)turns) & 15) == 0;
+    const int bx = ((vec ? H / 4 : (H + 1) / 2) + 127) / 128;
     for (int t0 = 0; t0 < T; t0 += 65535) {                       // (the y extent of a grid)
         const int n = T - t0 < 65535 ? T - t0 : 65535;
         if (table_dtype == PL_F32)
             PL_CUDA(launch_pdl(embedding_sinusoid_kernel<float>, dim3(bx, n), dim3(128), 0, stream, (const float*)table, ids + t0,
-                               positions + t0, turns, out + (size_t)t0 * H, H, V, scale));
+                               positions + t0, turns, out + (size_t)t0 * H, H, V, scale, vec));
         else if (table_dtype == PL_BF16)
             PL_CUDA(launch_pdl(embedding_sinusoid_kernel<__nv_bfloat16>, dim3(bx, n), dim3(128), 0, stream, (const __nv_bfloat16*)table,
-                               ids + t0, positions + t0, turns, out + (size_t)t0 * H, H, V, scale));
+                               ids + t0, positions + t0, turns, out + (size_t)t0 * H, H, V, scale, vec));
         else
             return pl_fail("embedding_sinusoid: unknown dtype %d", table_dtype);
     }
@@ -54,13 +79,6 @@ PL_EXPORT int pl_embedding_sinusoid(const void* table, int table_dtype, const in
 }
 
 // ------------------------------------------------------------------ residual sum + a copy in the activations' type
-__device__ __forceinline__ float4 quad(const float* p) { return *reinterpret_cast<const float4*>(p); }
-__device__ __forceinline__ float4 quad(const __nv_bfloat16* p) {
-    const uint2 raw = *reinterpret_cast<const uint2*>(p);
-    const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&raw.x), b = *reinterpret_cast<const __nv_bfloat162*>(&raw.y);
-    return make_float4(__low2float(a), __high2float(a), __low2float(b), __high2float(b));
-}
-
 template <typename TB>
 __global__ void __launch_bounds__(256) add_copy_kernel(float* __restrict__ x, const TB* __restrict__ branch,
                                                        __nv_bfloat16* __restrict__ copy, long long n, int vec) {
