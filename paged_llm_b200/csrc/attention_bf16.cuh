@@ -209,6 +209,15 @@ __global__ void __launch_bounds__(32 * MW * NW) attn_bf16_kernel(AttnParams p) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) oacc[j][e] = 0.f;
     const float scale_log2 = p.scale * LOG2E;
+    // (with modifiers) the first and last position of this warp's rows that see anything, and the highest first key
+    // among them: a tile whose keys all of them see needs no mask
+    int pos_lo = 0, first_hi = 0;
+    bool has_bias = false;
+    if (MOD) {
+        pos_lo = __reduce_min_sync(0xffffffffu, min(pos[0] < 0 ? 0x7fffffff : pos[0], pos[1] < 0 ? 0x7fffffff : pos[1]));
+        first_hi = __reduce_max_sync(0xffffffffu, max(pos[0] < 0 ? 0 : first[0], pos[1] < 0 ? 0 : first[1]));
+        has_bias = p.dist_bias != nullptr;
+    }
 
     const int n_tiles = (main_hi - it.key_lo + BN - 1) / BN;
     // The first keys are on their way while Q is fetched.  A cluster block has not waited for the
@@ -266,6 +275,19 @@ __global__ void __launch_bounds__(32 * MW * NW) attn_bf16_kernel(AttnParams p) {
         const __nv_bfloat16* vst = Vs + stage * BN * PITCH + wn * KPW * PITCH;
         const int kbase = tile_lo + wn * KPW;
         if (kbase < hi_cur) {                                  // uniform per warp
+            // the biases of this thread's scores are asked for before the product (a key behind the query reads entry 0)
+            float bz[MOD ? KPW / 8 : 1][4];
+            if (MOD) {
+#pragma unroll
+                for (int j = 0; j < KPW / 8; ++j)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const int place = kbase + 8 * j + 2 * t4 + (e & 1);
+                        const int n = place >= p.keep_first ? place + it.gap : place;
+                        bz[j][e] = has_bias && brow[e >> 1] != nullptr
+                                       ? __ldg(brow[e >> 1] + min(max(pos[e >> 1] - n, 0), p.dist_len - 1)) * LOG2E : 0.f;
+                    }
+            }
             float sacc[KPW / 8][4];
 #pragma unroll
             for (int j = 0; j < KPW / 8; ++j)
@@ -290,12 +312,17 @@ __global__ void __launch_bounds__(32 * MW * NW) attn_bf16_kernel(AttnParams p) {
                                                                         pos[1] < 0 ? 0x7fffffff : pos[1]));
             const bool full_tile = !modified && p.window <= 0 && p.chunk <= 0 && kbase + KPW <= hi_cur && kbase + KPW - 1 <= pos_min_warp;
             float mx[2] = {-INFINITY, -INFINITY};
-            if (full_tile) {
+            bool mod_full = false;
+            if (MOD && p.softcap <= 0.f && p.slopes == nullptr && kbase + KPW <= hi_cur) {
+                const int k0 = kbase >= p.keep_first ? kbase + it.gap : kbase, k1 = kbase + KPW - 1 + (kbase + KPW - 1 >= p.keep_first ? it.gap : 0);
+                mod_full = k1 <= pos_lo && (k0 >= first_hi || kbase + KPW <= p.keep_first);
+            }
+            if (full_tile || mod_full) {
 #pragma unroll
                 for (int j = 0; j < KPW / 8; ++j)
 #pragma unroll
                     for (int e = 0; e < 4; ++e) {
-                        const float s = sacc[j][e] * scale_log2;
+                        const float s = MOD ? fmaf(sacc[j][e], scale_log2, bz[j][e]) : sacc[j][e] * scale_log2;
                         sacc[j][e] = s;
                         mx[e >> 1] = fmaxf(mx[e >> 1], s);
                     }
@@ -309,7 +336,7 @@ __global__ void __launch_bounds__(32 * MW * NW) attn_bf16_kernel(AttnParams p) {
                         const int pr = pos[e >> 1];
                         const bool vis = place < hi_cur && n <= pr && (n >= first[e >> 1] || (MOD && n < p.keep_first));
                         const float s = !vis ? -INFINITY
-                                        : modified ? attn_score(p, sacc[j][e], slope[e >> 1], n, pr, brow[e >> 1]) * LOG2E
+                                        : modified ? fmaf(attn_score(p, sacc[j][e], slope[e >> 1], n, pr), LOG2E, bz[j][e])
                                                    : sacc[j][e] * scale_log2;
                         sacc[j][e] = s;
                         mx[e >> 1] = fmaxf(mx[e >> 1], s);
@@ -693,8 +720,13 @@ PL_EXPORT int PL_CAT(pl_attention_bf16_d, PL_DPAD)(const AttnParams* params, cud
                                             "do not combine");
         // the score modifiers live in instantiations of their own of the mma.sync kernel (the tcgen05
         // kernels step aside for them)
+#if PL_DPAD == 64
+        if (p.cluster > 0) return launch_attn_cluster<PL_DPAD, 16, true, 2, 8, false, true>(p, stream);
+        if (p.is_small) return launch_attn_bf16<PL_DPAD, 1, 8, 16, true, 2, true>(p, stream);
+#else
         if (p.cluster > 0) return launch_attn_cluster<PL_DPAD, KPW_CLUSTER, true, 2, 4, false, true>(p, stream);
         if (p.is_small) return launch_attn_bf16<PL_DPAD, 1, 4, KPW_CLUSTER, true, 2, true>(p, stream);
+#endif
         return launch_attn_bf16<PL_DPAD, PL_LARGE_MW, 1, 64, true>(p, stream);
     }
     // All forms of the small shape run warp-private copy pipelines (WP): 49 against 53 us at 64 requests x

@@ -356,7 +356,21 @@ struct Shape {
     static constexpr int Q_PANEL = BM * 128, K_PANEL = BN * 128;
     static constexpr int Q_BYTES = PANELS * Q_PANEL, K_BYTES = PANELS * K_PANEL;
     static constexpr int SMEM_BYTES = Q_BYTES + 2 * STAGES * K_BYTES + 1024;
+    // A learned bias by distance, staged per key tile by the warp that brings the keys: per head of the group the distances
+    // between the block's tokens and the tile's keys.  S(m) is only issued once the softmax is done with tile m - 2, and a
+    // stage of keys is refilled once its S is done, so with STAGES + 2 slots the one being filled is never still read.
+    static constexpr int BIAS_SLOTS = STAGES + 2, BIAS_FLOATS = 800;
+    static constexpr int SMEM_BIAS = SMEM_BYTES + BIAS_SLOTS * BIAS_FLOATS * 4;
 };
+
+// Floats between the heads' rows of a slot: as many as a row needs, and such that the lanes of a warp (G heads of 32 / G
+// consecutive tokens) read different banks.
+__host__ __device__ inline int bias_row_floats(int G) {
+    const int span = (BM + G - 1) / G + 1 + BN - 1, want = 32 / G;
+    int n = span;
+    while (want > 0 && n % 32 != want % 32) ++n;
+    return n;
+}
 
 __device__ __forceinline__ void mbar_arrive(uint64_t* bar) {
     asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(saddr(bar)) : "memory");
@@ -419,7 +433,9 @@ __device__ __forceinline__ void tmem_ld64(uint32_t taddr, float (&v)[64]) {
 
 // WIDE (head size 128 only): O += P V as one product 128 x 128 x 16 per step, the value panels
 // being the two 64-column groups of its MN-major operand, instead of one product per panel.
-template <int D, bool WIDE>
+// BIAS: 0 neither a bias by distance nor kept first keys (the kernel of plain prompts carries none of their code), 1 a bias,
+// if any, is read from its table per score, 2 it is staged in shared memory; first keys may be kept with 1 and 2.
+template <int D, bool WIDE, int BIAS>
 __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, const __grid_constant__ CUtensorMap kv_map) {
     using SH = Shape<D>;
     constexpr int PANELS = SH::PANELS, STAGES = SH::STAGES, Q_PANEL = SH::Q_PANEL, K_PANEL = SH::K_PANEL;
@@ -436,21 +452,26 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
     unsigned char* Vs = Ks + STAGES * K_BYTES;                 // [STAGES][PANELS][64 keys][128 B]
     __shared__ uint64_t k_full[STAGES], k_empty[STAGES], v_full[STAGES], v_empty[STAGES];
     __shared__ uint64_t s_full[2], p_full[2], pv_done[2];
+    __shared__ uint64_t b_full[BIAS == 2 ? SH::BIAS_SLOTS : 1];
     __shared__ uint32_t tmem_base_slot;
+    float* bias_slots = reinterpret_cast<float*>(Vs + STAGES * K_BYTES);
 
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int kvh = blockIdx.x % p.nkv, G = p.nh / p.nkv;
     const __nv_bfloat16* q = (const __nv_bfloat16*)p.q;
+    const int pos_first = it.lk - it.nq + it.row_base / G;     // position of the block's first token
+    const int bias_ld = BIAS == 2 ? bias_row_floats(G) : 0;
     // Keys [0, kept) and [key_lo, key_hi), by position: the first keys of the request kept beside the window, if any,
     // and the item's window.  Tiles start at multiples of 64; the kept keys' tiles come first unless one of them is the
     // window's first tile.
-    const int kept = it.gap > 0 ? p.keep_first : 0;
-    const int key_lo = it.gap > 0 ? p.keep_first + it.gap : it.key_lo, key_hi = it.key_hi + it.gap;
-    const int near_tile = kept > 0 && ((kept + BN - 1) & ~(BN - 1)) > key_lo ? 0 : key_lo & ~(BN - 1);
-    const int kept_tiles = near_tile > 0 ? (kept + BN - 1) / BN : 0;
+    constexpr bool KEEP = BIAS != 0;
+    const int kept = KEEP && it.gap > 0 ? p.keep_first : 0;
+    const int key_lo = KEEP && it.gap > 0 ? p.keep_first + it.gap : it.key_lo, key_hi = KEEP ? it.key_hi + it.gap : it.key_hi;
+    const int near_tile = KEEP && kept > 0 && ((kept + BN - 1) & ~(BN - 1)) > key_lo ? 0 : key_lo & ~(BN - 1);
+    const int kept_tiles = KEEP && near_tile > 0 ? (kept + BN - 1) / BN : 0;
     const int n_tiles = kept_tiles + (key_hi - near_tile + BN - 1) / BN;
-    auto tile_key = [&](int t) { return t < kept_tiles ? t * BN : near_tile + (t - kept_tiles) * BN; };
-    auto in_range = [&](int n) { return n < kept || (n >= key_lo && n < key_hi); };
+    auto tile_key = [&](int t) { return KEEP && t < kept_tiles ? t * BN : near_tile + (t - kept_tiles) * BN; };
+    auto in_range = [&](int n) { return (KEEP && n < kept) || (n >= key_lo && n < key_hi); };
 
     if (warp == MMA_WARP) {
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n" ::"r"(saddr(&tmem_base_slot)),
@@ -469,6 +490,8 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
             mbar_init(&p_full[b], SOFTMAX_WARPS * 32);
             mbar_init(&pv_done[b], 1);
         }
+        if (BIAS == 2)
+            for (int b = 0; b < SH::BIAS_SLOTS; ++b) mbar_init(&b_full[b], 32);
         asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
     }
     // Q tile: row R = token * G + head; eight 16-byte chunks per row and panel
@@ -498,7 +521,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
         uint64_t* empty = values ? v_empty : k_empty;
         auto page_of = [&](int t) {                             // page of this lane's box of tile t, or -1
             const int n0 = tile_key(t) + lane * box_rows;
-            if (t >= n_tiles || lane >= boxes || n0 >= key_hi || (n0 + box_rows <= key_lo && n0 >= kept)) return -1;
+            if (t >= n_tiles || lane >= boxes || n0 >= key_hi || (n0 + box_rows <= key_lo && (!KEEP || n0 >= kept))) return -1;
             return bt[n0 >> p.ps_shift];
         };
         int pg_next = page_of(0);
@@ -517,6 +540,17 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
 #pragma unroll
                 for (int c = 0; c < PANELS; ++c)
                     tma_box(ring + s * K_BYTES + c * K_PANEL + lane * box_bytes, &kv_map, c * 64, row, &full[s]);
+            }
+            if (BIAS == 2 && !values) {
+                // entry x of head hh: the bias of distance pos_first - (the tile's last key) + x, in units of the raw product
+                float* slot = bias_slots + (t % SH::BIAS_SLOTS) * SH::BIAS_FLOATS;
+                const int d0 = pos_first - tile_key(t) - (BN - 1), span = (BM + G - 1) / G + BN, far = p.dist_len - 1;
+                const float unit = 1.f / p.scale;
+                for (int hh = 0; hh < G; ++hh) {
+                    const float* src = p.dist_bias + (size_t)(kvh * G + hh) * p.dist_len;
+                    for (int x = lane; x < span; x += 32) slot[hh * bias_ld + x] = __ldg(src + min(max(d0 + x, 0), far)) * unit;
+                }
+                mbar_arrive(&b_full[t % SH::BIAS_SLOTS]);
             }
         }
     } else if (warp == MMA_WARP) {
@@ -581,9 +615,9 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
         const bool capped = p.softcap > 0.f;
         const float cap_in = capped ? 2.f * 1.4426950408889634f * p.scale / p.softcap : 0.f;
         const float cap_out = capped ? p.softcap / p.scale : 0.f;
-        const float* bias_row = p.dist_bias != nullptr && R < it.rows_total
-                                    ? p.dist_bias + (size_t)(kvh * G + R % G) * p.dist_len : nullptr;
+        const float* bias_row = BIAS == 1 && p.dist_bias != nullptr && R < it.rows_total ? p.dist_bias + (size_t)(kvh * G + R % G) * p.dist_len : nullptr;
         const float bias_unit = 1.f / p.scale;
+        const int bias_at = BIAS == 2 && R < it.rows_total ? (R % G) * bias_ld + (R / G - it.row_base / G) + BN - 1 : BN - 1;
         float m_run = -INFINITY, l_run = 0.f;
         float sv[64];
         for (int t = 0; t < n_tiles; ++t) {
@@ -601,7 +635,14 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
                     sv[i] = fmaf(-2.f * cap_out, r, cap_out);
                 }
             }
-            if (bias_row != nullptr) {
+            if (BIAS == 2) {
+                const int b6 = t % SH::BIAS_SLOTS;
+                mbar_wait(&b_full[b6], (t / SH::BIAS_SLOTS) & 1);
+                const float* bs = bias_slots + b6 * SH::BIAS_FLOATS + bias_at;
+#pragma unroll
+                for (int i = 0; i < 64; ++i) sv[i] += bs[-i];
+            }
+            if (BIAS == 1 && bias_row != nullptr) {
                 // a learned bias by distance, brought into the units of the raw product (the scale comes below); a
                 // key behind the query reads entry 0 and is masked below
                 const int far = p.dist_len - 1;
@@ -609,13 +650,13 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
                 for (int i = 0; i < 64; ++i)
                     sv[i] = fmaf(__ldg(bias_row + min(max(pos - kbase - i, 0), far)), bias_unit, sv[i]);
             }
-            const bool row_full = ((kbase >= key_lo && kbase >= first) || kbase + BN <= kept) && kbase + BN <= key_hi && kbase + BN - 1 <= pos;
+            const bool row_full = ((kbase >= key_lo && kbase >= first) || (KEEP && kbase + BN <= kept)) && kbase + BN <= key_hi && kbase + BN - 1 <= pos;
             const bool warp_full = __all_sync(0xffffffffu, row_full);
             if (!warp_full) {
 #pragma unroll
                 for (int i = 0; i < 64; ++i) {
                     const int n = kbase + i;
-                    const bool vis = in_range(n) && n <= pos && (n >= first || n < p.keep_first);
+                    const bool vis = in_range(n) && n <= pos && (n >= first || (KEEP && n < p.keep_first));
                     sv[i] = vis ? sv[i] : -INFINITY;
                 }
             }
@@ -664,7 +705,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
                     tmem_st_wait();
                 }
             }
-            if (kbase + BN > kept && (kbase < key_lo || kbase + BN > key_hi)) {
+            if ((!KEEP || kbase + BN > kept) && (kbase < key_lo || kbase + BN > key_hi)) {
                 // Value rows of keys outside the range are zeroed, so that 0 * anything stays 0 (a
                 // page may hold anything behind the last token).
                 mbar_wait(&v_full[t % STAGES], (t / STAGES) & 1);
@@ -723,30 +764,38 @@ inline bool takes(const AttnParams& p) {
            ((uintptr_t)p.kv & 15) == 0;
 }
 
-template <int D, bool WIDE>
+template <int D, bool WIDE, int BIAS>
 inline int launch_as(const AttnParams& p, cudaStream_t stream) {
     static bool attr_set = false;
-    auto kernel = attn_tc2_kernel<D, WIDE>;
+    auto kernel = attn_tc2_kernel<D, WIDE, BIAS>;
+    constexpr int smem = BIAS == 2 ? Shape<D>::SMEM_BIAS : Shape<D>::SMEM_BYTES;
     if (!attr_set) {
-        PL_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, Shape<D>::SMEM_BYTES));
+        PL_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
         PL_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout,
                                      (int)cudaSharedmemCarveoutMaxShared));
         attr_set = true;
     }
     alignas(64) CUtensorMap map;
     if (!kv_tensor_map(&map, p)) return 1;
-    PL_CUDA(launch_pdl(kernel, dim3(p.n_work * p.nkv), dim3(THREADS), (size_t)Shape<D>::SMEM_BYTES, stream, p, map));
+    PL_CUDA(launch_pdl(kernel, dim3(p.n_work * p.nkv), dim3(THREADS), (size_t)smem, stream, p, map));
     return 0;
 }
 
 // p.d must be D.
 template <int D>
 inline int launch(const AttnParams& p, cudaStream_t stream) {
+    constexpr bool wide = D == 128;
+    if (p.dist_bias != nullptr) {
+        const int G = p.nh / p.nkv;
+        const bool staged = G * bias_row_floats(G) <= Shape<D>::BIAS_FLOATS;
+        return staged ? launch_as<D, wide, 2>(p, stream) : launch_as<D, wide, 1>(p, stream);
+    }
+    if (p.keep_first > 0) return launch_as<D, wide, 1>(p, stream);
     if constexpr (D == 128) {
         static const bool narrow = getenv("PAGED_LLM_B200_TC2_NARROW") != nullptr;   // one product per value panel
-        return narrow ? launch_as<D, false>(p, stream) : launch_as<D, true>(p, stream);
+        return narrow ? launch_as<D, false, 0>(p, stream) : launch_as<D, true, 0>(p, stream);
     }
-    return launch_as<D, false>(p, stream);
+    return launch_as<D, false, 0>(p, stream);
 }
 
 }  // namespace tc2

@@ -114,6 +114,10 @@ LENS = [1, 137, 70, 2]
     (64, attention(20, 1, 16, 16, 40, (30, 2)), 8, 16),
     (64, attention(2, 1, 200, 256, 40, (30, 2)), 8, 16),
     (48, attention(4, 2, 64, 64, 40, (24, 0)), 8, 16),
+    (48, attention(8, 1, 64, 64, 70, (90, 3)), 8, 16),                        # the largest group whose biases are staged,
+    (48, attention(9, 1, 64, 64, 70, (90, 3)), 8, 16),                        # and one beyond it
+    (48, attention(3, 1, 128, 128, 70.5), 16, 16),
+    (48, attention(14, 2, 64, 64, 300), 16, 16),
 ])
 def test_attention_alone(ops, dtype, W, m, rows, ps):
     parts.check_attention(ops, "cuda", dtype, W, m, LENS, seed=3, rows=rows, ps=ps)
