@@ -356,7 +356,7 @@ struct Shape {
     static constexpr int Q_PANEL = BM * 128, K_PANEL = BN * 128;
     static constexpr int Q_BYTES = PANELS * Q_PANEL, K_BYTES = PANELS * K_PANEL;
     static constexpr int SMEM_BYTES = Q_BYTES + 2 * STAGES * K_BYTES + 1024;
-    // A learned bias by distance, staged per key tile by the warp that brings the keys: per head of the group the distances
+    // A learned bias by distance, staged per key tile by the two copy warps: per head of the group the distances
     // between the block's tokens and the tile's keys.  S(m) is only issued once the softmax is done with tile m - 2, and a
     // stage of keys is refilled once its S is done, so with STAGES + 2 slots the one being filled is never still read.
     static constexpr int BIAS_SLOTS = STAGES + 2, BIAS_FLOATS = 800;
@@ -377,6 +377,9 @@ __device__ __forceinline__ void mbar_arrive(uint64_t* bar) {
 }
 __device__ __forceinline__ void mbar_arrive_expect(uint64_t* bar, uint32_t bytes) {
     asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;\n" ::"r"(saddr(bar)), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ void cp4(uint32_t dst, const float* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(dst), "l"(src));
 }
 // One box of the tensor map at rows [row, row + box rows), columns [col, col + 64) (col a
 // multiple of 64), to shared memory; the bytes are counted on `bar`.
@@ -491,7 +494,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
             mbar_init(&pv_done[b], 1);
         }
         if (BIAS == 2)
-            for (int b = 0; b < SH::BIAS_SLOTS; ++b) mbar_init(&b_full[b], 32);
+            for (int b = 0; b < SH::BIAS_SLOTS; ++b) mbar_init(&b_full[b], 64);
         asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
     }
     // Q tile: row R = token * G + head; eight 16-byte chunks per row and panel
@@ -524,6 +527,20 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
             if (t >= n_tiles || lane >= boxes || n0 >= key_hi || (n0 + box_rows <= key_lo && (!KEEP || n0 >= kept))) return -1;
             return bt[n0 >> p.ps_shift];
         };
+        // the entries of a bias slot that this lane fills (the two warps share a slot): place in the table of the group's heads
+        // in front of the distance, and place in its row
+        constexpr int BI = (SH::BIAS_FLOATS + 63) / 64;
+        const int e_first = lane + (values ? 32 : 0);
+        const int bias_total = BIAS == 2 ? G * bias_ld : 0;
+        int head_off[BIAS == 2 ? BI : 1], in_row[BIAS == 2 ? BI : 1];
+        if (BIAS == 2) {
+#pragma unroll
+            for (int i = 0; i < BI; ++i) {
+                const int e = e_first + 64 * i, hh = e / max(bias_ld, 1);
+                in_row[i] = e - hh * bias_ld;
+                head_off[i] = hh * p.dist_len;
+            }
+        }
         int pg_next = page_of(0);
         for (int t = 0; t < n_tiles; ++t) {
             const int s = t % STAGES;
@@ -541,16 +558,23 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
                 for (int c = 0; c < PANELS; ++c)
                     tma_box(ring + s * K_BYTES + c * K_PANEL + lane * box_bytes, &kv_map, c * 64, row, &full[s]);
             }
-            if (BIAS == 2 && !values) {
-                // entry x of head hh: the bias of distance pos_first - (the tile's last key) + x, in units of the raw product
-                float* slot = bias_slots + (t % SH::BIAS_SLOTS) * SH::BIAS_FLOATS;
-                const int d0 = pos_first - tile_key(t) - (BN - 1), span = (BM + G - 1) / G + BN, far = p.dist_len - 1;
-                const float unit = 1.f / p.scale;
-                for (int hh = 0; hh < G; ++hh) {
-                    const float* src = p.dist_bias + (size_t)(kvh * G + hh) * p.dist_len;
-                    for (int x = lane; x < span; x += 32) slot[hh * bias_ld + x] = __ldg(src + min(max(d0 + x, 0), far)) * unit;
+            if (BIAS == 2) {
+                // entry x of a head: the bias of distance pos_first - (the tile's last key) + x, copied as it is; the barrier
+                // counts this lane once its copies have landed
+                const uint32_t slot = saddr(bias_slots + (t % SH::BIAS_SLOTS) * SH::BIAS_FLOATS + e_first);
+                const int d0 = pos_first - tile_key(t) - (BN - 1), far = p.dist_len - 1;
+                const float* src = p.dist_bias + (size_t)kvh * G * p.dist_len;
+                if (d0 >= 0 && d0 + bias_ld <= p.dist_len) {
+                    const float* from = src + d0;
+#pragma unroll
+                    for (int i = 0; i < BI; ++i)
+                        if (e_first + 64 * i < bias_total) cp4(slot + 256 * i, from + (head_off[i] + in_row[i]));
+                } else {
+#pragma unroll
+                    for (int i = 0; i < BI; ++i)
+                        if (e_first + 64 * i < bias_total) cp4(slot + 256 * i, src + (head_off[i] + min(max(d0 + in_row[i], 0), far)));
                 }
-                mbar_arrive(&b_full[t % SH::BIAS_SLOTS]);
+                asm volatile("cp.async.mbarrier.arrive.noinc.shared::cta.b64 [%0];\n" ::"r"(saddr(&b_full[t % SH::BIAS_SLOTS])) : "memory");
             }
         }
     } else if (warp == MMA_WARP) {
@@ -640,7 +664,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
                 mbar_wait(&b_full[b6], (t / SH::BIAS_SLOTS) & 1);
                 const float* bs = bias_slots + b6 * SH::BIAS_FLOATS + bias_at;
 #pragma unroll
-                for (int i = 0; i < 64; ++i) sv[i] += bs[-i];
+                for (int i = 0; i < 64; ++i) sv[i] = fmaf(bs[-i], bias_unit, sv[i]);
             }
             if (BIAS == 1 && bias_row != nullptr) {
                 // a learned bias by distance, brought into the units of the raw product (the scale comes below); a
