@@ -677,10 +677,12 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc2_kernel(AttnParams p, cons
             const bool row_full = ((kbase >= key_lo && kbase >= first) || (KEEP && kbase + BN <= kept)) && kbase + BN <= key_hi && kbase + BN - 1 <= pos;
             const bool warp_full = __all_sync(0xffffffffu, row_full);
             if (!warp_full) {
+                // (a row's first key lies in the window and its position in front of the range's end, so these three bounds
+                // imply the block's own range)
+                const int first_i = first - kbase, last_i = min(pos, key_hi - 1) - kbase, keep_i = p.keep_first - kbase;
 #pragma unroll
                 for (int i = 0; i < 64; ++i) {
-                    const int n = kbase + i;
-                    const bool vis = in_range(n) && n <= pos && (n >= first || (KEEP && n < p.keep_first));
+                    const bool vis = i <= last_i && (i >= first_i || (KEEP && i < keep_i));
                     sv[i] = vis ? sv[i] : -INFINITY;
                 }
             }
