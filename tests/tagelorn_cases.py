@@ -74,9 +74,9 @@ CASE_B = model(77, 92, 2, 5, [
 ], eps=1e-6, scale=0.5, cap=30.0)
 
 # C: heads of 64 and 128 (the tensor-core prefill kernels) with windows around a tile's size; one tap (no history); eight
-# query heads on two kv heads; four of twelve experts out of two of four groups.
+# query heads on two kv heads; four of sixteen experts out of two of four groups.
 CASE_C = model(300, 128, 1, 16, [
-    layer("attention", attention(8, 2, 64, 64, 128, (65, 6)), moe(64, 12, 4, 2.0, (4, 2), shared=32)),
+    layer("attention", attention(8, 2, 64, 64, 128, (65, 6)), moe(64, 16, 4, 1.8, (4, 2), shared=32)),
     layer("general_delta", delta(2, 64), dense(96)),
     layer("attention", attention(2, 1, 128, 128, 50, (100, 70)), moe(32, 8, 2, 1.0, (2, 1), shared=64)),
 ], scale=8.0, cap=20.0)

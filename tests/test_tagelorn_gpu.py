@@ -60,7 +60,7 @@ def test_sinusoids(ops, dtype, W, scale):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("W,dim,layers,which,rows", [(32, 12, 3, 1, 9), (48, 8, 1, 0, 1), (20, 5, 4, 3, 17), (1024, 64, 2, 1, 300), (256, 24, 5, 4, 16),
+@pytest.mark.parametrize("W,dim,layers,which,rows", [(32, 12, 3, 1, 9), (48, 8, 1, 0, 1), (20, 5, 4, 3, 17), (1024, 64, 2, 1, 300), (288, 40, 3, 2, 16),
                                                      (5000, 32, 2, 0, 3)])
 def test_token_input(ops, dtype, W, dim, layers, which, rows):
     """The stream takes the branch and the normed token input in, and the next norm reads the result; widths that four-element
@@ -134,7 +134,7 @@ def test_delta_rule_alone(ops, dtype, W, m, rank):
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("W,taps,inner,m", [(32, 4, "general_delta", delta(2, 8)), (24, 2, "attention", attention(2, 1, 8, 8, 40, (5, 2))),
                                             (24, 1, "attention", attention(2, 2, 8, 8, 40)), (20, 7, "general_delta", delta(1, 12)),
-                                            (27, 3, "general_delta", delta(1, 8)), (256, 3, "general_delta", delta(2, 16))])
+                                            (27, 3, "general_delta", delta(1, 8)), (288, 5, "general_delta", delta(2, 16))])
 def test_input_convolution_alone(ops, dtype, W, taps, inner, m):
     parts.check_input_convolution(ops, "cuda", dtype, W, taps, inner, m, [1, 3, 70, 33], seed=9)
 
