@@ -74,6 +74,10 @@ def _register_builtin() -> None:
     from .tagelorn import TagelornConfig
     if "Tagelorn" not in ARCHITECTURES:
         register_architecture("Tagelorn", TagelornConfig, tagelorn_spec)
+    from ..models.nopozen import nopozen_spec
+    from .nopozen import NopozenConfig
+    if "Nopozen" not in ARCHITECTURES:
+        register_architecture("Nopozen", NopozenConfig, nopozen_spec)
 
 
 _register_builtin()

@@ -35,7 +35,7 @@ HEAD_DIM_BUILDS = (16, 32, 64, 128, 256)
 
 MODULES: dict[str, list[str]] = {
     "core": ["common.cu", "elementwise.cu", "mixers.cu", "gemm_f32.cu", "gemm_skinny.cu", "gemm_tc.cu", "attention_f32.cu",
-             "sampling.cu", "token_input.cu"],
+             "sampling.cu", "token_input.cu", "branches.cu"],
     **{f"attn_bf16_d{d}": ["common.cu", f"attention_bf16_d{d}.cu"] for d in HEAD_DIM_BUILDS},
     # decode attention whose scratch is a static array of the library (see attention_decode_static.h)
     "attn_static": ["common.cu", "attention_decode_static.cu"],
@@ -47,6 +47,8 @@ MODULES: dict[str, list[str]] = {
     "streams": ["common.cu", "streams.cu"],
     # convolution with a gated recurrence per channel; gated linear attention; the delta rule
     "recurrent": ["common.cu", "recurrent.cu"],
+    # linear attention with a fixed decay per head; the norm over all heads with a gate; the convolution in front of attention
+    "lightning": ["common.cu", "lightning.cu"],
     # the generalized delta rule and the convolution added to a mixer's input
     "general_delta": ["common.cu", "general_delta.cu"],
 }

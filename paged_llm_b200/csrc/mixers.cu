@@ -357,10 +357,13 @@ PL_EXPORT int pl_normed_qkv_write(const void* proj, int dtype, int T, int ld, co
 
 // ------------------------------------------------------------------ unit root mean square per head + cache write
 // proj row: [q: nh*d | k: nkv*d | v: nkv*dv | ...], plus `bias` (float32, the same layout, may be null).  Every head of q
-// and k is divided by its own root mean square, x / sqrt(mean(x^2) + eps) over the d elements; Q out [T, nh*D], K and V to
-// the page slot, all padded to D with zeros.  A warp per (token, head): heads 0..nh-1 are queries, then keys, then values.
+// and k is divided by its own root mean square, x / sqrt(mean(x^2) + eps) over the d elements, and multiplied by a weight
+// [d] if there is one (qw, kw: one for all heads); with a table `rot`, q and k are then rotated by the token's position over
+// the table's leading elements of each head.  Q out [T, nh*D], K and V to the page slot, all padded to D with zeros.  A warp
+// per (token, head): heads 0..nh-1 are queries, then keys, then values.
 template <typename T>
 __global__ void __launch_bounds__(256) unit_qkv_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ bias, float eps,
+                                                       const float* __restrict__ qw, const float* __restrict__ kw, RotTable rot,
                                                        T* __restrict__ q_out, T* __restrict__ kv, SlotArgs sa, int nh, int nkv, int d,
                                                        int dv, int D, int write, int vec, long long items) {
     pdl_launch_dependents();
@@ -373,13 +376,15 @@ __global__ void __launch_bounds__(256) unit_qkv_kernel(const T* __restrict__ pro
     const int t = (int)(item / heads), head = (int)(item - (long long)t * heads);
     const int s = sa.token_seq[t];
     const bool is_q = head < nh, is_v = head >= nh + nkv;
-    const int n = is_v ? dv : d;
+    const int n = is_v ? dv : d, pos = sa.positions[t];
+    const float* hw = is_v ? nullptr : is_q ? qw : kw;
+    const float2* cs = !is_v && rot.table != nullptr && s >= 0 && pos >= 0 && pos < rot.len ? rot.table + (size_t)pos * (rot.rd >> 1) : nullptr;
     const int col = is_v ? (nh + nkv) * d + (head - nh - nkv) * dv : head * d;
     T* dst = nullptr;
     if (is_q) {
         dst = q_out + ((size_t)t * nh + head) * D;
     } else if (write && s >= 0) {
-        const long long slot = key_slot(sa, t, s, sa.positions[t], nkv, D);
+        const long long slot = key_slot(sa, t, s, pos, nkv, D);
         if (slot >= 0) dst = kv + slot + (size_t)(is_v ? head - nkv - nh : head - nh) * sa.ps * D + (is_v ? (size_t)nkv * sa.ps * D : 0);
     }
     pdl_wait();
@@ -387,21 +392,34 @@ __global__ void __launch_bounds__(256) unit_qkv_kernel(const T* __restrict__ pro
     const T* src = proj + (size_t)t * ld + col;
     const float* b = bias != nullptr ? bias + col : nullptr;
     if (vec) {
-        // d, dv and D are multiples of 4 up to 256: a lane holds two quads of the head
+        // d, dv and D are multiples of 4 up to 256: a lane holds two quads of the head (rotation: quads do not straddle)
         float4 v[2];
         float sq = 0.f;
+        auto biased = [&](int c) {
+            float4 x = Quad4<T>::load(src + c);
+            if (b != nullptr) {
+                const float4 w = Quad4<float>::load(b + c);
+                x = make_float4(x.x + w.x, x.y + w.y, x.z + w.z, x.w + w.w);
+            }
+            return x;
+        };
+        auto weighted = [&](float4 x, int c) {
+            if (hw == nullptr) return x;
+            const float4 w = Quad4<float>::load(hw + c);
+            return make_float4(x.x * w.x, x.y * w.y, x.z * w.z, x.w * w.w);
+        };
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
             const int c = (lane + 32 * i) * 4;
-            v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            v[i] = c < n && s >= 0 ? biased(c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            sq += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
             if (c < n && s >= 0) {
-                v[i] = Quad4<T>::load(src + c);
-                if (b != nullptr) {
-                    const float4 w = Quad4<float>::load(b + c);
-                    v[i] = make_float4(v[i].x + w.x, v[i].y + w.y, v[i].z + w.z, v[i].w + w.w);
+                v[i] = weighted(v[i], c);
+                if (cs != nullptr && c < rot.rd) {
+                    const int other = c >= (rot.rd >> 1) ? c - (rot.rd >> 1) : c + (rot.rd >> 1);
+                    v[i] = turned_quad(cs, rot.rd, c, v[i], weighted(biased(other), other));
                 }
             }
-            sq += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
         }
         const float f = is_v ? 1.f : 1.0f / sqrtf(warp_sum(sq) / (float)d + eps);
 #pragma unroll
@@ -418,10 +436,12 @@ __global__ void __launch_bounds__(256) unit_qkv_kernel(const T* __restrict__ pro
         sq = fmaf(x, x, sq);
     }
     const float f = is_v ? 1.f : 1.0f / sqrtf(warp_sum(sq) / (float)d + eps);
-    for (int c = lane; c < D; c += 32) dst[c] = from_float<T>(value(c) * f);
+    auto weighted = [&](int c) { return hw != nullptr && c < n ? value(c) * __ldg(hw + c) : value(c); };
+    for (int c = lane; c < D; c += 32) dst[c] = from_float<T>(turned(cs, rot.rd, rot.inter, 1.f, c, weighted) * f);
 }
 
-PL_EXPORT int pl_unit_qkv_write(const void* proj, int dtype, int T, int ld, const float* bias, float eps, void* q_out, void* kv,
+PL_EXPORT int pl_unit_qkv_write(const void* proj, int dtype, int T, int ld, const float* bias, float eps, const float* qw,
+                                const float* kw, const float* rot_table, int rot_len, int rot_rd, int rot_inter, void* q_out, void* kv,
                                 const int* positions, const int* token_seq, const int* block_table, int bt_stride, int num_pages,
                                 int ps, int nh, int nkv, int d, int dv, int D, int write, cudaStream_t stream) {
     if (T == 0) return 0;
@@ -430,25 +450,168 @@ PL_EXPORT int pl_unit_qkv_write(const void* proj, int dtype, int T, int ld, cons
     SlotArgs sa{positions, token_seq, block_table, bt_stride, num_pages, ps};
     const long long items = (long long)T * (nh + 2 * nkv), blocks = (items + 7) / 8;
     PL_REQUIRE(blocks < (1ll << 31), "unit_qkv_write: %d tokens", T);
+    PL_REQUIRE(rot_table == nullptr || (rot_rd > 0 && rot_rd % 2 == 0 && rot_rd <= d), "unit_qkv_write: %d rotated elements of %d", rot_rd, d);
+    const RotTable rot{(const float2*)rot_table, rot_len, rot_rd, rot_inter};
     const int vec = d % 4 == 0 && dv % 4 == 0 && D % 4 == 0 && D <= 256 && ld % 4 == 0 &&
-                    (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)kv | (uintptr_t)bias) & 15) == 0;
+                    (rot_table == nullptr || (rot_rd % 8 == 0 && !rot_inter)) &&
+                    (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)kv | (uintptr_t)bias | (uintptr_t)qw | (uintptr_t)kw |
+                      (uintptr_t)rot_table) & 15) == 0;
     if (dtype == PL_F32)
-        PL_CUDA(launch_pdl(unit_qkv_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, (const float*)proj, ld, bias, eps,
+        PL_CUDA(launch_pdl(unit_qkv_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, (const float*)proj, ld, bias, eps, qw, kw, rot,
                            (float*)q_out, (float*)kv, sa, nh, nkv, d, dv, D, write, vec, items));
     else if (dtype == PL_BF16)
         PL_CUDA(launch_pdl(unit_qkv_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(256), 0, stream, (const __nv_bfloat16*)proj, ld,
-                           bias, eps, (__nv_bfloat16*)q_out, (__nv_bfloat16*)kv, sa, nh, nkv, d, dv, D, write, vec, items));
+                           bias, eps, qw, kw, rot, (__nv_bfloat16*)q_out, (__nv_bfloat16*)kv, sa, nh, nkv, d, dv, D, write, vec, items));
     else
         return pl_fail("unit_qkv_write: unknown dtype %d", dtype);
     return 0;
 }
 
+// ------------------------------------------------------------------ short convolution + rotation + cache write
+// proj row: [q: nh*d | k: nkv*d | v: nkv*dv | ...].  Every one of these C channels goes through a causal convolution over the
+// request's tokens, y_t = sum_j cw[j] u_(t - taps + 1 + j) (cw [taps][C] float32, no bias); q and k are then rotated by the
+// token's position; Q out [T, nh*D], K and V to the page slot, all padded to D with zeros.  The request's last taps-1 inputs
+// are its state slot ([taps-1][C] float32).
+// grid: (requests, groups of heads, token chunks of QC_TOK); a warp per (head, token), `wh` of the block's eight warps side
+// by side on heads and the rest on tokens.  The block of chunk 0 is the only one that reads a head's old inputs, and it
+// alone writes the new ones, after a barrier.
+constexpr int QC_TOK = 64;
+
+template <typename T>
+__global__ void __launch_bounds__(256) conv_qkv_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ cw, int taps,
+                                                       float* __restrict__ state, long long state_stride, const int* __restrict__ cu_q,
+                                                       const int* __restrict__ slots, RotTable rot, T* __restrict__ q_out,
+                                                       T* __restrict__ kv, SlotArgs sa, int nh, int nkv, int d, int dv, int D, int write,
+                                                       int wh, int vec) {
+    pdl_launch_dependents();
+    const int s = blockIdx.x, hist = taps - 1, C = nh * d + nkv * (d + dv);
+    const int q0 = cu_q[s], nq = cu_q[s + 1] - q0, slot = hist > 0 ? slots[s] : 0;
+    const int t_lo = blockIdx.z * QC_TOK, t_hi = min(nq, t_lo + QC_TOK);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int head = blockIdx.y * wh + warp % wh, wt = 8 / wh;
+    pdl_wait();
+    if (slot < 0 || t_lo >= nq) return;
+    const bool live = head < nh + 2 * nkv, is_q = head < nh, is_v = head >= nh + nkv;
+    const int n = is_v ? dv : d, col = is_v ? (nh + nkv) * d + (head - nh - nkv) * dv : head * d;
+    float* st = hist > 0 ? state + (size_t)slot * state_stride + col : nullptr;
+    const T* in = proj + (size_t)q0 * ld + col;
+    const float* w = cw + col;
+    if (live) {
+        for (int t = t_lo + warp / wh; t < t_hi; t += wt) {
+            const int pos = sa.positions[q0 + t];
+            T* dst = nullptr;
+            if (is_q) {
+                dst = q_out + ((size_t)(q0 + t) * nh + head) * D;
+            } else if (write) {
+                const long long at = key_slot(sa, q0 + t, s, pos, nkv, D);
+                if (at >= 0) dst = kv + at + (size_t)(is_v ? head - nkv - nh : head - nh) * sa.ps * D + (is_v ? (size_t)nkv * sa.ps * D : 0);
+            }
+            const float2* cs = !is_v && rot.table != nullptr && pos >= 0 && pos < rot.len ? rot.table + (size_t)pos * (rot.rd >> 1) : nullptr;
+            if (vec) {
+                // sizes are multiples of 4 up to 256: a lane holds two quads of the head
+                float4 v[2];
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    const int c = (lane + 32 * i) * 4;
+                    v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+                    if (c < n) {
+                        for (int k = 0; k < taps; ++k) {
+                            const int src = t - hist + k;
+                            const float4 u = src >= 0 ? Quad4<T>::load(in + (size_t)src * ld + c)
+                                                      : *reinterpret_cast<const float4*>(st + (size_t)(hist + src) * C + c);
+                            const float4 f = *reinterpret_cast<const float4*>(w + (size_t)k * C + c);
+                            v[i].x = fmaf(f.x, u.x, v[i].x), v[i].y = fmaf(f.y, u.y, v[i].y);
+                            v[i].z = fmaf(f.z, u.z, v[i].z), v[i].w = fmaf(f.w, u.w, v[i].w);
+                        }
+                    }
+                }
+                if (cs != nullptr) {
+                    // a quad's partner sits in another lane (or this lane's other quad)
+                    float4 other[2];
+#pragma unroll
+                    for (int i = 0; i < 2; ++i) {
+                        const int quad = lane + 32 * i, hq = rot.rd >> 3;
+                        const int pq = quad >= 2 * hq ? quad : quad >= hq ? quad - hq : quad + hq;
+                        float4 a, b;
+                        a.x = __shfl_sync(0xffffffffu, v[0].x, pq & 31), b.x = __shfl_sync(0xffffffffu, v[1].x, pq & 31);
+                        a.y = __shfl_sync(0xffffffffu, v[0].y, pq & 31), b.y = __shfl_sync(0xffffffffu, v[1].y, pq & 31);
+                        a.z = __shfl_sync(0xffffffffu, v[0].z, pq & 31), b.z = __shfl_sync(0xffffffffu, v[1].z, pq & 31);
+                        a.w = __shfl_sync(0xffffffffu, v[0].w, pq & 31), b.w = __shfl_sync(0xffffffffu, v[1].w, pq & 31);
+                        other[i] = pq >= 32 ? b : a;
+                    }
+#pragma unroll
+                    for (int i = 0; i < 2; ++i) v[i] = turned_quad(cs, rot.rd, (lane + 32 * i) * 4, v[i], other[i]);
+                }
+                if (dst == nullptr) continue;
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    const int c = (lane + 32 * i) * 4;
+                    if (c < D) Quad4<T>::store(dst + c, v[i]);
+                }
+            } else if (dst != nullptr) {
+                auto value = [&](int c) {
+                    float a = 0.f;
+                    for (int k = 0; k < taps && c < n; ++k) {
+                        const int src = t - hist + k;
+                        a = fmaf(w[(size_t)k * C + c], src >= 0 ? to_float(in[(size_t)src * ld + c]) : st[(size_t)(hist + src) * C + c], a);
+                    }
+                    return a;
+                };
+                for (int c = lane; c < D; c += 32) dst[c] = from_float<T>(turned(cs, rot.rd, rot.inter, 1.f, c, value));
+            }
+        }
+    }
+    if (blockIdx.z != 0 || hist == 0) return;
+    __syncthreads();                                                    // every read of the old inputs is done
+    if (live && warp / wh == 0) {
+        // the last taps-1 inputs of [old inputs ; this step's inputs]: in place from the front, since entry j reads old
+        // entry j + nq > j or a new input
+        for (int c = lane; c < n; c += 32)
+            for (int j = 0; j < hist; ++j) {
+                const int src = nq + j - hist;
+                st[(size_t)j * C + c] = src >= 0 ? to_float(in[(size_t)src * ld + c]) : st[(size_t)(j + nq) * C + c];
+            }
+    }
+}
+
+// `max_tokens`: no request of the step brings more.  state null: one tap, nothing to keep.
+PL_EXPORT int pl_conv_qkv_write(const void* proj, int dtype, int ld, const float* cw, int taps, float* state, long long state_stride,
+                                const int* cu_q, const int* slots, int num_seqs, int max_tokens, const float* rot_table, int rot_len,
+                                int rot_rd, int rot_inter, void* q_out, void* kv, const int* positions, const int* token_seq,
+                                const int* block_table, int bt_stride, int num_pages, int ps, int nh, int nkv, int d, int dv, int D,
+                                int write, cudaStream_t stream) {
+    if (num_seqs == 0) return 0;
+    const int C = nh * d + nkv * (d + dv);
+    PL_REQUIRE(nh > 0 && nkv > 0 && d > 0 && dv > 0 && D >= d && D >= dv && ps > 0 && ld >= C && max_tokens >= 1,
+               "conv_qkv_write: bad sizes d=%d dv=%d D=%d ld=%d", d, dv, D, ld);
+    PL_REQUIRE(taps >= 1 && taps <= QC_TOK && (taps == 1 || (state != nullptr && state_stride >= (long long)(taps - 1) * C)),
+               "conv_qkv_write: %d taps (at most %d), a state of %lld floats", taps, QC_TOK, state_stride);
+    PL_REQUIRE(rot_table == nullptr || (rot_rd > 0 && rot_rd % 2 == 0 && rot_rd <= d), "conv_qkv_write: %d rotated elements of %d", rot_rd, d);
+    const SlotArgs sa{positions, token_seq, block_table, bt_stride, num_pages, ps};
+    const RotTable rot{(const float2*)rot_table, rot_len, rot_rd, rot_inter};
+    const int vec = d % 4 == 0 && dv % 4 == 0 && D % 4 == 0 && D <= 256 && ld % 4 == 0 && state_stride % 4 == 0 &&
+                    (rot_table == nullptr || (rot_rd % 8 == 0 && !rot_inter)) &&
+                    (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)kv | (uintptr_t)cw | (uintptr_t)state | (uintptr_t)rot_table) & 15) == 0;
+    const int wh = max_tokens >= 8 ? 1 : max_tokens >= 4 ? 2 : max_tokens >= 2 ? 4 : 8;
+    const dim3 grid(num_seqs, (nh + 2 * nkv + wh - 1) / wh, (max_tokens + QC_TOK - 1) / QC_TOK);
+    PL_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "conv_qkv_write: %d tokens, %d heads in a step", max_tokens, nh);
+    if (dtype == PL_F32)
+        PL_CUDA(launch_pdl(conv_qkv_kernel<float>, grid, dim3(256), 0, stream, (const float*)proj, ld, cw, taps, state, state_stride, cu_q,
+                           slots, rot, (float*)q_out, (float*)kv, sa, nh, nkv, d, dv, D, write, wh, vec));
+    else if (dtype == PL_BF16)
+        PL_CUDA(launch_pdl(conv_qkv_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)proj, ld, cw, taps, state,
+                           state_stride, cu_q, slots, rot, (__nv_bfloat16*)q_out, (__nv_bfloat16*)kv, sa, nh, nkv, d, dv, D, write, wh, vec));
+    else
+        return pl_fail("conv_qkv_write: unknown dtype %d", dtype);
+    return 0;
+}
+
 // ------------------------------------------------------------------ sigmoid gate on the heads' outputs
 // out[t, h*dv + c] = o[t, h*D + c] * sigmoid(gate[t, h*dv + c]),  c < dv (the padding of a head is dropped).
-// gate null: the copy without the padding.
+// gate null: the copy without the padding.  `per_head`: one number per head, gate[t, h], for all its elements.
 template <typename T>
 __global__ void head_gate_kernel(const T* __restrict__ o, int D, const T* __restrict__ gate, int ldg, T* __restrict__ out,
-                                 long long n, int nh, int dv) {
+                                 long long n, int nh, int dv, int per_head) {
     pdl_launch_dependents();
     pdl_wait();
     const int row = nh * dv;
@@ -456,7 +619,7 @@ __global__ void head_gate_kernel(const T* __restrict__ o, int D, const T* __rest
         const long long t = i / row;
         const int e = (int)(i - t * row), h = e / dv, c = e - h * dv;
         float v = to_float(o[(size_t)t * nh * D + h * D + c]);
-        if (gate != nullptr) v *= 1.0f / (1.0f + expf(-to_float(gate[(size_t)t * ldg + e])));
+        if (gate != nullptr) v *= 1.0f / (1.0f + expf(-to_float(gate[(size_t)t * ldg + (per_head ? h : e)])));
         out[i] = from_float<T>(v);
     }
 }
@@ -464,7 +627,7 @@ __global__ void head_gate_kernel(const T* __restrict__ o, int D, const T* __rest
 // The same, four elements per thread: grid (quads of a row / 256, row groups).
 template <typename T>
 __global__ void __launch_bounds__(256) head_gate4_kernel(const T* __restrict__ o, int D, const T* __restrict__ gate, int ldg,
-                                                         T* __restrict__ out, int rows, int nh, int dv) {
+                                                         T* __restrict__ out, int rows, int nh, int dv, int per_head) {
     pdl_launch_dependents();
     pdl_wait();
     const int e = (blockIdx.x * 256 + threadIdx.x) * 4;
@@ -473,7 +636,9 @@ __global__ void __launch_bounds__(256) head_gate4_kernel(const T* __restrict__ o
     for (int t = blockIdx.y; t < rows; t += gridDim.y) {
         float4 v = Quad4<T>::load(o + (size_t)t * nh * D + h * D + c);
         if (gate != nullptr) {
-            const float4 g = Quad4<T>::load(gate + (size_t)t * ldg + e);
+            float4 g;
+            if (per_head) g.x = g.y = g.z = g.w = to_float(gate[(size_t)t * ldg + h]);
+            else g = Quad4<T>::load(gate + (size_t)t * ldg + e);
             v = make_float4(v.x / (1.0f + expf(-g.x)), v.y / (1.0f + expf(-g.y)), v.z / (1.0f + expf(-g.z)),
                             v.w / (1.0f + expf(-g.w)));
         }
@@ -482,26 +647,27 @@ __global__ void __launch_bounds__(256) head_gate4_kernel(const T* __restrict__ o
 }
 
 template <typename T>
-static int launch_head_gate(const void* o, int T_, int D, const void* gate, int ldg, void* out, int nh, int dv,
+static int launch_head_gate(const void* o, int T_, int D, const void* gate, int ldg, void* out, int nh, int dv, int per_head,
                             cudaStream_t stream) {
-    if (dv % 4 == 0 && D % 4 == 0 && ldg % 4 == 0 && (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)out) & 15) == 0) {
+    const bool gate_ok = per_head || (ldg % 4 == 0 && ((uintptr_t)gate & 15) == 0);
+    if (dv % 4 == 0 && D % 4 == 0 && gate_ok && (((uintptr_t)o | (uintptr_t)out) & 15) == 0) {
         const dim3 grid((nh * dv / 4 + 255) / 256, T_ < 65535 ? T_ : 65535);
-        PL_CUDA(launch_pdl(head_gate4_kernel<T>, grid, dim3(256), 0, stream, (const T*)o, D, (const T*)gate, ldg, (T*)out, T_, nh, dv));
+        PL_CUDA(launch_pdl(head_gate4_kernel<T>, grid, dim3(256), 0, stream, (const T*)o, D, (const T*)gate, ldg, (T*)out, T_, nh, dv, per_head));
         return 0;
     }
     const long long n = (long long)T_ * nh * dv;
     const long long blocks = (n + 255) / 256;
     PL_CUDA(launch_pdl(head_gate_kernel<T>, dim3((unsigned)(blocks < 4096 ? blocks : 4096)), dim3(256), 0, stream, (const T*)o, D,
-                       (const T*)gate, ldg, (T*)out, n, nh, dv));
+                       (const T*)gate, ldg, (T*)out, n, nh, dv, per_head));
     return 0;
 }
 
 PL_EXPORT int pl_head_gate(const void* o, int dtype, int T, int D, const void* gate, int ldg, void* out, int nh, int dv,
-                           cudaStream_t stream) {
+                           int per_head, cudaStream_t stream) {
     if (T == 0) return 0;
     PL_REQUIRE(nh > 0 && dv > 0 && D >= dv, "head_gate: bad sizes dv=%d D=%d", dv, D);
-    if (dtype == PL_F32) return launch_head_gate<float>(o, T, D, gate, ldg, out, nh, dv, stream);
-    if (dtype == PL_BF16) return launch_head_gate<__nv_bfloat16>(o, T, D, gate, ldg, out, nh, dv, stream);
+    if (dtype == PL_F32) return launch_head_gate<float>(o, T, D, gate, ldg, out, nh, dv, per_head, stream);
+    if (dtype == PL_BF16) return launch_head_gate<__nv_bfloat16>(o, T, D, gate, ldg, out, nh, dv, per_head, stream);
     return pl_fail("head_gate: unknown dtype %d", dtype);
 }
 

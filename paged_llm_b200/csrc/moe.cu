@@ -23,10 +23,10 @@ __device__ __forceinline__ float act_mul_f(int act, float limit, float g, float 
 
 // ------------------------------------------------------------------ the router's choice
 // The logits z[t][0..E) (and, if `shared_gate`, z[t][E], whose sigmoid is the token's factor for the shared
-// expert) come from a product of the kernel library in float32.  One warp per token picks the k largest, one
+// expert) come from a product of the kernel library in float32; `bias` [E] (or null) is added to them.  One warp per token picks the k largest, one
 // after the other (among equals the lowest index), and forms the softmax over the chosen.
 __global__ void __launch_bounds__(128) moe_topk_kernel(const float* __restrict__ z_all, int ldz, int tokens, int E, int k,
-                                                       int shared_gate, int* __restrict__ top_idx,
+                                                       int shared_gate, const float* __restrict__ bias, int* __restrict__ top_idx,
                                                        float* __restrict__ top_w, float* __restrict__ gate) {
     extern __shared__ float z_smem[];                   // [4][E]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -34,7 +34,7 @@ __global__ void __launch_bounds__(128) moe_topk_kernel(const float* __restrict__
     if (t >= tokens) return;
     float* z = z_smem + warp * E;
     const float* src = z_all + (size_t)t * ldz;
-    for (int e = lane; e < E; e += 32) z[e] = src[e];
+    for (int e = lane; e < E; e += 32) z[e] = bias != nullptr ? src[e] + __ldg(bias + e) : src[e];
     if (shared_gate && lane == 0) gate[t] = 1.0f / (1.0f + expf(-src[E]));
     __syncwarp();
     float chosen_z = 0.f, z_max = 0.f;
@@ -524,13 +524,14 @@ int launch_moe_bf16(const MoeGemm& p, int max_tiles, cudaStream_t stream) {
 
 }  // namespace
 
-PL_EXPORT int pl_moe_topk(const float* z, int ldz, int tokens, int E, int k, int shared_gate, int* top_idx, float* top_w,
-                          float* gate, cudaStream_t stream) {
+// bias: [E] float32 on the logits, or null.
+PL_EXPORT int pl_moe_topk(const float* z, int ldz, int tokens, int E, int k, int shared_gate, const float* bias, int* top_idx,
+                          float* top_w, float* gate, cudaStream_t stream) {
     if (tokens == 0) return 0;
     PL_REQUIRE(tokens > 0 && E > 0 && k > 0 && k <= E && k <= 32 && E <= 1024 && ldz >= E + (shared_gate ? 1 : 0),
                "moe_topk: tokens=%d experts=%d top=%d (top <= 32, experts <= 1024)", tokens, E, k);
-    moe_topk_kernel<<<(tokens + 3) / 4, 128, (size_t)4 * E * sizeof(float), stream>>>(z, ldz, tokens, E, k, shared_gate, top_idx,
-                                                                                   top_w, gate);
+    moe_topk_kernel<<<(tokens + 3) / 4, 128, (size_t)4 * E * sizeof(float), stream>>>(z, ldz, tokens, E, k, shared_gate, bias,
+                                                                                   top_idx, top_w, gate);
     PL_LAUNCHED("moe_topk");
     return 0;
 }

@@ -19,6 +19,7 @@ import numpy as np
 import torch
 
 from ..csrc import build
+from ..parts.base import LazyExperts, LazyLinear, LazySum
 from . import plan as planning
 from .errors import KernelError
 
@@ -260,7 +261,14 @@ class CudaOps:
         return logits
 
     def add_copy(self, x: torch.Tensor, branch=None) -> torch.Tensor:
-        """x += branch in place (float32 stream; the branch may be None); returns x in the compute dtype."""
+        """x += branch in place (float32 stream; the branch may be None or lazy); returns x in the compute dtype."""
+        if isinstance(branch, (LazySum, LazyExperts)):
+            parts = list(branch.parts) if isinstance(branch, LazySum) else [branch]
+            copy = torch.empty(x.shape, dtype=self.compute_dtype, device=self.device) if self.compute_dtype != torch.float32 else None
+            self._branch_norm(x, parts, None, 0.0, copy)
+            return x if copy is None else copy
+        if hasattr(branch, "materialize"):
+            branch = branch.materialize(self)
         if self.compute_dtype == torch.float32:
             return self.add_rows(x, branch)
         assert x.dtype == torch.float32 and x.is_contiguous()
@@ -271,12 +279,14 @@ class CudaOps:
         self.launches += 1
         return copy
 
+    def stream_copy(self, x: torch.Tensor) -> torch.Tensor:
+        """x (float32 stream) in the compute dtype (x itself where that is float32)."""
+        return self.add_copy(x, None)
+
     def token_side_gate(self, x: torch.Tensor, branch, w_gate: torch.Tensor, table: torch.Tensor, offset: int, dim: int,
                         ids: torch.Tensor) -> torch.Tensor:
         """x += branch (in place; a tensor or a lazy branch), then gelu_tanh(x @ w_gate^T) * table[ids, offset : offset + dim].
         `w_gate` may have rows beyond `dim`; the result's columns there are zero."""
-        if hasattr(branch, "materialize"):
-            branch = branch.materialize(self)
         z = self.linear(self.add_copy(x, branch), w_gate)
         T, n = z.shape
         assert z.is_contiguous() and table.dtype == z.dtype and table.is_contiguous() and dim <= n
@@ -326,6 +336,48 @@ class CudaOps:
                                                self._p(y), self._code(y), rows, H, c_float(eps), self._stream))
         self.launches += 1
         return y
+
+    # ---- sums of branches --------------------------------------------------------
+    def branches_add_rms_norm(self, x: torch.Tensor, parts: list, w: torch.Tensor, eps: float) -> torch.Tensor:
+        """x += the sum of the branches (float32 stream, in place), then RMSNorm(x) * w in the compute dtype: one kernel behind
+        the branches' own products.  A branch is a tensor, a `LazyLinear` (its bias joins here) or a `LazyExperts`."""
+        y = torch.empty(x.shape, dtype=self.compute_dtype, device=self.device)
+        self._branch_norm(x, parts, w, eps, y)
+        return y
+
+    def branch_sum(self, parts: list) -> torch.Tensor:
+        """The sum of one or two branches as float32."""
+        first = parts[0]
+        rows = first.count if isinstance(first, LazyExperts) else (first.input if isinstance(first, LazyLinear) else first).shape[0]
+        width = first.rows_.shape[1] if isinstance(first, LazyExperts) else first.weight.shape[0] if isinstance(first, LazyLinear) else first.shape[1]
+        y = torch.empty((rows, width), dtype=torch.float32, device=self.device)
+        self._branch_norm(None, parts, None, 0.0, y)
+        return y
+
+    def _branch_norm(self, x, parts: list, w, eps: float, y) -> None:
+        shape = x.shape if x is not None else y.shape
+        rows, W = shape
+        assert 1 <= len(parts) <= 2 and (x is None or (x.dtype == torch.float32 and x.is_contiguous()))
+        args, keep = [], []
+        for b in list(parts) + [None] * (2 - len(parts)):
+            if b is None:
+                args += [c_void_p(0), 0, c_void_p(0), 0, c_void_p(0), c_void_p(0), c_void_p(0)]
+                continue
+            if isinstance(b, LazyExperts):
+                assert b.count == rows and b.rows_.shape[1] == W and b.rows_.is_contiguous()
+                args += [self._p(b.rows_), self._code(b.rows_), c_void_p(0), b.top, self._p(b.place), self._p(b.weights), self._p(b.tokens)]
+                continue
+            bias = None
+            if isinstance(b, LazyLinear):
+                b, bias = self.linear(b.input, b.weight, out_float32=b.float32), b.bias
+            elif hasattr(b, "materialize"):
+                b = b.materialize(self)
+            assert b.shape == shape and b.is_contiguous() and (bias is None or (bias.dtype == torch.float32 and bias.numel() == W))
+            keep.append(b)
+            args += [self._p(b), self._code(b), self._p(bias), 0, c_void_p(0), c_void_p(0), c_void_p(0)]
+        _check(self.core, self.core.pl_branch_norm(self._p(x), *args, self._p(w), self._code(w) if w is not None else PL_F32, self._p(y),
+                                                   self._code(y) if y is not None else PL_F32, c_longlong(rows), W, c_float(eps), self._stream))
+        self.launches += 1
 
     def dyt(self, x: torch.Tensor | None, branch: torch.Tensor | None, post, pre, out_dtype=None):
         """Dynamic tanh around the residual sum, one kernel: x += post(branch) in place (x the float32 stream),
@@ -454,7 +506,7 @@ class CudaOps:
         self.launches += 1
         return out
 
-    def linear_add_rms_norm(self, h, w, x, norm_w, eps):
+    def linear_add_rms_norm(self, h, w, x, norm_w, eps, out_float32: bool = False):
         """x += h @ w^T (float32 stream, in place), then RMSNorm(x) * norm_w.  With few tokens
         the product's epilogue adds and the result is a `LazyNorm` that the next product
         forms while loading; else the product is followed by the fused sum+norm kernel."""
@@ -473,7 +525,7 @@ class CudaOps:
                 and x.is_contiguous() and N % 4 == 0):
             self._gemm_tc(h, w, None, x, N, 3)
             return self.rms_norm(x, norm_w, eps)
-        return self.add_rms_norm(x, self.linear(h, w), norm_w, eps)
+        return self.add_rms_norm(x, self.linear(h, w, out_float32=out_float32), norm_w, eps)
 
     def gated_silu_linear(self, h, w_gate_up: torch.Tensor) -> torch.Tensor:
         return self.gated_act_linear(h, w_gate_up, "silu")
@@ -573,33 +625,64 @@ class CudaOps:
         self.launches += 1
         return q
 
-    def unit_qkv_write(self, proj, bias, nh, nkv, d, dv, D, eps, ctx, kv, block_table, write=True) -> torch.Tensor:
+    def unit_qkv_write(self, proj, bias, nh, nkv, d, dv, D, eps, ctx, kv, block_table, write=True, position=None, q_weight=None,
+                       k_weight=None) -> torch.Tensor:
         """proj rows [q: nh*d | k: nkv*d | v: nkv*dv | ...] (+ `bias`, float32, the same layout): every head of q and k is
-        divided by its own root mean square; returns the queries [T, nh*D] (heads padded to D with zeros) and writes keys and
-        values, padded the same way, to their page slots."""
+        divided by its own root mean square, multiplied by `q_weight` / `k_weight` (float32 [d], one for all heads) if they are
+        given and rotated by the token's position with `position` if that is; returns the queries [T, nh*D] (heads padded to D
+        with zeros) and writes keys and values, padded the same way, to their page slots."""
         T, ld = proj.shape
         assert proj.is_contiguous() and kv.is_contiguous() and kv.dtype == proj.dtype and kv.shape[4] == D
         assert bias is None or (bias.dtype == torch.float32 and bias.numel() == nh * d + nkv * (d + dv))
         q = torch.empty((T, nh * D), dtype=proj.dtype, device=self.device)
+        for t in (q_weight, k_weight):
+            assert t is None or (t.dtype == torch.float32 and t.numel() == d and t.is_contiguous())
         _check(self.core, self.core.pl_unit_qkv_write(
-            self._p(proj), self._code(proj), T, ld, self._p(bias), c_float(eps), self._p(q), self._p(kv), self._p(ctx.positions),
-            self._p(ctx.token_seq), self._p(block_table), block_table.shape[1], kv.shape[0], kv.shape[3], nh, nkv, d, dv, D,
+            self._p(proj), self._code(proj), T, ld, self._p(bias), c_float(eps), self._p(q_weight), self._p(k_weight),
+            *self._rot_args(position), self._p(q), self._p(kv), self._p(ctx.positions), self._p(ctx.token_seq), self._p(block_table), block_table.shape[1], kv.shape[0], kv.shape[3], nh, nkv, d, dv, D,
             1 if write else 0, self._stream))
         self.launches += 1
         return q
 
+    def conv_qkv_write(self, proj, conv_w, nh, nkv, d, dv, D, position, state, ctx, kv, block_table, write=True) -> torch.Tensor:
+        """proj rows [q: nh*d | k: nkv*d | v: nkv*dv | ...]: each of these C channels convolved over the request's tokens,
+        y_t = sum_j conv_w[j] * u_(t - taps + 1 + j) (`conv_w` float32 [taps, C]); q and k are then rotated with `position`; returns
+        the queries [T, nh*D] (heads padded to D with zeros) and writes keys and values, padded the same way, to their page slots.
+        The request's last taps-1 inputs are its state slot ([taps-1][C] float32) and are replaced by the new ones (state None:
+        one tap, nothing to keep)."""
+        T, ld = proj.shape
+        taps, C = conv_w.shape
+        assert proj.is_contiguous() and kv.is_contiguous() and kv.dtype == proj.dtype and kv.shape[4] == D
+        assert conv_w.dtype == torch.float32 and conv_w.is_contiguous() and C == nh * d + nkv * (d + dv)
+        assert state is None or (state.dtype == torch.float32 and state.is_contiguous() and state.dim() == 2)
+        q = torch.empty((T, nh * D), dtype=proj.dtype, device=self.device)
+        _check(self.core, self.core.pl_conv_qkv_write(
+            self._p(proj), self._code(proj), ld, self._p(conv_w), taps, self._p(state), c_longlong(state.shape[1] if state is not None else 0),
+            self._p(ctx.cu_seqlens_q), self._p(ctx.state_slots), ctx.num_seqs, self._longest(ctx, T), *self._rot_args(position),
+            self._p(q), self._p(kv), self._p(ctx.positions), self._p(ctx.token_seq), self._p(block_table), block_table.shape[1],
+            kv.shape[0], kv.shape[3], nh, nkv, d, dv, D, 1 if write else 0, self._stream))
+        self.launches += 1
+        return q
+
+    @staticmethod
+    def _longest(ctx, T: int) -> int:
+        """The most tokens a request of the step may bring.  A graph of mixed items replays steps of other portions than it was
+        captured with: any of them may have all the tokens."""
+        return max(T if getattr(ctx, "padded", False) else int(ctx.max_q_len), 1)
+
     def head_gate(self, o, nh, D, dv, gate=None) -> torch.Tensor:
         """[T, nh*dv]: the first dv columns of each head of o [T, nh*D], times sigmoid(gate) if a gate
-        (a column view [T, nh*dv] of a row-major tensor) is given."""
+        (a column view of a row-major tensor, [T, nh*dv] or, one number per head, [T, nh]) is given."""
         T = o.shape[0]
         assert o.is_contiguous() and o.shape[1] == nh * D
         out = torch.empty((T, nh * dv), dtype=o.dtype, device=self.device)
         ldg = 0
+        per_head = gate is not None and gate.shape[1] == nh
         if gate is not None:
-            assert gate.dtype == o.dtype and gate.stride(1) == 1 and gate.shape == (T, nh * dv)
+            assert gate.dtype == o.dtype and gate.stride(1) == 1 and gate.shape == (T, nh if per_head else nh * dv)
             ldg = gate.stride(0)
         _check(self.core, self.core.pl_head_gate(self._p(o), self._code(o), T, D, self._p(gate), ldg, self._p(out), nh, dv,
-                                                 self._stream))
+                                                 1 if per_head else 0, self._stream))
         self.launches += 1
         return out
 
@@ -825,8 +908,7 @@ class CudaOps:
         assert h.is_contiguous() and conv_w.dtype == torch.float32 and conv_w.is_contiguous() and conv_w.shape[1] == C
         assert state is None or (state.dtype == torch.float32 and state.is_contiguous() and state.dim() == 2)
         out = torch.empty_like(h)
-        # (a graph of mixed items replays steps of other portions than it was captured with)
-        longest = max(T if getattr(ctx, "padded", False) else int(ctx.max_q_len), 1)
+        longest = self._longest(ctx, T)
         _check(lib, lib.pl_residual_conv(self._p(h), self._code(h), C, self._p(conv_w), taps, self._p(state),
                                          c_longlong(state.shape[1] if state is not None else 0), self._p(ctx.cu_seqlens_q),
                                          self._p(ctx.state_slots), ctx.num_seqs, longest, self._p(out), self._stream))
@@ -957,7 +1039,7 @@ class CudaOps:
         assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] == H * dv * d
         o = torch.empty((T, H * dv), dtype=torch.float32, device=self.device)
         # a long prompt is cut into segments that run side by side: each leaves its end state and the product of its decays
-        seg, longest = lib.pl_gla_segment(), max(int(ctx.max_q_len), 1)
+        seg, longest = lib.pl_gla_segment(), self._longest(ctx, T)
         cut = longest >= 2 * seg
         seg_state = seg_decay = None
         if cut:
@@ -969,6 +1051,46 @@ class CudaOps:
                                     self._p(seg_decay), self._p(o), self._stream))
         self.launches += 3 if cut else 1
         return o
+
+    LIGHTNING_STEP_TOKENS = 8            # requests that bring no more than this run token by token in one kernel
+
+    def fixed_decay_attention(self, proj, H, d, dv, decay, state, ctx) -> torch.Tensor:
+        """Linear attention with a fixed decay per head.  proj rows [q: H*d | k: H*d | v: H*dv | ...], each through silu;
+        S_t = decay[h] S_(t-1) + k_t v_t^T, o_t = S_t^T q_t (`decay` float32 [H]).  state: [slots, H*dv*d] float32 (a head's columns
+        one after the other), updated in place.  Returns o float32 [T, H*dv].  A step of few tokens per request, and float32, run
+        token by token in one kernel; longer portions in chunks on the tensor cores: what every chunk adds to the state, the
+        states at the chunks' starts, the outputs."""
+        lib = load_module("lightning")
+        T, ld = proj.shape
+        assert proj.is_contiguous() and decay.dtype == torch.float32 and decay.numel() == H
+        assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] == H * dv * d
+        o = torch.empty((T, H * dv), dtype=torch.float32, device=self.device)
+        if proj.dtype == torch.float32 or self._longest(ctx, T) <= self.LIGHTNING_STEP_TOKENS:
+            _check(lib, lib.pl_lightning_step(self._p(proj), self._code(proj), ld, H, d, dv, self._p(decay), self._p(state),
+                                              c_longlong(state.shape[1]), self._p(ctx.cu_seqlens_q), self._p(ctx.state_slots),
+                                              ctx.num_seqs, self._p(o), self._stream))
+            self.launches += 1
+            return o
+        numbers = T // lib.pl_lightning_chunk() + ctx.num_seqs
+        buf = torch.empty(numbers * H * dv * (-(-d // 16) * 16), dtype=torch.float32, device=self.device)
+        _check(lib, lib.pl_lightning_chunks(self._p(proj), ld, H, d, dv, self._p(decay), self._p(buf), numbers, self._p(state),
+                                            c_longlong(state.shape[1]), self._p(ctx.cu_seqlens_q), self._p(ctx.state_slots), ctx.num_seqs,
+                                            self._p(o), self._stream))
+        self.launches += 3
+        return o
+
+    def row_norm_gate(self, o, proj, g_col0, norm_w, eps) -> torch.Tensor:
+        """Rows of o (float32 [T, W]) divided by their root mean square, times `norm_w`, times sigmoid(proj[:, g_col0 : g_col0 + W]);
+        in the compute dtype."""
+        lib = load_module("lightning")
+        T, W = o.shape
+        assert o.is_contiguous() and proj.is_contiguous() and norm_w.dtype == torch.float32 and norm_w.numel() == W
+        out = torch.empty((T, W), dtype=proj.dtype, device=self.device)
+        g = c_void_p(proj.data_ptr() + g_col0 * proj.element_size())
+        _check(lib, lib.pl_row_norm_gate(self._p(o), g, self._code(proj), proj.shape[1], self._p(norm_w), c_float(eps), self._p(out),
+                                         c_longlong(T), W, self._stream))
+        self.launches += 1
+        return out
 
     def head_norm_gate(self, o, proj, g_col0, H, dv, norm_w, eps, gate="silu") -> torch.Tensor:
         """Each head of o (float32 [T, H*dv]) divided by its root mean square over dv, times `norm_w` ([dv] for all heads
@@ -989,8 +1111,9 @@ class CudaOps:
     def routed_experts(self, h, w_router, w_gate_up, w_down, top_k: int, activation: str = "silu", shared=None,
                        shared_activation: str = "silu", activation_limit: float = 0.0, scoring: str = "softmax_top",
                        groups=None, gated: bool = True, shared_gate: bool = True, correction=None, renorm: bool = False,
-                       weight_scale: float = 1.0) -> torch.Tensor:
-        """The feed-forward of routed experts for the step's tokens: float32 [T, D].
+                       weight_scale: float = 1.0, router_bias=None, defer_sum: bool = False):
+        """The feed-forward of routed experts for the step's tokens: float32 [T, D] (with `defer_sum` a `LazyExperts`: the
+        weighted sum is left to whoever consumes it).  `router_bias` (float32 [E]): added to the logits.
 
         w_router [E (+1) or more, D]: the router's rows and, with a shared expert, the row of its gate (further rows
         are ignored); w_gate_up
@@ -1032,7 +1155,8 @@ class CudaOps:
                                                self._p(correction), count, keep, best, 1 if renorm else 0, c_float(weight_scale),
                                                self._p(top_idx), self._p(top_w), self._stream))
         else:
-            _check(lib, lib.pl_moe_topk(self._p(z), z.shape[1], T, E, top_k, 1 if gate_row else 0,
+            assert router_bias is None or (router_bias.dtype == torch.float32 and router_bias.numel() == E)
+            _check(lib, lib.pl_moe_topk(self._p(z), z.shape[1], T, E, top_k, 1 if gate_row else 0, self._p(router_bias),
                                         self._p(top_idx), self._p(top_w), self._p(gate), self._stream))
         tensor_cores = h.dtype == torch.bfloat16 and D % 8 == 0 and F % 8 == 0
         # Many pairs per expert (prompt portions): the experts' products run on the tcgen05 kernel of the dense
@@ -1072,6 +1196,9 @@ class CudaOps:
                                         self._p(tile_expert), self._p(n_tiles), self._p(top_w), pairs, D, F, 0, act, lim, code, BM,
                                         max_tiles, 1 if tensor_cores else 0, self._stream))
             self.launches += 4
+        if defer_sum:
+            assert shared is None
+            return LazyExperts(pair_out, top_k, place, top_w if grouped_tc else None, T)
         s = None
         if shared is not None:
             inner = self.gated_act_linear(h, shared[0], shared_activation) if gated else self.relu2_linear(h, shared[0])

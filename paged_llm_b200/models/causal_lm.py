@@ -12,7 +12,7 @@ from dataclasses import dataclass
 
 import torch
 
-from ..parts.base import (BLOCKS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS, NORMS, POSITION_ENCODINGS, FixedState,
+from ..parts.base import (BLOCKS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS, NORMS, POSITION_ENCODINGS, STREAM_JOINS, FixedState,
                           LazyLinear, ModelSpec, PagedKV, PartSpec, TensorSpec, cache_leaves, make_part, materialize)
 
 
@@ -64,10 +64,13 @@ class CausalLM:
             self.blocks.append(block_cls(mixer, ffn, norms, **block_args))
         self.final_norm = make_part(NORMS, "norm", spec.final_norm)
         self.head = make_part(HEADS, "head", spec.head)
+        self.stream_join = make_part(STREAM_JOINS, "stream join", spec.stream_join) if spec.stream_join is not None else None
         self.schedule = list(spec.schedule)
         for i, entry in enumerate(self.schedule):
             if not 0 <= entry.layer < len(self.blocks):
                 raise ValueError(f"schedule entry {i} names layer {entry.layer}, there are {len(self.blocks)}")
+            if entry.join_embedding and self.stream_join is None:
+                raise ValueError(f"schedule entry {i} joins the embedding's output, but the model has no stream join")
             if entry.cache_from is not None:
                 if not 0 <= entry.cache_from < i or self.schedule[entry.cache_from].cache_from is not None:
                     raise ValueError(f"schedule entry {i}: cache_from must name an earlier entry that owns a cache")
@@ -79,7 +82,8 @@ class CausalLM:
 
     # ---- weights ---------------------------------------------------------------
     def _parts(self):
-        return [self.embedding, *self.blocks, self.final_norm, self.head, *self.positions.values()]
+        join = [self.stream_join] if self.stream_join is not None else []
+        return [self.embedding, *self.blocks, self.final_norm, self.head, *self.positions.values(), *join]
 
     def tensor_specs(self) -> dict[str, TensorSpec]:
         out: dict[str, TensorSpec] = {}
@@ -107,6 +111,8 @@ class CausalLM:
         """Bytes of weights a decode step reads: every scheduled run reads its
         layer's matrices once, plus the head (the embedding is a gather)."""
         total = sum(self.blocks[e.layer].bytes_read_per_step() for e in self.schedule)
+        if self.stream_join is not None:
+            total += self.stream_join.bytes_read_per_step() * sum(e.join_embedding for e in self.schedule)
         return total + self.final_norm.bytes_read_per_step() + self.head.bytes_read_per_step()
 
     # ---- cache needs -----------------------------------------------------------
@@ -127,7 +133,11 @@ class CausalLM:
         pending = None
         # the stream is summed up in place, so a model that adds the embedding's output again keeps a copy
         again = x.clone() if any(e.add_embedding for e in self.schedule) else None
+        joins = sum(e.join_embedding for e in self.schedule)
+        shared = self.stream_join.start(x, joins, ctx) if joins else None
         for i, entry in enumerate(self.schedule):
+            if entry.join_embedding:
+                x, pending = self.stream_join.forward(x, pending, shared, ctx)
             if entry.add_embedding:
                 x = ctx.ops.add_rows(x, materialize(pending, ctx.ops), again)
                 pending = None

@@ -120,6 +120,11 @@ def pad16(n: int) -> int:
     return -(-n // 16) * 16
 
 
+def padded_rows(w: torch.Tensor, multiple: int) -> torch.Tensor:
+    """`w` with rows of zeros behind it up to a multiple: the product's rows then start aligned."""
+    return torch.nn.functional.pad(w, (0, 0, 0, -w.shape[0] % multiple)).contiguous()
+
+
 MAX_HEAD_DIM = 256      # the largest build of the attention kernels
 
 
@@ -142,7 +147,10 @@ class GatedAttention(Mixer):
     neither scaled nor masked and counts once; `head_norm`: in place of the norm over whole projections every head of q
     and k is divided by its own root mean square, without a weight; `bias`: q, k and v have biases (tensors
     `q_proj_bias`, ...); `keep_first` k: beside a window every query sees the request's first k tokens too, at their
-    true distances, and the cache keeps their pages.
+    true distances, and the cache keeps their pages; `chunk` c: a query sees only the keys of its own chunk of c positions,
+    counted from position 0; `head_norm_weight`: the norms per head have a weight of the head's size, one for all heads
+    (tensors `q_norm`, `k_norm`); `out_bias`: the output projection has a bias (`o_proj_bias`); `gate` "head": the gate is one
+    number per head, sigmoid(w_g[h] . input), in place of one per element.
 
     `window` w: the query at position p sees keys p-w+1 .. p.  `keep_window`: what the cache has to keep (the
     largest window of the layers that read it; a layer with `shares_cache` has no key and value projections and
@@ -153,9 +161,10 @@ class GatedAttention(Mixer):
 
     def __init__(self, weights: dict[str, str], hidden_size: int, num_heads: int, num_kv_heads: int, head_dim: int,
                  value_dim: int, scale: float, eps: float, window: int | None = None, keep_window: int | None = 0,
-                 distance_bias: bool = False, bias_far: float = 0.0, bias_rows: int = 32, gate: bool = True,
+                 distance_bias: bool = False, bias_far: float = 0.0, bias_rows: int = 32, gate: "bool | str" = True,
                  shares_cache: bool = False, sink: bool = False, position=None, query_temperature=None,
-                 head_norm: bool = False, bias: bool = False, keep_first: int = 0):
+                 head_norm: bool = False, bias: bool = False, keep_first: int = 0, chunk: int | None = None,
+                 head_norm_weight: bool = False, out_bias: bool = False):
         if num_heads % num_kv_heads:
             raise ValueError(f"num_heads={num_heads} is not a multiple of num_kv_heads={num_kv_heads}")
         self.hidden_size, self.num_heads, self.num_kv_heads = hidden_size, num_heads, num_kv_heads
@@ -165,15 +174,23 @@ class GatedAttention(Mixer):
         self.keep_window = None if self.window is None or keep_window is None else max(int(keep_window), self.window)
         # the table's number of rows is the checkpoint's (`bias_rows` only says how many the random-weights mode draws)
         self.distance_bias, self.bias_far, self.bias_rows = bool(distance_bias), float(bias_far), int(bias_rows)
-        self.gate, self.shares_cache = bool(gate), bool(shares_cache)
+        if gate not in (True, False, "head"):
+            raise ValueError(f"gate={gate!r}: one per element (True), one per head (\"head\") or none (False)")
+        self.gate, self.shares_cache = gate, bool(shares_cache)
         self.has_sink, self.position = bool(sink), position
         if position is not None and position.rotary_dim > head_dim:
             raise ValueError(f"a rotation of {position.rotary_dim} elements in heads of {head_dim}")
         self.head_norm, self.bias = bool(head_norm), bool(bias)
         if self.bias and not self.head_norm:
             raise ValueError("biases on q, k and v come with the norm per head")
-        if self.head_norm and (shares_cache or gate or position is not None or query_temperature is not None):
-            raise ValueError("the norm per head comes without a gate, a rotation, a temperature or a shared cache")
+        if self.head_norm and (shares_cache or query_temperature is not None):
+            raise ValueError("the norm per head comes without a temperature or a shared cache")
+        self.head_norm_weight, self.out_bias = bool(head_norm_weight), bool(out_bias)
+        if self.head_norm_weight and not self.head_norm:
+            raise ValueError("head_norm_weight goes with head_norm")
+        if chunk is not None and (int(chunk) < 1 or shares_cache):
+            raise ValueError(f"chunk={chunk} must be positive, in a layer with a cache of its own")
+        self.chunk = int(chunk) if chunk else None
         self.keep_first = int(keep_first) if self.window is not None else 0
         if self.keep_first < 0:
             raise ValueError(f"keep_first={keep_first}")
@@ -188,14 +205,16 @@ class GatedAttention(Mixer):
         if self.cache_dim > MAX_HEAD_DIM:
             raise ValueError(f"head sizes {head_dim} / {value_dim}: the attention kernels take heads of at most {MAX_HEAD_DIM}")
         self.names = weights
-        self.w_in = self.b_in = self.w_o = self.q_weight = self.k_weight = self.bias_by_distance = None
+        self.w_in = self.b_in = self.w_o = self.b_o = self.q_weight = self.k_weight = self.bias_by_distance = None
 
     def cache_requirement(self):
-        return PagedKV(self.num_kv_heads, self.cache_dim, self.keep_window, keep_first=self.keep_first)
+        return PagedKV(self.num_kv_heads, self.cache_dim, self.keep_window, self.chunk, self.keep_first)
 
     def attention_plan_key(self):
         key = (self.num_heads // self.num_kv_heads, self.num_kv_heads, self.window, self.cache_dim)
-        return key + (None, self.keep_first) if self.keep_first else key
+        if self.keep_first:
+            return key + (self.chunk, self.keep_first)
+        return key + (self.chunk,) if self.chunk else key
 
     def tensor_specs(self):
         h, d, dv = self.hidden_size, self.head_dim, self.value_dim
@@ -203,6 +222,11 @@ class GatedAttention(Mixer):
                self.names["o_proj"]: TensorSpec((h, self.num_heads * dv))}
         if not self.head_norm:
             out[self.names["q_norm"]] = TensorSpec((self.num_heads * d,), role="vector", init="norm")
+        elif self.head_norm_weight:
+            for k in ("q_norm", "k_norm"):
+                out[self.names[k]] = TensorSpec((d,), role="vector", init="norm")
+        if self.out_bias:
+            out[self.names["o_proj_bias"]] = TensorSpec((h,), role="vector", init="norm_zero")
         if not self.shares_cache:
             out[self.names["k_proj"]] = TensorSpec((self.num_kv_heads * d, h))
             out[self.names["v_proj"]] = TensorSpec((self.num_kv_heads * dv, h))
@@ -214,7 +238,7 @@ class GatedAttention(Mixer):
         if self.distance_bias:
             out[self.names["rel"]] = TensorSpec((-1, self.num_heads), role="vector", draw_shape=(self.bias_rows, self.num_heads))
         if self.gate:
-            out[self.names["g_proj"]] = TensorSpec((self.num_heads * dv, h))
+            out[self.names["g_proj"]] = TensorSpec((self.num_heads * (1 if self.gate == "head" else dv), h))
         if self.has_sink:
             out[self.names["sink"]] = TensorSpec((self.num_heads,), role="vector", init="norm_zero")
         return out
@@ -223,8 +247,12 @@ class GatedAttention(Mixer):
         if self.has_sink:
             self.sink = tensors[self.names["sink"]].float().contiguous()
         stack = ["q_proj"] + ([] if self.shares_cache else ["k_proj", "v_proj"]) + (["g_proj"] if self.gate else [])
-        self.w_in = torch.cat([tensors[self.names[k]] for k in stack], dim=0).contiguous()
+        self.w_in = padded_rows(torch.cat([tensors[self.names[k]] for k in stack], dim=0), 8 if self.gate == "head" else 1)
         self.w_o = tensors[self.names["o_proj"]].contiguous()
+        if self.out_bias:
+            self.b_o = tensors[self.names["o_proj_bias"]].float().contiguous()
+        if self.head_norm_weight:
+            self.q_weight, self.k_weight = (tensors[self.names[k]].float().contiguous() for k in ("q_norm", "k_norm"))
         if not self.head_norm:
             self.q_weight = tensors[self.names["q_norm"]].float().contiguous()
             self.k_weight = None if self.shares_cache else tensors[self.names["k_norm"]].float().contiguous()
@@ -251,19 +279,29 @@ class GatedAttention(Mixer):
         block_table = ctx.block_tables[cache.group]
         proj = ops.linear(h, self.w_in)
         if self.head_norm:
-            q = ops.unit_qkv_write(proj, self.b_in, nh, nkv, d, dv, D, self.eps, ctx, cache.kv, block_table, write=cache.owner)
+            options = {} if self.position is None and not self.head_norm_weight else dict(
+                position=self.position, q_weight=self.q_weight, k_weight=self.k_weight)
+            q = ops.unit_qkv_write(proj, self.b_in, nh, nkv, d, dv, D, self.eps, ctx, cache.kv, block_table, write=cache.owner, **options)
         else:
             q = ops.normed_qkv_write(proj, nh, nkv, d, dv, D, self.q_weight, self.k_weight, self.eps, ctx, cache.kv,
                                      block_table, has_kv=not self.shares_cache, write=cache.owner and not self.shares_cache,
                                      position=self.position, query_temperature=self.query_temperature)
+        return self._attend(q, proj, ctx, cache, block_table)
+
+    def _attend(self, q, proj, ctx, cache, block_table):
+        """Attention of the queries [T, heads * cache_dim] over the cache, the gate, the output projection."""
+        ops = ctx.ops
+        nh, nkv, d, dv, D = self.num_heads, self.num_kv_heads, self.head_dim, self.value_dim, self.cache_dim
         extra = {"keep_first": self.keep_first} if self.keep_first else {}
+        if self.chunk:
+            extra["chunk"] = self.chunk
         o = ops.paged_attention(q, nh, nkv, D, cache.kv, block_table, ctx, self.scale, self.window,
                                 dist_bias=self.bias_by_distance, sink=self.sink, **extra)
         if not self.gate and D == dv:
-            return LazyLinear(o, self.w_o)
+            return LazyLinear(o, self.w_o, self.b_o)
         g0 = nh * d + (0 if self.shares_cache else nkv * (d + dv))
-        o = ops.head_gate(o, nh, D, dv, proj[:, g0:g0 + nh * dv] if self.gate else None)
-        return LazyLinear(o, self.w_o)
+        o = ops.head_gate(o, nh, D, dv, proj[:, g0:g0 + nh * (1 if self.gate == "head" else dv)] if self.gate else None)
+        return LazyLinear(o, self.w_o, self.b_o)
 
 
 @register_mixer("rotated_value_attention")

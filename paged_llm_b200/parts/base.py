@@ -53,11 +53,13 @@ class ScheduleEntry:
     `cache_from` names an earlier schedule entry whose cache this run reads
     instead of keeping one itself.  `add_embedding`: before this run the output
     of the embedding (the stream as it was in front of the first run) is added
-    to the stream once more."""
+    to the stream once more.  `join_embedding`: before this run the model's
+    `stream_join` forms the stream anew from itself and the embedding's output."""
 
     layer: int
     cache_from: int | None = None
     add_embedding: bool = False
+    join_embedding: bool = False
 
 
 @dataclass
@@ -70,6 +72,7 @@ class ModelSpec:
     final_norm: PartSpec
     head: PartSpec
     positions: dict[str, PartSpec] = field(default_factory=dict)   # position encodings by name
+    stream_join: PartSpec | None = None                            # for schedule entries with `join_embedding`
     ignored_tensors: tuple[str, ...] = ()                          # name suffixes a checkpoint may carry
 
 
@@ -145,19 +148,20 @@ class LazyLinear:
     instead of a tensor.  The norm that consumes the branch can then let one
     kernel do projection + residual sum + normalisation; anything else calls
     `materialize`.  A part that returns a plain tensor works everywhere too.
-    `bias` (float32 [out] or None) is added to the product."""
+    `bias` (float32 [out] or None) is added to the product; `float32`: the product stays float32."""
 
     input: torch.Tensor
     weight: torch.Tensor
     bias: torch.Tensor | None = None
+    float32: bool = False
 
     def materialize(self, ops) -> torch.Tensor:
-        y = ops.linear(self.input, self.weight)
+        y = ops.linear(self.input, self.weight, out_float32=self.float32)
         return y if self.bias is None else ops.add_bias(y, self.bias)
 
     def rows(self, ops, idx: torch.Tensor) -> "LazyLinear":
         """The same branch for the rows `idx` only."""
-        return LazyLinear(ops.gather_rows(self.input, idx), self.weight, self.bias)
+        return LazyLinear(ops.gather_rows(self.input, idx), self.weight, self.bias, self.float32)
 
 
 @dataclass
@@ -216,6 +220,44 @@ class LazyNormedPair:
         return LazyNormedPair(ops.gather_rows(self.a, idx), ops.gather_rows(self.b, idx), self.weights, self.scales, self.eps)
 
 
+@dataclass
+class LazyExperts:
+    """The weighted sum of a token's chosen experts' outputs, not formed yet: token t's value is the sum over j < top of
+    weights[t, j] * rows[place[t, j]].  `place` None: the pair (t, j) is row t * top + j; `weights` None: the rows carry
+    their weights already.  `tokens` (int32, on the device): the branch holds these tokens only, in this order.  A norm may
+    form the sum beside the residual sum; anything else calls `materialize`."""
+
+    rows_: torch.Tensor
+    top: int
+    place: torch.Tensor | None
+    weights: torch.Tensor | None
+    count: int
+    tokens: torch.Tensor | None = None
+
+    def materialize(self, ops) -> torch.Tensor:
+        return ops.branch_sum([self])
+
+    def rows(self, ops, idx: torch.Tensor) -> "LazyExperts":
+        if self.tokens is not None:
+            raise ValueError("rows of rows of a deferred sum of experts")
+        return LazyExperts(self.rows_, self.top, self.place, self.weights, idx.numel(), idx)
+
+
+@dataclass
+class LazySum:
+    """A branch output that is the sum of one or two branches (tensors, `LazyLinear` or `LazyExperts`), not formed yet (a
+    layer whose mixer and feed-forward read the same norm).  The RMS norm that follows adds both to the stream in its own
+    kernel; anything else calls `materialize`."""
+
+    parts: tuple
+
+    def materialize(self, ops) -> torch.Tensor:
+        return ops.branch_sum(list(self.parts))
+
+    def rows(self, ops, idx: torch.Tensor) -> "LazySum":
+        return LazySum(tuple(p.rows(ops, idx) if hasattr(p, "rows") else ops.gather_rows(p, idx) for p in self.parts))
+
+
 def branch_args(branch, ops):
     """(branch tensor, keyword arguments) for `ops.stream_norm`: a pair travels as two branches with their scales and
     biases, everything else as one tensor."""
@@ -241,7 +283,8 @@ class StreamBranch:
 
 
 def materialize(branch, ops):
-    return branch.materialize(ops) if isinstance(branch, (LazyLinear, LazyNormed, LazyPair, LazyNormedPair)) else branch
+    lazy = (LazyLinear, LazyNormed, LazyPair, LazyNormedPair, LazyExperts, LazySum)
+    return branch.materialize(ops) if isinstance(branch, lazy) else branch
 
 
 # --------------------------------------------------------------------------- interfaces
@@ -329,6 +372,19 @@ class FeedForward(Part):
         raise NotImplementedError
 
 
+class StreamJoin(Part):
+    """Forms the stream anew from itself and the embedding's output, in front of a run of a layer."""
+
+    def start(self, x0: torch.Tensor, times: int, ctx):
+        """What the step's joins share, formed once from the embedding's output `x0` [T, hidden] float32, which is not
+        kept (the stream is summed up in place).  `times`: how often `forward` will be called."""
+        raise NotImplementedError
+
+    def forward(self, x, pending, shared, ctx):
+        """The stream (x, pending) -> the new one, again a pair."""
+        raise NotImplementedError
+
+
 class Block(Part):
     """Arrangement of norms, mixer and feed-forward around the residual stream.
 
@@ -372,6 +428,7 @@ POSITION_ENCODINGS: dict[str, Callable[..., PositionEncoding]] = {}
 BLOCKS: dict[str, Callable[..., Block]] = {}
 EMBEDDINGS: dict[str, Callable[..., Embedding]] = {}
 HEADS: dict[str, Callable[..., Head]] = {}
+STREAM_JOINS: dict[str, Callable[..., StreamJoin]] = {}
 
 
 def _register(table: dict, what: str):
@@ -392,6 +449,7 @@ register_position_encoding = _register(POSITION_ENCODINGS, "position encoding")
 register_block = _register(BLOCKS, "block")
 register_embedding = _register(EMBEDDINGS, "embedding")
 register_head = _register(HEADS, "head")
+register_stream_join = _register(STREAM_JOINS, "stream join")
 
 
 def make_part(table: dict, what: str, spec: PartSpec, **extra):

@@ -8,7 +8,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import (NORMS, Block, LazyLinear, LazyNormed, PartSpec, StreamBranch, TensorSpec, branch_args, make_part,
+from .base import (NORMS, Block, LazyLinear, LazyNormed, LazySum, PartSpec, StreamBranch, TensorSpec, branch_args, make_part,
                    register_block)
 
 
@@ -28,6 +28,21 @@ class PreNormBlock(Block):
             h = ctx.ops.materialize(h)
         f = self.feed_forward.forward(h, ctx)
         return x, f
+
+
+@register_block("parallel_norm")
+class ParallelNormBlock(Block):
+    """One norm in front of both parts: h = input(x); x += mixer(h) + ffn(h).  Both outputs travel unsummed (`LazySum`), so
+    that the norm that follows adds them, with the bias an output projection may have, in its own kernel."""
+
+    NORM_NAMES = ("input",)
+
+    def forward(self, x, pending, ctx, cache):
+        h = self.norms["input"].add_forward(x, pending, ctx)
+        if not (self.mixer.accepts_lazy_input and (self.feed_forward is None or self.feed_forward.accepts_lazy_input)):
+            h = ctx.ops.materialize(h)
+        a = self.mixer.forward(h, ctx, cache)
+        return x, LazySum((a,) if self.feed_forward is None else (a, self.feed_forward.forward(h, ctx)))
 
 
 @register_block("sandwich_norm")

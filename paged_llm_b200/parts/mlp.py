@@ -47,6 +47,34 @@ class GatedMLP(FeedForward):
         return LazyLinear(ops.gated_act_linear(h, self.w_gate_up, self.activation), self.w_down)
 
 
+@register_feed_forward("ungated_mlp")
+class UngatedMLP(FeedForward):
+    """down(act(up(x))) with no gate and no bias; act is the square of relu ("relu2")."""
+
+    accepts_lazy_input = True
+
+    def __init__(self, weights: dict[str, str], hidden_size: int, intermediate_size: int, activation: str = "relu2"):
+        if activation != "relu2":
+            raise ValueError(f"activation {activation!r} is not implemented (relu2 only)")
+        self.hidden_size, self.intermediate_size, self.activation = hidden_size, intermediate_size, activation
+        self.names = weights
+        self.w_up = self.w_down = None
+
+    def tensor_specs(self):
+        h, i = self.hidden_size, self.intermediate_size
+        return {self.names["up_proj"]: TensorSpec((i, h)), self.names["down_proj"]: TensorSpec((h, i))}
+
+    def load(self, tensors):
+        self.w_up = tensors[self.names["up_proj"]].contiguous()
+        self.w_down = tensors[self.names["down_proj"]].contiguous()
+
+    def bytes_read_per_step(self):
+        return sum(w.numel() * w.element_size() for w in (self.w_up, self.w_down))
+
+    def forward(self, h, ctx):
+        return LazyLinear(ctx.ops.relu2_linear(h, self.w_up), self.w_down)
+
+
 @register_feed_forward("poly_norm_mlp")
 class PolyNormMLP(FeedForward):
     """down(act(up(x))) with no gate and no bias, where the activation is a polynomial of unit-norm powers:

@@ -12,7 +12,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import LazyLinear, LazyNormed, LazyNormedPair, LazyPair, Norm, StreamBranch, TensorSpec, branch_args, materialize, register_norm
+from .base import LazyExperts, LazyLinear, LazyNormed, LazyNormedPair, LazyPair, LazySum, Norm, StreamBranch, TensorSpec, branch_args, materialize, register_norm
 
 
 @register_norm("rms_norm")
@@ -55,6 +55,9 @@ class RMSNorm(Norm):
             return ops.stream_norm(x, self.streams, y, None, None, None, self.weight, self.groups, self.eps, **pair)
         if branch is None:
             return ctx.ops.rms_norm(x, self.weight, self.eps)
+        if isinstance(branch, (LazySum, LazyExperts)):
+            # the branches' sum, their biases, the residual sum and this norm in one kernel
+            return ctx.ops.branches_add_rms_norm(x, list(branch.parts) if isinstance(branch, LazySum) else [branch], self.weight, self.eps)
         if isinstance(branch, LazyNormedPair):
             # both norms of the pair, the residual sum and this norm in one kernel
             return ctx.ops.normed_pair_add_rms_norm(x, branch.a, branch.b, branch.weights[0], branch.weights[1],
@@ -66,7 +69,8 @@ class RMSNorm(Norm):
         if isinstance(branch, LazyPair) or (isinstance(branch, LazyLinear) and branch.bias is not None):
             branch = branch.materialize(ctx.ops)
         if isinstance(branch, LazyLinear):
-            return ctx.ops.linear_add_rms_norm(branch.input, branch.weight, x, self.weight, self.eps)
+            return ctx.ops.linear_add_rms_norm(branch.input, branch.weight, x, self.weight, self.eps,
+                                               **({"out_float32": True} if branch.float32 else {}))
         return ctx.ops.add_rms_norm(x, branch, self.weight, self.eps)
 
 

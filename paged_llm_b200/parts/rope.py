@@ -57,7 +57,7 @@ def yarn_rescale(inv_freq: torch.Tensor, base: float, factor: float, original: f
 @register_position_encoding("rotary")
 class RotaryEncoding(PositionEncoding):
     def __init__(self, weights: dict[str, str], head_dim: int, theta: float,
-                 scaling: dict | None = None, rotary_dim: int | None = None, pairing: str = "half"):
+                 scaling: dict | None = None, rotary_dim: int | None = None, pairing: str = "half", exact: bool = False):
         self.head_dim = head_dim
         self.rotary_dim = head_dim if rotary_dim is None else rotary_dim
         if self.rotary_dim % 2 or not 0 < self.rotary_dim <= head_dim:
@@ -65,6 +65,7 @@ class RotaryEncoding(PositionEncoding):
         if pairing not in ("half", "interleaved"):
             raise ValueError(f"unknown rotary pairing {pairing!r}")
         self.theta, self.scaling, self.pairing = float(theta), scaling, pairing
+        self.exact = bool(exact)     # frequencies formed in float64 and rounded once (else float32, the reference's order)
         self.table = None            # [P, rotary_dim/2, 2] float32: (cos, sin)
         self.max_positions = 0
 
@@ -81,12 +82,13 @@ class RotaryEncoding(PositionEncoding):
             sc = self.scaling
             return yarn_rescale(inv, self.theta, float(sc["factor"]), float(sc["original"]), float(sc["fast"]),
                                 float(sc["slow"]))
-        inv = 1.0 / (self.theta ** (torch.arange(0, rd, 2, dtype=torch.float32) / rd))
+        dtype = torch.float64 if self.exact else torch.float32
+        inv = 1.0 / (self.theta ** (torch.arange(0, rd, 2, dtype=dtype) / rd))
         if kind == "llama3":
             inv = llama3_rescale(inv, **{k: v for k, v in self.scaling.items() if k not in ("rope_type", "type")})
         elif kind not in (None, "default"):
             raise NotImplementedError(f"rope_type={kind!r} not supported (default, llama3 and yarn only)")
-        return inv, 1.0
+        return inv.float(), 1.0
 
     def prepare(self, max_positions, device, ops):
         self.max_positions = int(max_positions)

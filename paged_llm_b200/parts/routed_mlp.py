@@ -12,6 +12,8 @@ groups can be chosen.  `activation` "swish_clamped" with `activation_limit` L: g
 the expert's inner vector is g * sigmoid(1.702 g) * (u + 1).  `scoring` "softmax": the scores are the softmax of z over
 all experts.  `correction`: one learned number per expert joins its score for the choice (and in the groups' scores), not
 for the weights.  `renorm`: the chosen scores are divided by their sum (+ 1e-20); `weight_scale` multiplies the weights.
+`router_bias`: one learned number per expert is added to z (tensor `router_bias`), so it takes part in the choice and in the
+softmax over the chosen.  `defer_sum`: the weighted sum is left to the norm that follows (`LazyExperts`).
 `gated` False: an expert, and the shared one, is down(act(up h)) with the square of relu ("relu2") as act.  `shared_gate`
 False: the shared expert is added as it is.
 
@@ -37,7 +39,7 @@ class RoutedMLP(FeedForward):
                  activation: str = "silu", shared_size: int | None = None, shared_activation: str | None = None,
                  activation_limit: float | None = None, scoring: str = "softmax_top", groups=None,
                  group_score_top: int = 2, gated: bool = True, shared_gate: bool = True, correction: bool = False,
-                 renorm: bool = False, weight_scale: float = 1.0):
+                 renorm: bool = False, weight_scale: float = 1.0, router_bias: bool = False, defer_sum: bool = False):
         if not 1 <= top_k <= num_experts:
             raise ValueError(f"top_k={top_k} of {num_experts} experts")
         for a in (activation, shared_activation or activation):
@@ -52,6 +54,11 @@ class RoutedMLP(FeedForward):
             raise ValueError(f"scoring {scoring!r} is not implemented (softmax_top, sigmoid and softmax only)")
         if scoring == "softmax_top" and (correction or renorm or weight_scale != 1.0):
             raise ValueError("a correction, renormalised weights and their scale go with sigmoid and softmax scores")
+        if router_bias and scoring != "softmax_top":
+            raise ValueError("a bias on the router's logits goes with the softmax over the chosen logits")
+        if defer_sum and shared_size is not None:
+            raise ValueError("a shared expert is added where the experts' sum is formed: the sum cannot be deferred")
+        self.has_router_bias, self.defer_sum, self.router_bias = bool(router_bias), bool(defer_sum), None
         if shared_size is not None and shared_gate and scoring != "softmax_top":
             raise ValueError("a shared expert's gate rides with the softmax over the chosen experts only")
         self.gated, self.shared_gate, self.has_correction = bool(gated), bool(shared_gate), bool(correction)
@@ -84,6 +91,8 @@ class RoutedMLP(FeedForward):
             out[self.names[f"e{e}.down"]] = TensorSpec((d, f))
         if self.has_correction:
             out[self.names["correction"]] = TensorSpec((self.num_experts,), role="vector", init="norm_zero")
+        if self.has_router_bias:
+            out[self.names["router_bias"]] = TensorSpec((self.num_experts,), role="vector", init="norm_zero")
         if self.shared_size is not None:
             s = self.shared_size
             if self.gated:
@@ -106,6 +115,8 @@ class RoutedMLP(FeedForward):
             if self.shared_gate:
                 router.append(t[n["shared.sg"]])
             self.shared = (first("shared.").contiguous(), t[n["shared.down"]].contiguous())
+        if self.has_router_bias:
+            self.router_bias = t[n["router_bias"]].float().contiguous()
         if self.has_correction:
             self.correction = t[n["correction"]].float().contiguous()
         rows = sum(r.shape[0] for r in router)
@@ -132,6 +143,10 @@ class RoutedMLP(FeedForward):
         out = {}
         if not self.gated:
             out["gated"] = False
+        if self.router_bias is not None:
+            out["router_bias"] = self.router_bias
+        if self.defer_sum:
+            out["defer_sum"] = True
         if self.shared is not None and not self.shared_gate:
             out["shared_gate"] = False
         if self.scoring != "softmax_top" and (self.correction is not None or self.renorm or self.weight_scale != 1.0):

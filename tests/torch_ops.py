@@ -44,6 +44,29 @@ class TorchOps:
         self._count("softcap")
         return cap * torch.tanh(logits / cap)
 
+    def add_copy(self, x, branch):
+        branch = self.branch_sum(list(branch.parts)) if hasattr(branch, "parts") else branch
+        if hasattr(branch, "materialize"):
+            branch = branch.materialize(self)
+        return self.add_rows(x, branch).to(self.compute_dtype)
+
+    def stream_copy(self, x):
+        return x.to(self.compute_dtype)
+
+    def branch_sum(self, parts):
+        self._count("branch_sum")
+        total = 0.0
+        for b in parts:
+            y = b
+            if hasattr(b, "materialize"):
+                y = self.linear(b.input, b.weight).float() + (b.bias if b.bias is not None else 0.0)
+            total = total + y.float()
+        return total
+
+    def branches_add_rms_norm(self, x, parts, w, eps):
+        x += self.branch_sum(parts)
+        return self.rms_norm(x, w, eps)
+
     def token_side_gate(self, x, branch, w_gate, table, offset, dim, ids):
         self._count("token_side_gate")
         if hasattr(branch, "materialize"):
@@ -153,10 +176,12 @@ class TorchOps:
 
     def routed_experts(self, h, w_router, w_gate_up, w_down, top_k, activation="silu", shared=None,
                        shared_activation="silu", activation_limit=0.0, scoring="softmax_top", groups=None, gated=True,
-                       shared_gate=True, correction=None, renorm=False, weight_scale=1.0):
+                       shared_gate=True, correction=None, renorm=False, weight_scale=1.0, router_bias=None, defer_sum=False):
         self._count("routed_experts")
         E = w_gate_up.shape[0]
         z = h.float() @ w_router.float().T              # (rows behind the experts' and the gate's are padding)
+        if router_bias is not None:
+            z[:, :E] += router_bias
         if scoring in ("sigmoid", "softmax"):
             sc = torch.sigmoid(z[:, :E]) if scoring == "sigmoid" else torch.softmax(z[:, :E], dim=-1)
             pick = sc if correction is None else sc + correction
@@ -190,8 +215,8 @@ class TorchOps:
     def materialize(self, h):
         return h
 
-    def linear_add_rms_norm(self, h, w, x, norm_w, eps):
-        return self.add_rms_norm(x, self.linear(h, w), norm_w, eps)
+    def linear_add_rms_norm(self, h, w, x, norm_w, eps, out_float32=False):
+        return self.add_rms_norm(x, self.linear(h, w, out_float32), norm_w, eps)
 
     def gated_silu_linear(self, h, w_gate_up):
         return self.silu_mul(self.linear(h, w_gate_up))
@@ -540,7 +565,47 @@ class TorchOps:
         g = g * torch.sigmoid(g) if gate == "silu" else torch.sigmoid(g)
         return (v.reshape(T, H * dv) * g).to(self.compute_dtype)
 
-    def unit_qkv_write(self, proj, bias, nh, nkv, d, dv, D, eps, ctx, kv, block_table, write=True):
+    def conv_qkv_write(self, proj, conv_w, nh, nkv, d, dv, D, position, state, ctx, kv, block_table, write=True):
+        self._count("conv_qkv_write")
+        T = proj.shape[0]
+        taps, C = conv_w.shape
+        hist = taps - 1
+        out = torch.zeros(T, C)
+        cu = ctx.host.cu
+        for s, slot in enumerate(ctx.host.state_slots):
+            seq = proj[cu[s]:cu[s + 1], :C].float()
+            nq = seq.shape[0]
+            if hist:
+                assert slot >= 0, "a request of a model with state must own a slot"
+                seq = torch.cat([state[slot].view(hist, C), seq], dim=0)
+            for j in range(taps):
+                out[cu[s]:cu[s + 1]] += conv_w[j] * seq[j:j + nq]
+            if hist:
+                state[slot] = seq[nq:].reshape(-1).clone()
+        return self.rotated_qkv_write(out.to(proj.dtype), None, nh, nkv, d, dv, D, position, None, ctx, kv, block_table, write)
+
+    def fixed_decay_attention(self, proj, H, d, dv, decay, state, ctx):
+        self._count("fixed_decay_attention")
+        T = proj.shape[0]
+        pf = torch.nn.functional.silu(proj[:, :2 * H * d + H * dv].float())
+        q, k, v = pf[:, :H * d].view(T, H, d), pf[:, H * d:2 * H * d].view(T, H, d), pf[:, 2 * H * d:].view(T, H, dv)
+        out = torch.zeros(T, H * dv)
+        cu = ctx.host.cu
+        for s, slot in enumerate(ctx.host.state_slots):
+            assert slot >= 0, "a request of a model with state must own a slot"
+            S = state[slot].view(H, dv, d)
+            for t in range(cu[s], cu[s + 1]):
+                S.mul_(decay[:, None, None]).add_(v[t][:, :, None] * k[t][:, None, :])
+                out[t] = torch.einsum("hvd,hd->hv", S, q[t]).reshape(H * dv)
+        return out
+
+    def row_norm_gate(self, o, proj, g_col0, norm_w, eps):
+        self._count("row_norm_gate")
+        g = torch.sigmoid(proj[:, g_col0:g_col0 + o.shape[1]].float())
+        return (o * torch.rsqrt((o * o).mean(-1, keepdim=True) + eps) * norm_w * g).to(self.compute_dtype)
+
+    def unit_qkv_write(self, proj, bias, nh, nkv, d, dv, D, eps, ctx, kv, block_table, write=True, position=None, q_weight=None,
+                       k_weight=None):
         self._count("unit_qkv_write")
         T = proj.shape[0]
         pf = proj[:, :nh * d + nkv * (d + dv)].float()
@@ -550,9 +615,13 @@ class TorchOps:
         def unit(x):
             return x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps)
 
+        def finished(x, weight):
+            x = unit(x) if weight is None else unit(x) * weight
+            return x if position is None else self._turn(x, position, ctx.positions.long())
+
         q, k, v = torch.zeros(T, nh, D), torch.zeros(T, nkv, D), torch.zeros(T, nkv, D)
-        q[:, :, :d] = unit(pf[:, :nh * d].view(T, nh, d))
-        k[:, :, :d] = unit(pf[:, nh * d:(nh + nkv) * d].view(T, nkv, d))
+        q[:, :, :d] = finished(pf[:, :nh * d].view(T, nh, d), q_weight)
+        k[:, :, :d] = finished(pf[:, nh * d:(nh + nkv) * d].view(T, nkv, d), k_weight)
         v[:, :, :dv] = pf[:, (nh + nkv) * d:].view(T, nkv, dv)
         if write:
             self._write_slots(ctx, kv, block_table, k, v)
@@ -590,7 +659,8 @@ class TorchOps:
         T = o.shape[0]
         out = o.float().view(T, nh, D)[:, :, :dv].reshape(T, nh * dv)
         if gate is not None:
-            out = out * torch.sigmoid(gate.float())
+            g = torch.sigmoid(gate.float())
+            out = out * (g.repeat_interleave(dv, dim=1) if g.shape[1] == nh else g)
         return out.to(self.compute_dtype)
 
     @staticmethod
