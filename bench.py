@@ -122,6 +122,22 @@ TAGELORN_SIZES = {
     "t-tiny": dict(vocab=256, width=128, heads=4, kv_heads=2, dim=32, window=64, keep_first=4, delta_heads=4, delta_dim=16, ff=256,
                    experts=8, top=2, groups=(4, 2), expert_ff=64, shared_ff=64, taps=3, side_dim=24),
 }
+# Nopozen at the layer sizes of a 2k- and a 4k-wide model: chunked attention, linear attention with a fixed decay, convolved
+# attention; the first feed-forward dense, the others routed experts; layers 1 to 3 run twice.  The Pomisun beside it gets the
+# same widths, heads, chunk, experts and loop (attention only); the Munazen the same widths, heads and linear-attention heads
+# (its linear attention has a decay per channel), as many layers as the Nopozen has runs, and top * expert_ff as inner size
+NOPOZEN_SIZES = {
+    "n-2k": dict(vocab=32000, width=2048, heads=16, kv_heads=4, dim=128, chunk=1024, lin_heads=16, lin_dim=128, taps=3, ff=8192,
+                 experts=32, top=4, expert_ff=1024, rec_blocks=16),
+    "n-4k": dict(vocab=32000, width=4096, heads=32, kv_heads=8, dim=128, chunk=1024, lin_heads=32, lin_dim=128, taps=3, ff=14336,
+                 experts=64, top=6, expert_ff=1408, rec_blocks=16),
+    # heads of 64 in every mixer
+    "n-2k-64": dict(vocab=32000, width=2048, heads=32, kv_heads=8, dim=64, chunk=1024, lin_heads=32, lin_dim=64, taps=3, ff=8192,
+                    experts=32, top=4, expert_ff=1024, rec_blocks=16),
+    # for trying the option out quickly; never a result
+    "n-tiny": dict(vocab=256, width=128, heads=4, kv_heads=2, dim=32, chunk=64, lin_heads=4, lin_dim=16, taps=3, ff=256, experts=8,
+                   top=2, expert_ff=64, rec_blocks=4),
+}
 PROMPT_LEN, DECODE_LEN, PREFILL_TOKENS, BLOCK_SIZE = 512, 256, 2048, 16
 RAGGED_PROMPTS, RAGGED_OUTPUTS = (128, 4096), (64, 512)      # the ragged serving workload: lengths drawn uniformly
 
@@ -663,7 +679,11 @@ def rokarax_configs(name: str):
 
 def munazen_configs(name: str):
     """(Munazen configuration dict, Llama configuration dict of equal size, number of layers)."""
-    s = MUNAZEN_SIZES[name]
+    return munazen_configs_of(MUNAZEN_SIZES[name])
+
+
+def munazen_configs_of(s: dict):
+    """The same for sizes that no name stands for."""
     left = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5,
             "rot": {"dims": s["dim"], "base": 500000.0, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
     par = {"left": left, "right": {"width": s["rec_width"], "blocks": s["rec_blocks"], "conv": s["conv"]},
@@ -726,10 +746,37 @@ def tagelorn_configs(name: str):
     return tag, pir, len(order)
 
 
-def compare_with_llama(args, label: str, size: str, sizes: dict, model: dict, llama: dict, runs: int, beside: str = "llama") -> dict:
+def nopozen_configs(name: str):
+    """(Nopozen, Pomisun and Munazen configuration dicts of equal size, number of layer runs)."""
+    s = NOPOZEN_SIZES[name]
+    heads = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5}
+    rot = {"dims": s["dim"], "base": 500000.0}
+    chunked = dict(heads, mask={"size": s["chunk"]}, rot=dict(rot, scaling={"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}))
+    convolved = dict(heads, rot=dict(rot, dims=s["dim"] // 2), conv=s["taps"])
+    linear = {"heads": s["lin_heads"], "dim": s["lin_dim"], "vdim": s["lin_dim"],
+              "decay": [1.0 - 2.0 ** (-2.0 - 6.0 * i / s["lin_heads"]) for i in range(s["lin_heads"])]}
+    dense = {"kind": "dense", "ff": s["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": s["expert_ff"]}, "router": {"experts": s["experts"], "top": s["top"]}}
+    loop = {"start": 1, "stop": 4, "times": 2}
+    order = [("attention", chunked, dense), ("lightning", linear, moe), ("attention_2", convolved, moe), ("attention", chunked, moe),
+             ("lightning", linear, moe), ("attention_2", convolved, moe)]
+    top = {"vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}}
+    nop = dict(top, architecture="Nopozen", layers=[{"type": t, "mixer": m, "mlp": f} for t, m, f in order], loop=loop)
+    pom_mixer = dict(heads, mask={"size": s["chunk"]}, rot=dict(rot, scaling={"factor": 4.0, "original": 4096, "fast": 16.0, "slow": 2.0}))
+    pom = dict(top, architecture="Pomisun", layers=[{"type": "attention", "mixer": pom_mixer, "mlp": f} for _, _, f in order], loop=loop)
+    mun, _, _ = munazen_configs_of(dict(vocab=s["vocab"], width=s["width"], heads=s["heads"], kv_heads=s["kv_heads"], dim=s["dim"],
+                                        ff=s["top"] * s["expert_ff"], rec_width=s["width"], rec_blocks=s["rec_blocks"], conv=s["taps"],
+                                        gla_heads=s["lin_heads"], gla_dim=s["lin_dim"], gla_vdim=s["lin_dim"], streams=1, norm_groups=1))
+    kinds = mun["layers"][:2]                       # attention beside the recurrence, linear attention
+    mun["layers"] = [kinds[i] for i in (0, 1, 0) * 3]
+    return nop, pom, mun, len(order) + 3
+
+
+def compare_with_llama(args, label: str, size: str, sizes: dict, model: dict, llama: dict, runs: int, beside: str = "llama",
+                       more: tuple = ()) -> dict:
     """Prefill and decode of another decoder at layer sizes of a real model (random weights drawn on the
-    device) beside a Llama (or the model named by `beside`) of equal width, heads and layer runs: device-timed with CUDA events, with the device
-    time of every kernel inside the steps for the roofline of each."""
+    device) beside a Llama (or the model named by `beside`, and those in `more`) of equal width, heads and layer runs:
+    device-timed with CUDA events, with the device time of every kernel inside the steps for the roofline of each."""
     import torch
     from paged_llm_b200 import EngineConfig, LLMEngine
     from paged_llm_b200.config.registry import parse_model_config
@@ -742,7 +789,7 @@ def compare_with_llama(args, label: str, size: str, sizes: dict, model: dict, ll
     max_len = max(ctx_len + steps + args.warmup + 16, pre) + 64
     out = {"only": label, "size": size, "layer_runs": runs, "prefill_tokens": pre, "context": ctx_len,
            "sizes": sizes, "peaks": load_peaks()}
-    for arm, hf in ((label, model), (beside, llama)):
+    for arm, hf in ((label, model), (beside, llama), *more):
         with tempfile.TemporaryDirectory() as folder:
             _, cfg = parse_model_config(hf)
             write_random_stub(folder, cfg, seed=0, std=0.02, dtype="bfloat16")
@@ -795,6 +842,12 @@ def tagelorn_compare(args) -> dict:
     return compare_with_llama(args, "tagelorn", args.tagelorn_size, TAGELORN_SIZES[args.tagelorn_size], tag, pir, runs, beside="pirerax")
 
 
+def nopozen_compare(args) -> dict:
+    nop, pom, mun, runs = nopozen_configs(args.nopozen_size)
+    return compare_with_llama(args, "nopozen", args.nopozen_size, NOPOZEN_SIZES[args.nopozen_size], nop, pom, runs, beside="pomisun",
+                              more=(("munazen", mun),))
+
+
 def run_ours(args) -> dict:
     import torch
     from paged_llm_b200 import EngineConfig, LLMEngine
@@ -810,6 +863,8 @@ def run_ours(args) -> dict:
         return pirerax_compare(args)
     if args.only == "tagelorn":
         return tagelorn_compare(args)
+    if args.only == "nopozen":
+        return nopozen_compare(args)
     if args.only == "validate":
         return validate(args)
     if args.only == "sample":
@@ -1012,14 +1067,17 @@ def main() -> int:
                     help="with --only pirerax: the layer sizes (the Llama beside it gets the same)")
     ap.add_argument("--tagelorn-size", choices=sorted(TAGELORN_SIZES), default="t-2k",
                     help="with --only tagelorn: the layer sizes (the Pirerax beside it gets the same)")
+    ap.add_argument("--nopozen-size", choices=sorted(NOPOZEN_SIZES), default="n-2k",
+                    help="with --only nopozen: the layer sizes (the Pomisun and the Munazen beside it get the same)")
     ap.add_argument("--only", choices=["decode", "prefill", "ragged", "mixed", "validate", "sample", "pomisun", "rokarax", "munazen",
-                                       "pirerax", "tagelorn"], default=None,
+                                       "pirerax", "tagelorn", "nopozen"], default=None,
                     help="run only the decode loop, only the prefill step, the ragged serving workload through "
                          "LLMEngine.generate, one mixed step (--batch decoding requests of --context tokens beside one "
                          "portion of --prefill-tokens), the float32 validation run, the sampler's kernels on --batch rows, or "
                          "prefill and decode of the Pomisun, the Rokarax, the Munazen or the Pirerax decoder beside a Llama of equal size "
                          "(--pomisun-size, --rokarax-size, --munazen-size, --pirerax-size), or of the Tagelorn decoder beside a Pirerax of "
-                         "equal size (--tagelorn-size), and print "
+                         "equal size (--tagelorn-size), or of the Nopozen decoder beside a Pomisun and a Munazen of equal size "
+                         "(--nopozen-size), and print "
                          "a short line")
     args = ap.parse_args()
     if args.gpus != 1 or int(os.environ.get("WORLD_SIZE", "1")) > 1:

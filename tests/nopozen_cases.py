@@ -212,27 +212,30 @@ def rounding_error(folder: str, tokens, dtype=torch.float32) -> np.ndarray:
     return (rounded.double() - exact).pow(2).mean(dim=1).sqrt().numpy()
 
 
-def clear_requests(folder: str, vocab: int, lengths, seed: int = 0, margin: float = 0.04) -> dict[str, list[int]]:
+def clear_requests(folder: str, vocab: int, lengths, seed: int = 0, margin: float = 0.1) -> dict[str, list[int]]:
     """Random requests on which no router of the model comes close to a tie (the last chosen expert's logit leads the next by
     `margin` at every token): a bfloat16 engine then chooses the experts the plain model chooses, and the two differ by
-    rounding only.  A length for which 40 draws find no such request is shortened."""
+    rounding only.  From its first close call on a request is drawn again, until there is none; one that does not get there is
+    cut in front of it."""
     cfg, w = read_folder(folder)
     out = {}
     for i, n in enumerate(lengths):
-        while f"r{i}" not in out:
-            for attempt in range(40):
-                g = torch.Generator().manual_seed(seed * 100003 + i * 401 + attempt)
-                toks = torch.randint(0, vocab, (n,), generator=g).tolist()
-                margins: list[float] = []
-                with torch.no_grad():
-                    plain_nopozen.forward(cfg, w, toks, margins)
-                if min(margins, default=1.0) >= margin:
-                    out[f"r{i}"] = toks
-                    break
-            else:
-                if n <= 2:
-                    raise AssertionError("no request without a close call, however short")
-                n = max(2, n // 2)
+        g = torch.Generator().manual_seed(seed * 100003 + i * 401)
+        toks = torch.randint(0, vocab, (n,), generator=g).tolist()
+        for attempt in range(60):
+            margins: list[float] = []
+            with torch.no_grad():
+                plain_nopozen.forward(cfg, w, toks, margins)
+            close = (np.array(margins).reshape(-1, n).min(axis=0) < margin) if margins else np.zeros(n, bool)
+            if not close.any():
+                break
+            first = int(np.argmax(close))
+            toks[first:] = torch.randint(0, vocab, (n - first,), generator=g).tolist()
+        else:
+            toks = toks[:first]
+        if not toks:
+            raise AssertionError("no request without a close call, however short")
+        out[f"r{i}"] = toks
     return out
 
 
