@@ -10,7 +10,7 @@
 namespace {
 
 struct Branch {
-    const void* rows;       // null: no branch
+    const void* rows;       // null (the second one only): no branch
     int bf16;               // type of the rows: 0 float32, 1 bfloat16
     const float* bias;      // [W] or null
     int top;                // > 0: the rows are experts' outputs, `top` of them per token
@@ -42,26 +42,48 @@ __device__ __forceinline__ void put_quad(void* p, int bf16, size_t i, float4 v) 
     *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(p) + i) = raw;
 }
 
-__device__ __forceinline__ float4 branch_quad(const Branch& b, int r, int c, int W) {
-    float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+constexpr int QUADS = 4;        // quads of a row per thread in the vector form
+
+// v[i] += the branch at this thread's quads of row r.  Experts' rows come four at a time, all quads of the four at once.
+template <bool BF16>
+__device__ __forceinline__ void add_branch(const Branch& b, int r, int W, float4 (&v)[QUADS]) {
     if (b.top > 0) {
         const size_t first = (size_t)(b.tokens != nullptr ? b.tokens[r] : r) * b.top;
-#pragma unroll 4
-        for (int j = 0; j < b.top; ++j) {
-            const long long row = b.place != nullptr ? b.place[first + j] : (long long)(first + j);
-            if (row < 0) continue;
-            const float w = b.weight != nullptr ? b.weight[first + j] : 1.f;
-            const float4 v = quad(b.rows, b.bf16, (size_t)row * W + c);
-            s.x = fmaf(w, v.x, s.x), s.y = fmaf(w, v.y, s.y), s.z = fmaf(w, v.z, s.z), s.w = fmaf(w, v.w, s.w);
+        for (int j0 = 0; j0 < b.top; j0 += 4) {
+            long long row[4];
+            float w[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const bool in = j0 + j < b.top;
+                row[j] = !in ? -1 : b.place != nullptr ? (long long)b.place[first + j0 + j] : (long long)(first + j0 + j);
+                w[j] = in && b.weight != nullptr ? b.weight[first + j0 + j] : 1.f;
+            }
+#pragma unroll
+            for (int i = 0; i < QUADS; ++i) {
+                const int c = (threadIdx.x + i * blockDim.x) * 4;
+                if (c >= W) break;
+                float4 e[4];
+#pragma unroll
+                for (int j = 0; j < 4; ++j) e[j] = row[j] >= 0 ? quad(b.rows, BF16, (size_t)row[j] * W + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+                    v[i].x = fmaf(w[j], e[j].x, v[i].x), v[i].y = fmaf(w[j], e[j].y, v[i].y), v[i].z = fmaf(w[j], e[j].z, v[i].z),
+                    v[i].w = fmaf(w[j], e[j].w, v[i].w);
+            }
         }
-    } else {
-        s = quad(b.rows, b.bf16, (size_t)r * W + c);
+        return;
     }
-    if (b.bias != nullptr) {
-        const float4 t = *reinterpret_cast<const float4*>(b.bias + c);
-        s = make_float4(s.x + t.x, s.y + t.y, s.z + t.z, s.w + t.w);
+#pragma unroll
+    for (int i = 0; i < QUADS; ++i) {
+        const int c = (threadIdx.x + i * blockDim.x) * 4;
+        if (c >= W) break;
+        float4 s = quad(b.rows, BF16, (size_t)r * W + c);
+        if (b.bias != nullptr) {
+            const float4 t = *reinterpret_cast<const float4*>(b.bias + c);
+            s = make_float4(s.x + t.x, s.y + t.y, s.z + t.z, s.w + t.w);
+        }
+        v[i] = make_float4(v[i].x + s.x, v[i].y + s.y, v[i].z + s.z, v[i].w + s.w);
     }
-    return s;
 }
 
 __device__ __forceinline__ float branch_one(const Branch& b, int r, int c, int W) {
@@ -78,8 +100,6 @@ __device__ __forceinline__ float branch_one(const Branch& b, int r, int c, int W
     return b.bias != nullptr ? s + __ldg(b.bias + c) : s;
 }
 
-constexpr int QUADS = 4;        // quads of a row per thread in the vector form
-
 __global__ void branch_norm_kernel(float* __restrict__ x, Branch a, Branch b, const void* __restrict__ w, int w_bf16, void* __restrict__ y,
                                    int y_bf16, int W, float eps, int vec) {
     __shared__ float red[32];
@@ -94,17 +114,16 @@ __global__ void branch_norm_kernel(float* __restrict__ x, Branch a, Branch b, co
 #pragma unroll
         for (int i = 0; i < QUADS; ++i) {
             const int c = (threadIdx.x + i * blockDim.x) * 4;
-            v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            v[i] = x != nullptr && c < W ? *reinterpret_cast<const float4*>(x + base + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+        if (a.bf16) add_branch<true>(a, r, W, v); else add_branch<false>(a, r, W, v);
+        if (b.rows != nullptr) {
+            if (b.bf16) add_branch<true>(b, r, W, v); else add_branch<false>(b, r, W, v);
+        }
+#pragma unroll
+        for (int i = 0; i < QUADS; ++i) {
+            const int c = (threadIdx.x + i * blockDim.x) * 4;
             if (c < W) {
-                if (x != nullptr) v[i] = *reinterpret_cast<const float4*>(x + base + c);
-                if (a.rows != nullptr) {
-                    const float4 t = branch_quad(a, r, c, W);
-                    v[i] = make_float4(v[i].x + t.x, v[i].y + t.y, v[i].z + t.z, v[i].w + t.w);
-                }
-                if (b.rows != nullptr) {
-                    const float4 t = branch_quad(b, r, c, W);
-                    v[i] = make_float4(v[i].x + t.x, v[i].y + t.y, v[i].z + t.z, v[i].w + t.w);
-                }
                 if (x != nullptr) *reinterpret_cast<float4*>(x + base + c) = v[i];
                 if (w == nullptr && y != nullptr) put_quad(y, y_bf16, base + c, v[i]);
                 ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
@@ -125,7 +144,7 @@ __global__ void branch_norm_kernel(float* __restrict__ x, Branch a, Branch b, co
     float ss = 0.f;
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
         float v = x != nullptr ? x[base + c] : 0.f;
-        if (a.rows != nullptr) v += branch_one(a, r, c, W);
+        v += branch_one(a, r, c, W);
         if (b.rows != nullptr) v += branch_one(b, r, c, W);
         if (x != nullptr) x[base + c] = v;
         if (w == nullptr && y != nullptr) {

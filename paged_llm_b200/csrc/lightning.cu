@@ -13,9 +13,9 @@
 //  * in chunks of LC tokens (bfloat16 prompt portions): what a chunk adds to the state is one product per chunk, the states
 //    at the chunks' starts follow from those by a scan over chunks, and the outputs of a chunk are
 //        o_i = decay^(i+1) S_start^T q_i + sum_{j <= i} decay^(i-j) (q_i . k_j) v_j.
-//    The products run on the tensor cores (mma.sync).  q, k and v are bfloat16 already; every operand that is not (the
-//    state, the decayed keys, the decayed scores) is split into two bfloat16 parts, x = hi + lo, whose products are both
-//    added in float32.
+//    The products run on the tensor cores (mma.sync).  q, k and v are bfloat16 already (silu is applied in place by a kernel
+//    in front); every operand that is not (the state, the decayed values, the decayed scores) is split into two bfloat16
+//    parts, x = hi + lo, whose products are both added in float32.
 #include "common.cuh"
 
 namespace {
@@ -23,7 +23,12 @@ namespace {
 constexpr int LC = 128;         // tokens of a chunk
 constexpr int LH = 64;          // tokens worked on at once
 
-template <typename T> __device__ __forceinline__ float rounded_silu(float x) { return to_float(from_float<T>(silu_f(x))); }
+// silu as the compute type holds it.  Before the rounding to bfloat16 the quick exponential and division are exact enough.
+template <typename T> __device__ __forceinline__ float rounded_silu(float x);
+template <> __device__ __forceinline__ float rounded_silu<float>(float x) { return silu_f(x); }
+template <> __device__ __forceinline__ float rounded_silu<__nv_bfloat16>(float x) {
+    return __bfloat162float(__float2bfloat16_rn(__fdividef(x, 1.0f + __expf(fminf(-x, 80.f)))));
+}
 
 // ------------------------------------------------------------------ token by token
 // grid: (requests, heads, blocks of columns).  LPC lanes share a column, each holding NV float4 of its key channels (lane l:
@@ -177,41 +182,66 @@ __device__ __forceinline__ void split_pair(float x, float y, uint32_t& hi, uint3
     lo = *reinterpret_cast<const uint32_t*>(&r);
 }
 
-// Eight elements of a projection row after silu, as floats (zeros outside); `p` null: zeros.
-__device__ __forceinline__ void silu8(const __nv_bfloat16* p, int left, int vec, float (&v)[8]) {
+// silu of the first n columns of every row, in place.
+__global__ void __launch_bounds__(256) lightning_silu_kernel(__nv_bfloat16* __restrict__ proj, int ld, int n, int rows, int vec) {
+    pdl_launch_dependents();
+    pdl_wait();
+    if (vec) {
+        const int c = (blockIdx.x * 256 + threadIdx.x) * 8;
+        if (c >= n) return;
+        for (int r = blockIdx.y; r < rows; r += gridDim.y) {
+            uint4* p = reinterpret_cast<uint4*>(proj + (size_t)r * ld + c);
+            uint4 raw = *p;
+            __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
 #pragma unroll
-    for (int i = 0; i < 8; ++i) v[i] = 0.f;
-    if (p == nullptr || left <= 0) return;
-    if (vec && left >= 8) {
-        const uint4 raw = *reinterpret_cast<const uint4*>(p);
-        const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
-#pragma unroll
-        for (int i = 0; i < 4; ++i) v[2 * i] = __low2float(h2[i]), v[2 * i + 1] = __high2float(h2[i]);
-    } else {
-#pragma unroll
-        for (int i = 0; i < 8; ++i)
-            if (i < left) v[i] = __bfloat162float(p[i]);
+            for (int i = 0; i < 4; ++i)
+                h[i] = __floats2bfloat162_rn(rounded_silu<__nv_bfloat16>(__low2float(h[i])), rounded_silu<__nv_bfloat16>(__high2float(h[i])));
+            *p = raw;
+        }
+        return;
     }
-#pragma unroll
-    for (int i = 0; i < 8; ++i) v[i] = rounded_silu<__nv_bfloat16>(v[i]);
+    for (int r = blockIdx.y; r < rows; r += gridDim.y)
+        for (int c = blockIdx.x * 256 + threadIdx.x; c < n; c += gridDim.x * 256) {
+            __nv_bfloat16* p = proj + (size_t)r * ld + c;
+            *p = __float2bfloat16_rn(rounded_silu<__nv_bfloat16>(__bfloat162float(*p)));
+        }
 }
 
-__device__ __forceinline__ void store8(__nv_bfloat16* dst, const float (&v)[8]) {
-    __nv_bfloat162 h[4];
-#pragma unroll
-    for (int i = 0; i < 4; ++i) h[i] = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
-    *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<uint4*>(h);
+__device__ __forceinline__ void cp16(__nv_bfloat16* dst, const __nv_bfloat16* src, bool ok) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(ok ? 16 : 0));
+}
+__device__ __forceinline__ void cp_done() {
+    asm volatile("cp.async.commit_group;\n" ::);
+    asm volatile("cp.async.wait_group 0;\n" ::);
 }
 
-// What chunk c adds to the state by its end: buf[number][h][v][n] = sum_j decay^(len-1-j) v_j[v] k_j[n].  grid: (numbers,
+// A tile of `rows` rows and `cols` columns (a multiple of 8) into shared memory with row stride `ds`, zeros behind the first
+// `have_rows` rows and `have_cols` columns.  With `vec` by asynchronous copies of 16 bytes (cp_done), else element by element.
+__device__ __forceinline__ void load_tile(__nv_bfloat16* dst, int ds, const __nv_bfloat16* src, size_t ld, int rows, int cols, int have_rows,
+                                          int have_cols, int vec) {
+    const int units = cols / 8;
+    for (int e = threadIdx.x; e < rows * units; e += 128) {
+        const int r = e / units, c = (e - r * units) * 8;
+        if (vec) {
+            const bool in = r < have_rows && c < have_cols;
+            cp16(dst + r * ds + c, src + (in ? (size_t)r * ld + c : 0), in);
+        } else {
+#pragma unroll
+            for (int i = 0; i < 8; ++i)
+                dst[r * ds + c + i] = r < have_rows && c + i < have_cols ? src[(size_t)r * ld + c + i] : __float2bfloat16_rn(0.f);
+        }
+    }
+}
+
+// What chunk c adds to the state by its end: add[number][h][v][n] = sum_j decay^(len-1-j) v_j[v] k_j[n].  grid: (numbers,
 // heads, tiles of AV values x AK key channels); four warps of 16 values each.
 constexpr int AV = 64, AK = 128;
 
 __global__ void __launch_bounds__(128) lightning_add_kernel(const __nv_bfloat16* __restrict__ proj, int ld, int H, int d, int dv, int dp,
                                                             const float* __restrict__ decay, const int* __restrict__ cu_q,
-                                                            const int* __restrict__ slots, int num_seqs, float* __restrict__ buf,
+                                                            const int* __restrict__ slots, int num_seqs, float* __restrict__ add,
                                                             int vec) {
-    __shared__ __align__(16) __nv_bfloat16 vs[LH][AV + 8], kh[LH][AK + 8], kl[LH][AK + 8];
+    __shared__ __align__(16) __nv_bfloat16 vh[LH][AV + 8], vl[LH][AV + 8], ks[LH][AK + 8];
     __shared__ float pw[LC];
     const ChunkAt at = find_chunk(cu_q, num_seqs, blockIdx.x);
     if (at.s < 0 || slots[at.s] < 0) return;
@@ -219,51 +249,51 @@ __global__ void __launch_bounds__(128) lightning_add_kernel(const __nv_bfloat16*
     const int v0 = (blockIdx.z / ktiles) * AV, n0 = (blockIdx.z % ktiles) * AK;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int len = min(LC, at.nq - at.c * LC);
-    const __nv_bfloat16* base = proj + (size_t)(at.q0 + at.c * LC) * ld;
-    const float dec = __ldg(decay + h);
-    pw[tid] = powf(dec, (float)tid);
-    __syncthreads();
+    const __nv_bfloat16* kb = proj + (size_t)(at.q0 + at.c * LC) * ld + H * d + h * d + n0;
+    const __nv_bfloat16* vb = proj + (size_t)(at.q0 + at.c * LC) * ld + 2 * H * d + h * dv + v0;
+    pw[tid] = powf(__ldg(decay + h), (float)tid);
     float acc[AK / 8][4];
 #pragma unroll
     for (int i = 0; i < AK / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
     for (int t0 = 0; t0 < len; t0 += LH) {
         if (t0 > 0) __syncthreads();
-        for (int e = tid; e < LH * (AV / 8); e += 128) {
+        load_tile(&vh[0][0], AV + 8, vb + (size_t)t0 * ld, ld, LH, AV, len - t0, dv - v0, vec);
+        load_tile(&ks[0][0], AK + 8, kb + (size_t)t0 * ld, ld, LH, AK, len - t0, d - n0, vec);
+        cp_done();
+        __syncthreads();
+        for (int e = tid; e < LH * (AV / 8); e += 128) {                // the values times their decays, in two parts
             const int t = e / (AV / 8), c = (e % (AV / 8)) * 8;
-            float v[8];
-            silu8(t0 + t < len ? base + (size_t)(t0 + t) * ld + 2 * H * d + h * dv + v0 + c : nullptr, dv - v0 - c, vec, v);
-            store8(&vs[t][c], v);
-        }
-        for (int e = tid; e < LH * (AK / 8); e += 128) {
-            const int t = e / (AK / 8), c = (e % (AK / 8)) * 8;
-            float v[8];
-            silu8(t0 + t < len ? base + (size_t)(t0 + t) * ld + H * d + h * d + n0 + c : nullptr, d - n0 - c, vec, v);
             const float f = t0 + t < len ? pw[len - 1 - t0 - t] : 0.f;
-            uint32_t hi[4], lo[4];
+            uint4 hi = *reinterpret_cast<const uint4*>(&vh[t][c]), lo;
+            uint32_t* hw = reinterpret_cast<uint32_t*>(&hi);
+            uint32_t* lw = reinterpret_cast<uint32_t*>(&lo);
 #pragma unroll
-            for (int i = 0; i < 4; ++i) split_pair(v[2 * i] * f, v[2 * i + 1] * f, hi[i], lo[i]);
-            *reinterpret_cast<uint4*>(&kh[t][c]) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-            *reinterpret_cast<uint4*>(&kl[t][c]) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+            for (int i = 0; i < 4; ++i) {
+                const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(hw + i);
+                split_pair(__low2float(x) * f, __high2float(x) * f, hw[i], lw[i]);
+            }
+            *reinterpret_cast<uint4*>(&vh[t][c]) = hi;
+            *reinterpret_cast<uint4*>(&vl[t][c]) = lo;
         }
         __syncthreads();
 #pragma unroll
         for (int k0 = 0; k0 < LH; k0 += 16) {
-            uint32_t a[4];
-            ldm4t(a, &vs[k0 + (lane & 7) + (lane >= 16 ? 8 : 0)][warp * 16 + ((lane >> 3) & 1) * 8]);
+            uint32_t a[4], a2[4];
+            const int ar = k0 + (lane & 7) + (lane >= 16 ? 8 : 0), ac = warp * 16 + ((lane >> 3) & 1) * 8;
+            ldm4t(a, &vh[ar][ac]);
+            ldm4t(a2, &vl[ar][ac]);
 #pragma unroll
             for (int n = 0; n < AK; n += 16) {
-                uint32_t b[4], b2[4];
-                const int r = k0 + (lane & 7) + ((lane >> 3) & 1) * 8, c = n + (lane >= 16 ? 8 : 0);
-                ldm4t(b, &kh[r][c]);
-                ldm4t(b2, &kl[r][c]);
+                uint32_t b[4];
+                ldm4t(b, &ks[k0 + (lane & 7) + ((lane >> 3) & 1) * 8][n + (lane >= 16 ? 8 : 0)]);
                 mma16816(acc[n / 8], a, b[0], b[1]);
                 mma16816(acc[n / 8 + 1], a, b[2], b[3]);
-                mma16816(acc[n / 8], a, b2[0], b2[1]);
-                mma16816(acc[n / 8 + 1], a, b2[2], b2[3]);
+                mma16816(acc[n / 8], a2, b[0], b[1]);
+                mma16816(acc[n / 8 + 1], a2, b[2], b[3]);
             }
         }
     }
-    float* out = buf + ((size_t)blockIdx.x * H + h) * dv * dp;
+    float* out = add + ((size_t)blockIdx.x * H + h) * dv * dp;
 #pragma unroll
     for (int i = 0; i < AK / 8; ++i) {
         const int n = n0 + i * 8 + (lane & 3) * 2, v = v0 + warp * 16 + (lane >> 2);
@@ -273,10 +303,10 @@ __global__ void __launch_bounds__(128) lightning_add_kernel(const __nv_bfloat16*
     }
 }
 
-// The states at the chunks' starts, in place of what the chunks add: four values as four bfloat16 of their upper parts and
-// four of what those leave over.  The state behind the last chunk goes to the request's slot.  A thread per four values.
-__global__ void __launch_bounds__(256) lightning_scan_kernel(float* __restrict__ buf, int H, int d, int dv, int dp,
-                                                             const float* __restrict__ decay, const int* __restrict__ cu_q,
+// The states at the chunks' starts, as two parts of bfloat16: starts[number][h][hi, lo][v][n].  The state behind the last chunk
+// goes to the request's slot.  A thread per four values.
+__global__ void __launch_bounds__(256) lightning_scan_kernel(const float* __restrict__ add, __nv_bfloat16* __restrict__ starts, int H, int d,
+                                                             int dv, int dp, const float* __restrict__ decay, const int* __restrict__ cu_q,
                                                              const int* __restrict__ slots, float* __restrict__ state,
                                                              long long state_stride, int vec) {
     const int s = blockIdx.x, h = blockIdx.y;
@@ -296,24 +326,26 @@ __global__ void __launch_bounds__(256) lightning_scan_kernel(float* __restrict__
     }
     const float dec = __ldg(decay + h), whole = powf(dec, (float)LC);
     const int chunks = (nq + LC - 1) / LC;
-    const size_t step = (size_t)H * dv * dp;
-    float* p = buf + ((size_t)(q0 / LC + s) * H + h) * dv * dp + e;
+    const size_t step = (size_t)H * dv * dp, first = ((size_t)(q0 / LC + s) * H + h) * dv * dp;
+    const float* p = add + first + e;
+    __nv_bfloat16* w = starts + 2 * first + e;
     constexpr int AHEAD = 4;
     for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
-        float4 add[AHEAD];
+        float4 more[AHEAD];
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i)
-            if (c0 + i < chunks) add[i] = *reinterpret_cast<const float4*>(p + (size_t)(c0 + i) * step);
+            if (c0 + i < chunks) more[i] = *reinterpret_cast<const float4*>(p + (size_t)(c0 + i) * step);
 #pragma unroll
         for (int i = 0; i < AHEAD; ++i) {
             const int c = c0 + i;
             if (c >= chunks) break;
-            uint4 parts;
-            split_pair(S[0], S[1], parts.x, parts.z);
-            split_pair(S[2], S[3], parts.y, parts.w);
-            *reinterpret_cast<uint4*>(p + (size_t)c * step) = parts;
+            uint2 hi, lo;
+            split_pair(S[0], S[1], hi.x, lo.x);
+            split_pair(S[2], S[3], hi.y, lo.y);
+            *reinterpret_cast<uint2*>(w + 2 * (size_t)c * step) = hi;
+            *reinterpret_cast<uint2*>(w + 2 * (size_t)c * step + (size_t)dv * dp) = lo;
             const float f = c + 1 < chunks ? whole : powf(dec, (float)(nq - c * LC));
-            S[0] = fmaf(f, S[0], add[i].x), S[1] = fmaf(f, S[1], add[i].y), S[2] = fmaf(f, S[2], add[i].z), S[3] = fmaf(f, S[3], add[i].w);
+            S[0] = fmaf(f, S[0], more[i].x), S[1] = fmaf(f, S[1], more[i].y), S[2] = fmaf(f, S[2], more[i].z), S[3] = fmaf(f, S[3], more[i].w);
         }
     }
     if (vec && n < d) {
@@ -327,17 +359,17 @@ __global__ void __launch_bounds__(256) lightning_scan_kernel(float* __restrict__
 
 // The outputs of LH tokens of a chunk.  grid: (2 * numbers, heads, tiles of CV values); four warps of 16 tokens each.
 // Shared memory: q [LH][dp + 8], then either the start state's parts [2][CV][dp + 8] or k [LH][dp + 8] and v [LH][CV + 8].
-constexpr int CV = 128;
+constexpr int CV = 64;
 
 __host__ __device__ constexpr size_t lightning_out_smem(int dp) {
     const size_t st = (size_t)2 * CV * (dp + 8), kv = (size_t)LH * (dp + 8) + (size_t)LH * (CV + 8);
     return ((size_t)LH * (dp + 8) + (st > kv ? st : kv)) * 2;
 }
 
-__global__ void __launch_bounds__(128) lightning_out_kernel(const __nv_bfloat16* __restrict__ proj, int ld, int H, int d, int dv, int dp,
-                                                            const float* __restrict__ decay, const int* __restrict__ cu_q,
-                                                            const int* __restrict__ slots, int num_seqs, const float* __restrict__ buf,
-                                                            float* __restrict__ o, int vec) {
+__global__ void __launch_bounds__(128, 4) lightning_out_kernel(const __nv_bfloat16* __restrict__ proj, int ld, int H, int d, int dv, int dp,
+                                                               const float* __restrict__ decay, const int* __restrict__ cu_q,
+                                                               const int* __restrict__ slots, int num_seqs,
+                                                               const __nv_bfloat16* __restrict__ starts, float* __restrict__ o, int vec) {
     extern __shared__ __align__(16) __nv_bfloat16 smem[];
     __shared__ float pw[LC + 1];
     const int number = blockIdx.x >> 1, half = blockIdx.x & 1;
@@ -348,34 +380,26 @@ __global__ void __launch_bounds__(128) lightning_out_kernel(const __nv_bfloat16*
     if (i0 >= len) return;
     const int h = blockIdx.y, v0 = blockIdx.z * CV;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int row = dp + 8, units = dp / 8;
+    const int row = dp + 8;
     __nv_bfloat16* qs = smem;
     __nv_bfloat16* sh = smem + LH * row;
     __nv_bfloat16* sl = sh + CV * row;
     __nv_bfloat16* ks = smem + LH * row;
     __nv_bfloat16* vs = ks + LH * row;
     const __nv_bfloat16* base = proj + (size_t)(at.q0 + at.c * LC) * ld;
+    const __nv_bfloat16* start = starts + 2 * (((size_t)number * H + h) * dv * dp) + (size_t)v0 * dp;
+    load_tile(qs, row, base + (size_t)i0 * ld + h * d, ld, LH, dp, len - i0, d, vec);
+    load_tile(sh, row, start, dp, CV, dp, dv - v0, dp, 1);
+    load_tile(sl, row, start + (size_t)dv * dp, dp, CV, dp, dv - v0, dp, 1);
     const float dec = __ldg(decay + h);
     for (int i = tid; i <= LC; i += 128) pw[i] = powf(dec, (float)i);
-    for (int e = tid; e < LH * units; e += 128) {
-        const int t = e / units, c = (e - t * units) * 8;
-        float v[8];
-        silu8(i0 + t < len ? base + (size_t)(i0 + t) * ld + h * d + c : nullptr, d - c, vec, v);
-        store8(qs + t * row + c, v);
-    }
-    const float* start = buf + ((size_t)number * H + h) * dv * dp;
-    for (int e = tid; e < CV * (dp / 4); e += 128) {
-        const int v = e / (dp / 4), n = (e - v * (dp / 4)) * 4;
-        uint4 parts = make_uint4(0, 0, 0, 0);
-        if (v0 + v < dv) parts = *reinterpret_cast<const uint4*>(start + (size_t)(v0 + v) * dp + n);
-        *reinterpret_cast<uint2*>(sh + v * row + n) = make_uint2(parts.x, parts.y);
-        *reinterpret_cast<uint2*>(sl + v * row + n) = make_uint2(parts.z, parts.w);
-    }
+    cp_done();
     __syncthreads();
     float acc[CV / 8][4];
 #pragma unroll
     for (int i = 0; i < CV / 8; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
     const __nv_bfloat16* qa = qs + (warp * 16 + (lane & 15)) * row + (lane >> 4) * 8;        // rows of A: this warp's tokens
+#pragma unroll 2
     for (int k0 = 0; k0 < dp; k0 += 16) {
         uint32_t a[4];
         ldm4(a, qa + k0);
@@ -400,24 +424,16 @@ __global__ void __launch_bounds__(128) lightning_out_kernel(const __nv_bfloat16*
     }
     for (int j0 = 0; j0 <= i0; j0 += LH) {
         __syncthreads();                                                // the state (or the keys in front) has been read
-        for (int e = tid; e < LH * units; e += 128) {
-            const int t = e / units, c = (e - t * units) * 8;
-            float v[8];
-            silu8(j0 + t < len ? base + (size_t)(j0 + t) * ld + H * d + h * d + c : nullptr, d - c, vec, v);
-            store8(ks + t * row + c, v);
-        }
-        for (int e = tid; e < LH * (CV / 8); e += 128) {
-            const int t = e / (CV / 8), c = (e % (CV / 8)) * 8;
-            float v[8];
-            silu8(j0 + t < len ? base + (size_t)(j0 + t) * ld + 2 * H * d + h * dv + v0 + c : nullptr, dv - v0 - c, vec, v);
-            store8(vs + t * (CV + 8) + c, v);
-        }
+        load_tile(ks, row, base + (size_t)j0 * ld + H * d + h * d, ld, LH, dp, len - j0, d, vec);
+        load_tile(vs, CV + 8, base + (size_t)j0 * ld + 2 * H * d + h * dv + v0, ld, LH, CV, len - j0, dv - v0, vec);
+        cp_done();
         __syncthreads();
         // the keys that this warp's tokens see: all of an earlier half, else those up to the warp's last token
         const int keys = j0 < i0 ? LH : warp * 16 + 16;
         float sc[LH / 8][4];
 #pragma unroll
         for (int i = 0; i < LH / 8; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.f;
+#pragma unroll 2
         for (int k0 = 0; k0 < dp; k0 += 16) {
             uint32_t a[4];
             ldm4(a, qa + k0);
@@ -568,24 +584,31 @@ PL_EXPORT int pl_lightning_step(const void* proj, int dtype, int ld, int H, int 
     return pl_fail("lightning_step: unknown dtype %d", dtype);
 }
 
-// In chunks (bfloat16): `buf` holds total_tokens / pl_lightning_chunk() + num_seqs chunks of H * dv * pad16(d) floats.
+// In chunks (bfloat16): `numbers` = total_tokens / pl_lightning_chunk() + num_seqs; `buf` holds twice numbers * H * dv * pad16(d)
+// floats.  The first 2 * H * d + H * dv columns of proj's `rows` rows are overwritten by their silu.
 PL_EXPORT int pl_lightning_chunk() { return LC; }
 
-PL_EXPORT int pl_lightning_chunks(const void* proj, int ld, int H, int d, int dv, const float* decay, float* buf, int numbers,
+PL_EXPORT int pl_lightning_chunks(void* proj_, int ld, int rows, int H, int d, int dv, const float* decay, float* buf, int numbers,
                                   float* state, long long state_stride, const int* cu_q, const int* slots, int num_seqs, float* o,
                                   cudaStream_t stream) {
-    if (num_seqs == 0 || numbers == 0) return 0;
-    PL_REQUIRE(H > 0 && H <= 65535 && d > 0 && d <= 256 && dv > 0 && dv <= 8192 && ld >= 2 * H * d + H * dv && numbers > 0 &&
+    if (num_seqs == 0 || numbers == 0 || rows == 0) return 0;
+    PL_REQUIRE(H > 0 && H <= 65535 && d > 0 && d <= 256 && dv > 0 && dv <= 8192 && ld >= 2 * H * d + H * dv && numbers > 0 && rows > 0 &&
                    state_stride >= (long long)H * d * dv,
                "lightning_chunks: bad sizes H=%d d=%d dv=%d ld=%d (key size at most 256)", H, d, dv, ld);
-    const int dp = (d + 15) / 16 * 16;
-    const int vec = ld % 8 == 0 && d % 8 == 0 && dv % 8 == 0 && ((uintptr_t)proj & 15) == 0;
+    __nv_bfloat16* proj = (__nv_bfloat16*)proj_;
+    const int dp = (d + 15) / 16 * 16, n = 2 * H * d + H * dv;
+    const int vec = ld % 8 == 0 && d % 8 == 0 && dv % 8 == 0 && ((uintptr_t)proj & 15) == 0 && ((uintptr_t)buf & 15) == 0;
     const int vec_state = d % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state & 15) == 0;
+    PL_REQUIRE(((uintptr_t)buf & 15) == 0, "lightning_chunks: the scratch is not 16-byte aligned");
+    float* add = buf;
+    __nv_bfloat16* starts = (__nv_bfloat16*)(buf + (size_t)numbers * H * dv * dp);
+    const dim3 grid_s((n / (vec ? 8 : 1) + 255) / 256, rows < 65535 ? rows : 65535);
+    PL_CUDA(launch_pdl(lightning_silu_kernel, grid_s, dim3(256), 0, stream, proj, ld, n, rows, vec));
     const dim3 grid_a(numbers, H, (dv + AV - 1) / AV * ((dp + AK - 1) / AK));
-    lightning_add_kernel<<<grid_a, 128, 0, stream>>>((const __nv_bfloat16*)proj, ld, H, d, dv, dp, decay, cu_q, slots, num_seqs, buf, vec);
+    lightning_add_kernel<<<grid_a, 128, 0, stream>>>(proj, ld, H, d, dv, dp, decay, cu_q, slots, num_seqs, add, vec);
     PL_LAUNCHED("lightning_add");
     const dim3 grid_b(num_seqs, H, (dv * dp / 4 + 255) / 256);
-    lightning_scan_kernel<<<grid_b, 256, 0, stream>>>(buf, H, d, dv, dp, decay, cu_q, slots, state, state_stride, vec_state);
+    lightning_scan_kernel<<<grid_b, 256, 0, stream>>>(add, starts, H, d, dv, dp, decay, cu_q, slots, state, state_stride, vec_state);
     PL_LAUNCHED("lightning_scan");
     const size_t smem = lightning_out_smem(dp);
     static bool opted[64] = {};
@@ -597,8 +620,7 @@ PL_EXPORT int pl_lightning_chunks(const void* proj, int ld, int H, int d, int dv
         opted[dev] = true;
     }
     const dim3 grid_c(2 * numbers, H, (dv + CV - 1) / CV);
-    lightning_out_kernel<<<grid_c, 128, smem, stream>>>((const __nv_bfloat16*)proj, ld, H, d, dv, dp, decay, cu_q, slots, num_seqs, buf, o,
-                                                        vec);
+    lightning_out_kernel<<<grid_c, 128, smem, stream>>>(proj, ld, H, d, dv, dp, decay, cu_q, slots, num_seqs, starts, o, vec);
     PL_LAUNCHED("lightning_out");
     return 0;
 }

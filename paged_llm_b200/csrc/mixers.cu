@@ -361,11 +361,107 @@ PL_EXPORT int pl_normed_qkv_write(const void* proj, int dtype, int T, int ld, co
 // [d] if there is one (qw, kw: one for all heads); with a table `rot`, q and k are then rotated by the token's position over
 // the table's leading elements of each head.  Q out [T, nh*D], K and V to the page slot, all padded to D with zeros.  A warp
 // per (token, head): heads 0..nh-1 are queries, then keys, then values.
+// Vector form: sizes are multiples of 4, a lane holds NQ quads of a head (D <= 128 NQ), a warp takes HP heads of a token whose
+// loads go out together; the rotation's quads do not straddle its halves.
+__device__ __forceinline__ float4 shfl_quad(float4 v, int lane) {
+    return make_float4(__shfl_sync(0xffffffffu, v.x, lane), __shfl_sync(0xffffffffu, v.y, lane), __shfl_sync(0xffffffffu, v.z, lane),
+                       __shfl_sync(0xffffffffu, v.w, lane));
+}
+
+// The quads of a head (lane l: quads l, l + 32) after the rotation in halves; a quad's partner sits in another lane or in this
+// lane's other quad.  Called by whole warps.
+template <int NQ>
+__device__ __forceinline__ void turn_quads(const float2* cs, int rd, int lane, float4 (&v)[NQ]) {
+    float4 other[NQ];
+    const int hq = rd >> 3;                                             // quads of half the rotated elements
+#pragma unroll
+    for (int i = 0; i < NQ; ++i) {
+        const int quad = lane + 32 * i;
+        const int pq = quad >= 2 * hq ? quad : quad >= hq ? quad - hq : quad + hq;
+        other[i] = shfl_quad(v[0], pq & 31);
+        if (NQ > 1) {
+            const float4 b = shfl_quad(v[NQ - 1], pq & 31);
+            if (pq >= 32) other[i] = b;
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < NQ; ++i) v[i] = turned_quad(cs, rd, (lane + 32 * i) * 4, v[i], other[i]);
+}
+
+template <typename T, int NQ, int HP>
+__global__ void __launch_bounds__(256) unit_qkv_quads_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ bias, float eps,
+                                                             const float* __restrict__ qw, const float* __restrict__ kw, RotTable rot,
+                                                             T* __restrict__ q_out, T* __restrict__ kv, SlotArgs sa, int nh, int nkv, int d,
+                                                             int dv, int D, int write, long long items) {
+    pdl_launch_dependents();
+    const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (item >= items) {
+        pdl_wait();
+        return;
+    }
+    const int lane = threadIdx.x & 31, heads = nh + 2 * nkv, groups = (heads + HP - 1) / HP;
+    const int t = (int)(item / groups), head0 = (int)(item - (long long)t * groups) * HP;
+    const int s = sa.token_seq[t], pos = sa.positions[t];
+    const long long slot = write && s >= 0 ? key_slot(sa, t, s, pos, nkv, D) : -1;
+    const float2* cs = rot.table != nullptr && s >= 0 && pos >= 0 && pos < rot.len ? rot.table + (size_t)pos * (rot.rd >> 1) : nullptr;
+    pdl_wait();
+    const T* row = proj + (size_t)t * ld;
+    float4 v[HP][NQ];
+#pragma unroll
+    for (int p = 0; p < HP; ++p) {
+        const int head = head0 + p;
+        const bool is_v = head >= nh + nkv;
+        const int n = head >= heads || s < 0 ? 0 : is_v ? dv : d, col = is_v ? (nh + nkv) * d + (head - nh - nkv) * dv : head * d;
+#pragma unroll
+        for (int i = 0; i < NQ; ++i) {
+            const int c = (lane + 32 * i) * 4;
+            v[p][i] = c < n ? Quad4<T>::load(row + col + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            if (bias != nullptr && c < n) {
+                const float4 b = Quad4<float>::load(bias + col + c);
+                v[p][i] = make_float4(v[p][i].x + b.x, v[p][i].y + b.y, v[p][i].z + b.z, v[p][i].w + b.w);
+            }
+        }
+    }
+#pragma unroll
+    for (int p = 0; p < HP; ++p) {
+        const int head = head0 + p;
+        if (head >= heads) break;
+        const bool is_q = head < nh, is_v = head >= nh + nkv;
+        float f = 1.f;
+        if (!is_v) {
+            const float* hw = is_q ? qw : kw;
+            float sq = 0.f;
+#pragma unroll
+            for (int i = 0; i < NQ; ++i) {
+                float4& x = v[p][i];
+                sq += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+                const int c = (lane + 32 * i) * 4;
+                if (hw != nullptr && c < d) {
+                    const float4 w = Quad4<float>::load(hw + c);
+                    x = make_float4(x.x * w.x, x.y * w.y, x.z * w.z, x.w * w.w);
+                }
+            }
+            f = 1.0f / sqrtf(warp_sum(sq) / (float)d + eps);
+            if (cs != nullptr) turn_quads<NQ>(cs, rot.rd, lane, v[p]);
+        }
+        T* dst = is_q ? q_out + ((size_t)t * nh + head) * D
+                 : slot >= 0 ? kv + slot + (size_t)(is_v ? head - nkv - nh : head - nh) * sa.ps * D + (is_v ? (size_t)nkv * sa.ps * D : 0) : nullptr;
+        if (dst == nullptr) continue;
+#pragma unroll
+        for (int i = 0; i < NQ; ++i) {
+            const int c = (lane + 32 * i) * 4;
+            const float4 x = v[p][i];
+            if (c < D) Quad4<T>::store(dst + c, make_float4(x.x * f, x.y * f, x.z * f, x.w * f));
+        }
+    }
+}
+
+// Any sizes: a warp per (token, head), element by element.
 template <typename T>
 __global__ void __launch_bounds__(256) unit_qkv_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ bias, float eps,
                                                        const float* __restrict__ qw, const float* __restrict__ kw, RotTable rot,
                                                        T* __restrict__ q_out, T* __restrict__ kv, SlotArgs sa, int nh, int nkv, int d,
-                                                       int dv, int D, int write, int vec, long long items) {
+                                                       int dv, int D, int write, long long items) {
     pdl_launch_dependents();
     const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
     if (item >= items) {
@@ -391,44 +487,6 @@ __global__ void __launch_bounds__(256) unit_qkv_kernel(const T* __restrict__ pro
     if (dst == nullptr) return;
     const T* src = proj + (size_t)t * ld + col;
     const float* b = bias != nullptr ? bias + col : nullptr;
-    if (vec) {
-        // d, dv and D are multiples of 4 up to 256: a lane holds two quads of the head (rotation: quads do not straddle)
-        float4 v[2];
-        float sq = 0.f;
-        auto biased = [&](int c) {
-            float4 x = Quad4<T>::load(src + c);
-            if (b != nullptr) {
-                const float4 w = Quad4<float>::load(b + c);
-                x = make_float4(x.x + w.x, x.y + w.y, x.z + w.z, x.w + w.w);
-            }
-            return x;
-        };
-        auto weighted = [&](float4 x, int c) {
-            if (hw == nullptr) return x;
-            const float4 w = Quad4<float>::load(hw + c);
-            return make_float4(x.x * w.x, x.y * w.y, x.z * w.z, x.w * w.w);
-        };
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            const int c = (lane + 32 * i) * 4;
-            v[i] = c < n && s >= 0 ? biased(c) : make_float4(0.f, 0.f, 0.f, 0.f);
-            sq += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
-            if (c < n && s >= 0) {
-                v[i] = weighted(v[i], c);
-                if (cs != nullptr && c < rot.rd) {
-                    const int other = c >= (rot.rd >> 1) ? c - (rot.rd >> 1) : c + (rot.rd >> 1);
-                    v[i] = turned_quad(cs, rot.rd, c, v[i], weighted(biased(other), other));
-                }
-            }
-        }
-        const float f = is_v ? 1.f : 1.0f / sqrtf(warp_sum(sq) / (float)d + eps);
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            const int c = (lane + 32 * i) * 4;
-            if (c < D) Quad4<T>::store(dst + c, make_float4(v[i].x * f, v[i].y * f, v[i].z * f, v[i].w * f));
-        }
-        return;
-    }
     auto value = [&](int c) { return c < n && s >= 0 ? to_float(src[c]) + (b != nullptr ? __ldg(b + c) : 0.f) : 0.f; };
     float sq = 0.f;
     for (int c = lane; c < n; c += 32) {
@@ -440,6 +498,28 @@ __global__ void __launch_bounds__(256) unit_qkv_kernel(const T* __restrict__ pro
     for (int c = lane; c < D; c += 32) dst[c] = from_float<T>(turned(cs, rot.rd, rot.inter, 1.f, c, weighted) * f);
 }
 
+template <typename T>
+static int launch_unit_qkv(const void* proj, int T_, int ld, const float* bias, float eps, const float* qw, const float* kw, RotTable rot,
+                           void* q_out, void* kv, SlotArgs sa, int nh, int nkv, int d, int dv, int D, int write, int vec,
+                           cudaStream_t stream) {
+    const int heads = nh + 2 * nkv, hp = vec && T_ >= 256 ? (D <= 128 ? 4 : 2) : 1;
+    const long long items = (long long)T_ * ((heads + hp - 1) / hp), blocks = (items + 7) / 8;
+    PL_REQUIRE(blocks < (1ll << 31), "unit_qkv_write: %d tokens", T_);
+#define UNIT_QUADS(NQ, HP)                                                                                                              \
+    PL_CUDA(launch_pdl(unit_qkv_quads_kernel<T, NQ, HP>, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)proj, ld, bias, eps, qw, kw, rot, \
+                       (T*)q_out, (T*)kv, sa, nh, nkv, d, dv, D, write, items))
+    if (!vec)
+        PL_CUDA(launch_pdl(unit_qkv_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)proj, ld, bias, eps, qw, kw, rot,
+                           (T*)q_out, (T*)kv, sa, nh, nkv, d, dv, D, write, items));
+    else if (D <= 128) {
+        if (hp == 4) UNIT_QUADS(1, 4); else UNIT_QUADS(1, 1);
+    } else {
+        if (hp == 2) UNIT_QUADS(2, 2); else UNIT_QUADS(2, 1);
+    }
+#undef UNIT_QUADS
+    return 0;
+}
+
 PL_EXPORT int pl_unit_qkv_write(const void* proj, int dtype, int T, int ld, const float* bias, float eps, const float* qw,
                                 const float* kw, const float* rot_table, int rot_len, int rot_rd, int rot_inter, void* q_out, void* kv,
                                 const int* positions, const int* token_seq, const int* block_table, int bt_stride, int num_pages,
@@ -448,8 +528,6 @@ PL_EXPORT int pl_unit_qkv_write(const void* proj, int dtype, int T, int ld, cons
     PL_REQUIRE(T > 0 && nh > 0 && nkv > 0 && d > 0 && dv > 0 && D >= d && D >= dv && ps > 0 && ld >= nh * d + nkv * (d + dv),
                "unit_qkv_write: bad sizes d=%d dv=%d D=%d ld=%d", d, dv, D, ld);
     SlotArgs sa{positions, token_seq, block_table, bt_stride, num_pages, ps};
-    const long long items = (long long)T * (nh + 2 * nkv), blocks = (items + 7) / 8;
-    PL_REQUIRE(blocks < (1ll << 31), "unit_qkv_write: %d tokens", T);
     PL_REQUIRE(rot_table == nullptr || (rot_rd > 0 && rot_rd % 2 == 0 && rot_rd <= d), "unit_qkv_write: %d rotated elements of %d", rot_rd, d);
     const RotTable rot{(const float2*)rot_table, rot_len, rot_rd, rot_inter};
     const int vec = d % 4 == 0 && dv % 4 == 0 && D % 4 == 0 && D <= 256 && ld % 4 == 0 &&
@@ -457,14 +535,10 @@ PL_EXPORT int pl_unit_qkv_write(const void* proj, int dtype, int T, int ld, cons
                     (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)kv | (uintptr_t)bias | (uintptr_t)qw | (uintptr_t)kw |
                       (uintptr_t)rot_table) & 15) == 0;
     if (dtype == PL_F32)
-        PL_CUDA(launch_pdl(unit_qkv_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, (const float*)proj, ld, bias, eps, qw, kw, rot,
-                           (float*)q_out, (float*)kv, sa, nh, nkv, d, dv, D, write, vec, items));
-    else if (dtype == PL_BF16)
-        PL_CUDA(launch_pdl(unit_qkv_kernel<__nv_bfloat16>, dim3((unsigned)blocks), dim3(256), 0, stream, (const __nv_bfloat16*)proj, ld,
-                           bias, eps, qw, kw, rot, (__nv_bfloat16*)q_out, (__nv_bfloat16*)kv, sa, nh, nkv, d, dv, D, write, vec, items));
-    else
-        return pl_fail("unit_qkv_write: unknown dtype %d", dtype);
-    return 0;
+        return launch_unit_qkv<float>(proj, T, ld, bias, eps, qw, kw, rot, q_out, kv, sa, nh, nkv, d, dv, D, write, vec, stream);
+    if (dtype == PL_BF16)
+        return launch_unit_qkv<__nv_bfloat16>(proj, T, ld, bias, eps, qw, kw, rot, q_out, kv, sa, nh, nkv, d, dv, D, write, vec, stream);
+    return pl_fail("unit_qkv_write: unknown dtype %d", dtype);
 }
 
 // ------------------------------------------------------------------ short convolution + rotation + cache write
@@ -525,23 +599,7 @@ __global__ void __launch_bounds__(256) conv_qkv_kernel(const T* __restrict__ pro
                         }
                     }
                 }
-                if (cs != nullptr) {
-                    // a quad's partner sits in another lane (or this lane's other quad)
-                    float4 other[2];
-#pragma unroll
-                    for (int i = 0; i < 2; ++i) {
-                        const int quad = lane + 32 * i, hq = rot.rd >> 3;
-                        const int pq = quad >= 2 * hq ? quad : quad >= hq ? quad - hq : quad + hq;
-                        float4 a, b;
-                        a.x = __shfl_sync(0xffffffffu, v[0].x, pq & 31), b.x = __shfl_sync(0xffffffffu, v[1].x, pq & 31);
-                        a.y = __shfl_sync(0xffffffffu, v[0].y, pq & 31), b.y = __shfl_sync(0xffffffffu, v[1].y, pq & 31);
-                        a.z = __shfl_sync(0xffffffffu, v[0].z, pq & 31), b.z = __shfl_sync(0xffffffffu, v[1].z, pq & 31);
-                        a.w = __shfl_sync(0xffffffffu, v[0].w, pq & 31), b.w = __shfl_sync(0xffffffffu, v[1].w, pq & 31);
-                        other[i] = pq >= 32 ? b : a;
-                    }
-#pragma unroll
-                    for (int i = 0; i < 2; ++i) v[i] = turned_quad(cs, rot.rd, (lane + 32 * i) * 4, v[i], other[i]);
-                }
+                if (cs != nullptr) turn_quads<2>(cs, rot.rd, lane, v);
                 if (dst == nullptr) continue;
 #pragma unroll
                 for (int i = 0; i < 2; ++i) {
@@ -574,6 +632,93 @@ __global__ void __launch_bounds__(256) conv_qkv_kernel(const T* __restrict__ pro
     }
 }
 
+// The same for portions of many tokens, up to four taps and heads of at most 128 elements in quads: a warp takes QC_STRIP
+// consecutive tokens of a head, whose inputs (and the TAPS - 1 in front) it loads together.
+constexpr int QC_STRIP = 8;
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256) conv_qkv_strip_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ cw,
+                                                             float* __restrict__ state, long long state_stride, const int* __restrict__ cu_q,
+                                                             const int* __restrict__ slots, RotTable rot, T* __restrict__ q_out,
+                                                             T* __restrict__ kv, SlotArgs sa, int nh, int nkv, int d, int dv, int D, int write) {
+    static_assert(QC_STRIP * 8 == QC_TOK, "eight warps cover a chunk");
+    pdl_launch_dependents();
+    constexpr int hist = TAPS - 1;
+    const int s = blockIdx.x, head = blockIdx.y, C = nh * d + nkv * (d + dv);
+    const int q0 = cu_q[s], nq = cu_q[s + 1] - q0, slot = hist > 0 ? slots[s] : 0;
+    const int t_lo = blockIdx.z * QC_TOK, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, c = lane * 4;
+    const bool is_q = head < nh, is_v = head >= nh + nkv;
+    const int n = is_v ? dv : d, col = is_v ? (nh + nkv) * d + (head - nh - nkv) * dv : head * d;
+    float4 f[TAPS];
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k)
+        f[k] = c < n ? *reinterpret_cast<const float4*>(cw + (size_t)k * C + col + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    pdl_wait();
+    if (slot < 0 || t_lo >= nq) return;
+    float* st = hist > 0 ? state + (size_t)slot * state_stride + col : nullptr;
+    const T* in = proj + (size_t)q0 * ld + col;
+    const int t0 = t_lo + warp * QC_STRIP;
+    if (t0 < nq) {
+        float4 u[QC_STRIP + hist];
+#pragma unroll
+        for (int r = 0; r < QC_STRIP + hist; ++r) {
+            const int src = t0 - hist + r;
+            u[r] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (c < n && src < nq)
+                u[r] = src >= 0 ? Quad4<T>::load(in + (size_t)src * ld + c) : *reinterpret_cast<const float4*>(st + (size_t)(hist + src) * C + c);
+        }
+        const int pos0 = sa.positions[q0 + t0];                         // (a request's tokens stand at consecutive positions)
+        T* dst[QC_STRIP];
+#pragma unroll
+        for (int i = 0; i < QC_STRIP; ++i) {
+            dst[i] = nullptr;
+            if (t0 + i >= nq) continue;
+            if (is_q) {
+                dst[i] = q_out + ((size_t)(q0 + t0 + i) * nh + head) * D;
+            } else if (write) {
+                const long long at = key_slot(sa, q0 + t0 + i, s, pos0 + i, nkv, D);
+                if (at >= 0) dst[i] = kv + at + (size_t)(is_v ? head - nkv - nh : head - nh) * sa.ps * D + (is_v ? (size_t)nkv * sa.ps * D : 0);
+            }
+        }
+#pragma unroll
+        for (int i = 0; i < QC_STRIP; ++i) {
+            if (t0 + i >= nq) break;
+            float4 v[1] = {make_float4(0.f, 0.f, 0.f, 0.f)};
+#pragma unroll
+            for (int k = 0; k < TAPS; ++k)
+                v[0].x = fmaf(f[k].x, u[i + k].x, v[0].x), v[0].y = fmaf(f[k].y, u[i + k].y, v[0].y),
+                v[0].z = fmaf(f[k].z, u[i + k].z, v[0].z), v[0].w = fmaf(f[k].w, u[i + k].w, v[0].w);
+            const int pos = pos0 + i;
+            if (!is_v && rot.table != nullptr && pos >= 0 && pos < rot.len)
+                turn_quads<1>(rot.table + (size_t)pos * (rot.rd >> 1), rot.rd, lane, v);
+            if (dst[i] != nullptr && c < D) Quad4<T>::store(dst[i] + c, v[0]);
+        }
+    }
+    if (blockIdx.z != 0 || hist == 0) return;
+    __syncthreads();                                                    // every read of the old inputs is done
+    if (warp == 0)
+        for (int e = lane; e < n; e += 32)
+            for (int j = 0; j < hist; ++j) {                            // (in place from the front, as above)
+                const int src = nq + j - hist;
+                st[(size_t)j * C + e] = src >= 0 ? to_float(in[(size_t)src * ld + e]) : st[(size_t)(j + nq) * C + e];
+            }
+}
+
+template <typename T>
+static int launch_conv_strip(const void* proj, int ld, const float* cw, int taps, float* state, long long state_stride, const int* cu_q,
+                             const int* slots, RotTable rot, void* q_out, void* kv, SlotArgs sa, int nh, int nkv, int d, int dv, int D,
+                             int write, dim3 grid, cudaStream_t stream) {
+#define STRIP(N)                                                                                                                   \
+    PL_CUDA(launch_pdl(conv_qkv_strip_kernel<T, N>, grid, dim3(256), 0, stream, (const T*)proj, ld, cw, state, state_stride, cu_q, \
+                       slots, rot, (T*)q_out, (T*)kv, sa, nh, nkv, d, dv, D, write))
+    if (taps == 1) STRIP(1);
+    else if (taps == 2) STRIP(2);
+    else if (taps == 3) STRIP(3);
+    else STRIP(4);
+#undef STRIP
+    return 0;
+}
+
 // `max_tokens`: no request of the step brings more.  state null: one tap, nothing to keep.
 PL_EXPORT int pl_conv_qkv_write(const void* proj, int dtype, int ld, const float* cw, int taps, float* state, long long state_stride,
                                 const int* cu_q, const int* slots, int num_seqs, int max_tokens, const float* rot_table, int rot_len,
@@ -595,14 +740,20 @@ PL_EXPORT int pl_conv_qkv_write(const void* proj, int dtype, int ld, const float
     const int wh = max_tokens >= 8 ? 1 : max_tokens >= 4 ? 2 : max_tokens >= 2 ? 4 : 8;
     const dim3 grid(num_seqs, (nh + 2 * nkv + wh - 1) / wh, (max_tokens + QC_TOK - 1) / QC_TOK);
     PL_REQUIRE(grid.y <= 65535 && grid.z <= 65535, "conv_qkv_write: %d tokens, %d heads in a step", max_tokens, nh);
+    PL_REQUIRE(dtype == PL_F32 || dtype == PL_BF16, "conv_qkv_write: unknown dtype %d", dtype);
+    if (wh == 1 && vec && taps <= 4 && D <= 128) {
+        if (dtype == PL_F32)
+            return launch_conv_strip<float>(proj, ld, cw, taps, state, state_stride, cu_q, slots, rot, q_out, kv, sa, nh, nkv, d, dv, D, write,
+                                            grid, stream);
+        return launch_conv_strip<__nv_bfloat16>(proj, ld, cw, taps, state, state_stride, cu_q, slots, rot, q_out, kv, sa, nh, nkv, d, dv, D,
+                                                write, grid, stream);
+    }
     if (dtype == PL_F32)
         PL_CUDA(launch_pdl(conv_qkv_kernel<float>, grid, dim3(256), 0, stream, (const float*)proj, ld, cw, taps, state, state_stride, cu_q,
                            slots, rot, (float*)q_out, (float*)kv, sa, nh, nkv, d, dv, D, write, wh, vec));
-    else if (dtype == PL_BF16)
+    else
         PL_CUDA(launch_pdl(conv_qkv_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)proj, ld, cw, taps, state,
                            state_stride, cu_q, slots, rot, (__nv_bfloat16*)q_out, (__nv_bfloat16*)kv, sa, nh, nkv, d, dv, D, write, wh, vec));
-    else
-        return pl_fail("conv_qkv_write: unknown dtype %d", dtype);
     return 0;
 }
 

@@ -1058,8 +1058,8 @@ class CudaOps:
         """Linear attention with a fixed decay per head.  proj rows [q: H*d | k: H*d | v: H*dv | ...], each through silu;
         S_t = decay[h] S_(t-1) + k_t v_t^T, o_t = S_t^T q_t (`decay` float32 [H]).  state: [slots, H*dv*d] float32 (a head's columns
         one after the other), updated in place.  Returns o float32 [T, H*dv].  A step of few tokens per request, and float32, run
-        token by token in one kernel; longer portions in chunks on the tensor cores: what every chunk adds to the state, the
-        states at the chunks' starts, the outputs."""
+        token by token in one kernel; longer portions in chunks on the tensor cores: silu in place on proj's columns, what every
+        chunk adds to the state, the states at the chunks' starts, the outputs."""
         lib = load_module("lightning")
         T, ld = proj.shape
         assert proj.is_contiguous() and decay.dtype == torch.float32 and decay.numel() == H
@@ -1072,11 +1072,11 @@ class CudaOps:
             self.launches += 1
             return o
         numbers = T // lib.pl_lightning_chunk() + ctx.num_seqs
-        buf = torch.empty(numbers * H * dv * (-(-d // 16) * 16), dtype=torch.float32, device=self.device)
-        _check(lib, lib.pl_lightning_chunks(self._p(proj), ld, H, d, dv, self._p(decay), self._p(buf), numbers, self._p(state),
+        buf = torch.empty(2 * numbers * H * dv * (-(-d // 16) * 16), dtype=torch.float32, device=self.device)
+        _check(lib, lib.pl_lightning_chunks(self._p(proj), ld, T, H, d, dv, self._p(decay), self._p(buf), numbers, self._p(state),
                                             c_longlong(state.shape[1]), self._p(ctx.cu_seqlens_q), self._p(ctx.state_slots), ctx.num_seqs,
                                             self._p(o), self._stream))
-        self.launches += 3
+        self.launches += 4
         return o
 
     def row_norm_gate(self, o, proj, g_col0, norm_w, eps) -> torch.Tensor:

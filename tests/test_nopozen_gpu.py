@@ -176,7 +176,7 @@ def test_steps_of_a_padded_graph_take_any_portions(ops):
     for padded, longest in ((False, 300), (True, 1)):
         ctx = types.SimpleNamespace(num_seqs=3, cu_seqlens_q=dev([0, 300, 305, 375]), state_slots=dev([2, 0, 1]), max_q_len=longest, padded=padded)
         state = torch.zeros(3, H * d * d, device="cuda")
-        outs.append((ops.fixed_decay_attention(proj, H, d, d, decay, state, ctx).cpu(), state.cpu()))
+        outs.append((ops.fixed_decay_attention(proj.clone(), H, d, d, decay, state, ctx).cpu(), state.cpu()))     # (silu is in place)
     assert torch.equal(outs[0][0], outs[1][0]) and torch.equal(outs[0][1], outs[1][1])
 
 
