@@ -135,6 +135,9 @@ class CacheStorage:
         states = self._state_tensors()
         if not states:
             return
+        if len(slots) == 1 and all(state.is_contiguous() for state in states):
+            torch._foreach_zero_([state[slots[0]] for state in states])     # one launch for all of them
+            return
         idx = torch.tensor(slots, dtype=torch.long).to(self.device, non_blocking=True)
         for state in states:
             state.index_fill_(0, idx, 0)

@@ -371,8 +371,7 @@ __device__ __forceinline__ float4 shfl_quad(float4 v, int lane) {
 // The quads of a head (lane l: quads l, l + 32) after the rotation in halves; a quad's partner sits in another lane or in this
 // lane's other quad.  Called by whole warps.
 template <int NQ>
-__device__ __forceinline__ void turn_quads(const float2* cs, int rd, int lane, float4 (&v)[NQ]) {
-    float4 other[NQ];
+__device__ __forceinline__ void partner_quads(int rd, int lane, const float4 (&v)[NQ], float4 (&other)[NQ]) {
     const int hq = rd >> 3;                                             // quads of half the rotated elements
 #pragma unroll
     for (int i = 0; i < NQ; ++i) {
@@ -384,39 +383,80 @@ __device__ __forceinline__ void turn_quads(const float2* cs, int rd, int lane, f
             if (pq >= 32) other[i] = b;
         }
     }
+}
+
+template <int NQ>
+__device__ __forceinline__ void turn_quads(const float2* cs, int rd, int lane, float4 (&v)[NQ]) {
+    float4 other[NQ];
+    partner_quads<NQ>(rd, lane, v, other);
 #pragma unroll
     for (int i = 0; i < NQ; ++i) v[i] = turned_quad(cs, rd, (lane + 32 * i) * 4, v[i], other[i]);
+}
+
+// The factors of a quad and of its partner in the rotation of elements c .. c+3; behind the rotated part 1 and 0.
+__device__ __forceinline__ void turn_factors(const float2* cs, int rd, int c, float4& cosine, float4& sine) {
+    cosine = make_float4(1.f, 1.f, 1.f, 1.f), sine = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c >= rd) return;
+    const int half = rd >> 1;
+    const bool second = c >= half;
+    const float4 t01 = *reinterpret_cast<const float4*>(cs + (second ? c - half : c));
+    const float4 t23 = *reinterpret_cast<const float4*>(cs + (second ? c - half : c) + 2);
+    const float sg = second ? 1.f : -1.f;
+    cosine = make_float4(t01.x, t01.z, t23.x, t23.z);
+    sine = make_float4(sg * t01.y, sg * t01.w, sg * t23.y, sg * t23.w);
+}
+
+__device__ __forceinline__ float4 turned_by(float4 v, float4 other, float4 c, float4 s) {
+    return make_float4(fmaf(v.x, c.x, other.x * s.x), fmaf(v.y, c.y, other.y * s.y), fmaf(v.z, c.z, other.z * s.z), fmaf(v.w, c.w, other.w * s.w));
 }
 
 template <typename T, int NQ, int HP>
 __global__ void __launch_bounds__(256) unit_qkv_quads_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ bias, float eps,
                                                              const float* __restrict__ qw, const float* __restrict__ kw, RotTable rot,
                                                              T* __restrict__ q_out, T* __restrict__ kv, SlotArgs sa, int nh, int nkv, int d,
-                                                             int dv, int D, int write, long long items) {
+                                                             int dv, int D, int write, int tokens) {
+    // grid: (groups of HP heads, tokens / 8)
     pdl_launch_dependents();
-    const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
-    if (item >= items) {
+    const int t = blockIdx.y * 8 + (threadIdx.x >> 5);
+    if (t >= tokens) {
         pdl_wait();
         return;
     }
-    const int lane = threadIdx.x & 31, heads = nh + 2 * nkv, groups = (heads + HP - 1) / HP;
-    const int t = (int)(item / groups), head0 = (int)(item - (long long)t * groups) * HP;
+    const int lane = threadIdx.x & 31, heads = nh + 2 * nkv, head0 = blockIdx.x * HP;
     const int s = sa.token_seq[t], pos = sa.positions[t];
-    const long long slot = write && s >= 0 ? key_slot(sa, t, s, pos, nkv, D) : -1;
-    const float2* cs = rot.table != nullptr && s >= 0 && pos >= 0 && pos < rot.len ? rot.table + (size_t)pos * (rot.rd >> 1) : nullptr;
     pdl_wait();
+    // (the row is read whatever the token is, so that its loads do not wait for the token's metadata)
     const T* row = proj + (size_t)t * ld;
     float4 v[HP][NQ];
 #pragma unroll
     for (int p = 0; p < HP; ++p) {
         const int head = head0 + p;
         const bool is_v = head >= nh + nkv;
-        const int n = head >= heads || s < 0 ? 0 : is_v ? dv : d, col = is_v ? (nh + nkv) * d + (head - nh - nkv) * dv : head * d;
+        const int n = head >= heads ? 0 : is_v ? dv : d, col = is_v ? (nh + nkv) * d + (head - nh - nkv) * dv : head * d;
 #pragma unroll
         for (int i = 0; i < NQ; ++i) {
             const int c = (lane + 32 * i) * 4;
             v[p][i] = c < n ? Quad4<T>::load(row + col + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-            if (bias != nullptr && c < n) {
+        }
+    }
+    const long long slot = write && s >= 0 ? key_slot(sa, t, s, pos, nkv, D) : -1;
+    const bool turn = rot.table != nullptr && s >= 0 && pos >= 0 && pos < rot.len && head0 < nh + nkv;
+    float4 cosine[NQ], sine[NQ];                                        // of this lane's elements, one token for all heads
+    if (turn) {
+        const float2* cs = rot.table + (size_t)pos * (rot.rd >> 1);
+#pragma unroll
+        for (int i = 0; i < NQ; ++i) turn_factors(cs, rot.rd, (lane + 32 * i) * 4, cosine[i], sine[i]);
+    }
+#pragma unroll
+    for (int p = 0; p < HP; ++p) {
+        const int head = head0 + p;
+        const bool is_v = head >= nh + nkv;
+        const int n = head >= heads ? 0 : is_v ? dv : d, col = is_v ? (nh + nkv) * d + (head - nh - nkv) * dv : head * d;
+#pragma unroll
+        for (int i = 0; i < NQ; ++i) {
+            const int c = (lane + 32 * i) * 4;
+            if (s < 0) v[p][i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (bias != nullptr && c < n && s >= 0) {
                 const float4 b = Quad4<float>::load(bias + col + c);
                 v[p][i] = make_float4(v[p][i].x + b.x, v[p][i].y + b.y, v[p][i].z + b.z, v[p][i].w + b.w);
             }
@@ -442,7 +482,12 @@ __global__ void __launch_bounds__(256) unit_qkv_quads_kernel(const T* __restrict
                 }
             }
             f = 1.0f / sqrtf(warp_sum(sq) / (float)d + eps);
-            if (cs != nullptr) turn_quads<NQ>(cs, rot.rd, lane, v[p]);
+            if (turn) {
+                float4 other[NQ];
+                partner_quads<NQ>(rot.rd, lane, v[p], other);
+#pragma unroll
+                for (int i = 0; i < NQ; ++i) v[p][i] = turned_by(v[p][i], other[i], cosine[i], sine[i]);
+            }
         }
         T* dst = is_q ? q_out + ((size_t)t * nh + head) * D
                  : slot >= 0 ? kv + slot + (size_t)(is_v ? head - nkv - nh : head - nh) * sa.ps * D + (is_v ? (size_t)nkv * sa.ps * D : 0) : nullptr;
@@ -503,11 +548,12 @@ static int launch_unit_qkv(const void* proj, int T_, int ld, const float* bias, 
                            void* q_out, void* kv, SlotArgs sa, int nh, int nkv, int d, int dv, int D, int write, int vec,
                            cudaStream_t stream) {
     const int heads = nh + 2 * nkv, hp = vec && T_ >= 256 ? (D <= 128 ? 4 : 2) : 1;
-    const long long items = (long long)T_ * ((heads + hp - 1) / hp), blocks = (items + 7) / 8;
-    PL_REQUIRE(blocks < (1ll << 31), "unit_qkv_write: %d tokens", T_);
+    const long long items = (long long)T_ * heads, blocks = (items + 7) / 8;
+    const dim3 grid((heads + hp - 1) / hp, (T_ + 7) / 8);
+    PL_REQUIRE(blocks < (1ll << 31) && grid.y <= 65535, "unit_qkv_write: %d tokens", T_);
 #define UNIT_QUADS(NQ, HP)                                                                                                              \
-    PL_CUDA(launch_pdl(unit_qkv_quads_kernel<T, NQ, HP>, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)proj, ld, bias, eps, qw, kw, rot, \
-                       (T*)q_out, (T*)kv, sa, nh, nkv, d, dv, D, write, items))
+    PL_CUDA(launch_pdl(unit_qkv_quads_kernel<T, NQ, HP>, grid, dim3(256), 0, stream, (const T*)proj, ld, bias, eps, qw, kw, rot, \
+                       (T*)q_out, (T*)kv, sa, nh, nkv, d, dv, D, write, T_))
     if (!vec)
         PL_CUDA(launch_pdl(unit_qkv_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)proj, ld, bias, eps, qw, kw, rot,
                            (T*)q_out, (T*)kv, sa, nh, nkv, d, dv, D, write, items));
@@ -636,8 +682,23 @@ __global__ void __launch_bounds__(256) conv_qkv_kernel(const T* __restrict__ pro
 // consecutive tokens of a head, whose inputs (and the TAPS - 1 in front) it loads together.
 constexpr int QC_STRIP = 8;
 
+// Four elements as they are stored.
+template <typename T> struct RawQuad;
+template <> struct RawQuad<float> {
+    float4 v;
+    __device__ __forceinline__ void load(const float* p) { v = *reinterpret_cast<const float4*>(p); }
+    __device__ __forceinline__ void set(float4 x) { v = x; }
+    __device__ __forceinline__ float4 get() const { return v; }
+};
+template <> struct RawQuad<__nv_bfloat16> {
+    uint2 v;
+    __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint2*>(p); }
+    __device__ __forceinline__ void set(float4 x) { Quad4<__nv_bfloat16>::store(reinterpret_cast<__nv_bfloat16*>(&v), x); }
+    __device__ __forceinline__ float4 get() const { return Quad4<__nv_bfloat16>::load(reinterpret_cast<const __nv_bfloat16*>(&v)); }
+};
+
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(256) conv_qkv_strip_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ cw,
+__global__ void __launch_bounds__(256, 3) conv_qkv_strip_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ cw,
                                                              float* __restrict__ state, long long state_stride, const int* __restrict__ cu_q,
                                                              const int* __restrict__ slots, RotTable rot, T* __restrict__ q_out,
                                                              T* __restrict__ kv, SlotArgs sa, int nh, int nkv, int d, int dv, int D, int write) {
@@ -659,39 +720,41 @@ __global__ void __launch_bounds__(256) conv_qkv_strip_kernel(const T* __restrict
     const T* in = proj + (size_t)q0 * ld + col;
     const int t0 = t_lo + warp * QC_STRIP;
     if (t0 < nq) {
-        float4 u[QC_STRIP + hist];
+        // (what the state holds of older inputs are values of T)
+        RawQuad<T> u[QC_STRIP + hist];
 #pragma unroll
         for (int r = 0; r < QC_STRIP + hist; ++r) {
             const int src = t0 - hist + r;
-            u[r] = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (c < n && src < nq)
-                u[r] = src >= 0 ? Quad4<T>::load(in + (size_t)src * ld + c) : *reinterpret_cast<const float4*>(st + (size_t)(hist + src) * C + c);
+            if (c < n && src >= 0 && src < nq) u[r].load(in + (size_t)src * ld + c);
+            else u[r].set(make_float4(0.f, 0.f, 0.f, 0.f));
+        }
+        if (t0 < hist && c < n) {
+#pragma unroll
+            for (int r = 0; r < hist; ++r)
+                if (t0 - hist + r < 0) u[r].set(*reinterpret_cast<const float4*>(st + (size_t)(t0 + r) * C + c));
         }
         const int pos0 = sa.positions[q0 + t0];                         // (a request's tokens stand at consecutive positions)
-        T* dst[QC_STRIP];
-#pragma unroll
-        for (int i = 0; i < QC_STRIP; ++i) {
-            dst[i] = nullptr;
-            if (t0 + i >= nq) continue;
-            if (is_q) {
-                dst[i] = q_out + ((size_t)(q0 + t0 + i) * nh + head) * D;
-            } else if (write) {
-                const long long at = key_slot(sa, q0 + t0 + i, s, pos0 + i, nkv, D);
-                if (at >= 0) dst[i] = kv + at + (size_t)(is_v ? head - nkv - nh : head - nh) * sa.ps * D + (is_v ? (size_t)nkv * sa.ps * D : 0);
-            }
-        }
 #pragma unroll
         for (int i = 0; i < QC_STRIP; ++i) {
             if (t0 + i >= nq) break;
+            T* dst = nullptr;
+            if (is_q) {
+                dst = q_out + ((size_t)(q0 + t0 + i) * nh + head) * D;
+            } else if (write) {
+                const long long at = key_slot(sa, q0 + t0 + i, s, pos0 + i, nkv, D);
+                if (at >= 0) dst = kv + at + (size_t)(is_v ? head - nkv - nh : head - nh) * sa.ps * D + (is_v ? (size_t)nkv * sa.ps * D : 0);
+            }
             float4 v[1] = {make_float4(0.f, 0.f, 0.f, 0.f)};
 #pragma unroll
-            for (int k = 0; k < TAPS; ++k)
-                v[0].x = fmaf(f[k].x, u[i + k].x, v[0].x), v[0].y = fmaf(f[k].y, u[i + k].y, v[0].y),
-                v[0].z = fmaf(f[k].z, u[i + k].z, v[0].z), v[0].w = fmaf(f[k].w, u[i + k].w, v[0].w);
+            for (int k = 0; k < TAPS; ++k) {
+                const float4 x = u[i + k].get();
+                v[0].x = fmaf(f[k].x, x.x, v[0].x), v[0].y = fmaf(f[k].y, x.y, v[0].y);
+                v[0].z = fmaf(f[k].z, x.z, v[0].z), v[0].w = fmaf(f[k].w, x.w, v[0].w);
+            }
             const int pos = pos0 + i;
             if (!is_v && rot.table != nullptr && pos >= 0 && pos < rot.len)
                 turn_quads<1>(rot.table + (size_t)pos * (rot.rd >> 1), rot.rd, lane, v);
-            if (dst[i] != nullptr && c < D) Quad4<T>::store(dst[i] + c, v[0]);
+            if (dst != nullptr && c < D) Quad4<T>::store(dst + c, v[0]);
         }
     }
     if (blockIdx.z != 0 || hist == 0) return;
