@@ -361,8 +361,8 @@ PL_EXPORT int pl_normed_qkv_write(const void* proj, int dtype, int T, int ld, co
 // [d] if there is one (qw, kw: one for all heads); with a table `rot`, q and k are then rotated by the token's position over
 // the table's leading elements of each head.  Q out [T, nh*D], K and V to the page slot, all padded to D with zeros.  A warp
 // per (token, head): heads 0..nh-1 are queries, then keys, then values.
-// Vector form: sizes are multiples of 4, a lane holds NQ quads of a head (D <= 128 NQ), a warp takes HP heads of a token whose
-// loads go out together; the rotation's quads do not straddle its halves.
+// Vector form: sizes are multiples of 4, LPH lanes share a head and hold NQ quads of it each (D <= 4 LPH NQ), a warp takes
+// HP * 32 / LPH heads of a token whose loads go out together; the rotation's quads do not straddle its halves.
 __device__ __forceinline__ float4 shfl_quad(float4 v, int lane) {
     return make_float4(__shfl_sync(0xffffffffu, v.x, lane), __shfl_sync(0xffffffffu, v.y, lane), __shfl_sync(0xffffffffu, v.z, lane),
                        __shfl_sync(0xffffffffu, v.w, lane));
@@ -370,17 +370,18 @@ __device__ __forceinline__ float4 shfl_quad(float4 v, int lane) {
 
 // The quads of a head (lane l: quads l, l + 32) after the rotation in halves; a quad's partner sits in another lane or in this
 // lane's other quad.  Called by whole warps.
-template <int NQ>
+template <int LPH, int NQ>
 __device__ __forceinline__ void partner_quads(int rd, int lane, const float4 (&v)[NQ], float4 (&other)[NQ]) {
     const int hq = rd >> 3;                                             // quads of half the rotated elements
+    const int base = threadIdx.x & 31 & ~(LPH - 1);                     // first lane of this head's
 #pragma unroll
     for (int i = 0; i < NQ; ++i) {
-        const int quad = lane + 32 * i;
+        const int quad = lane + LPH * i;
         const int pq = quad >= 2 * hq ? quad : quad >= hq ? quad - hq : quad + hq;
-        other[i] = shfl_quad(v[0], pq & 31);
+        other[i] = shfl_quad(v[0], base + (pq & (LPH - 1)));
         if (NQ > 1) {
-            const float4 b = shfl_quad(v[NQ - 1], pq & 31);
-            if (pq >= 32) other[i] = b;
+            const float4 b = shfl_quad(v[NQ - 1], base + (pq & (LPH - 1)));
+            if (pq >= LPH) other[i] = b;
         }
     }
 }
@@ -388,7 +389,7 @@ __device__ __forceinline__ void partner_quads(int rd, int lane, const float4 (&v
 template <int NQ>
 __device__ __forceinline__ void turn_quads(const float2* cs, int rd, int lane, float4 (&v)[NQ]) {
     float4 other[NQ];
-    partner_quads<NQ>(rd, lane, v, other);
+    partner_quads<32, NQ>(rd, lane, v, other);
 #pragma unroll
     for (int i = 0; i < NQ; ++i) v[i] = turned_quad(cs, rd, (lane + 32 * i) * 4, v[i], other[i]);
 }
@@ -410,19 +411,20 @@ __device__ __forceinline__ float4 turned_by(float4 v, float4 other, float4 c, fl
     return make_float4(fmaf(v.x, c.x, other.x * s.x), fmaf(v.y, c.y, other.y * s.y), fmaf(v.z, c.z, other.z * s.z), fmaf(v.w, c.w, other.w * s.w));
 }
 
-template <typename T, int NQ, int HP>
+template <typename T, int LPH, int NQ, int HP>
 __global__ void __launch_bounds__(256) unit_qkv_quads_kernel(const T* __restrict__ proj, int ld, const float* __restrict__ bias, float eps,
                                                              const float* __restrict__ qw, const float* __restrict__ kw, RotTable rot,
                                                              T* __restrict__ q_out, T* __restrict__ kv, SlotArgs sa, int nh, int nkv, int d,
                                                              int dv, int D, int write, int tokens) {
-    // grid: (groups of HP heads, tokens / 8)
+    // grid: (groups of HP * 32 / LPH heads, tokens / 8); LPH lanes share a head, so a warp has 32 / LPH of them side by side
+    constexpr int SIDE = 32 / LPH;
     pdl_launch_dependents();
     const int t = blockIdx.y * 8 + (threadIdx.x >> 5);
     if (t >= tokens) {
         pdl_wait();
         return;
     }
-    const int lane = threadIdx.x & 31, heads = nh + 2 * nkv, head0 = blockIdx.x * HP;
+    const int lane = threadIdx.x % LPH, heads = nh + 2 * nkv, first = blockIdx.x * (HP * SIDE), head0 = first + (threadIdx.x & 31) / LPH;
     const int s = sa.token_seq[t], pos = sa.positions[t];
     pdl_wait();
     // (the row is read whatever the token is, so that its loads do not wait for the token's metadata)
@@ -430,31 +432,31 @@ __global__ void __launch_bounds__(256) unit_qkv_quads_kernel(const T* __restrict
     float4 v[HP][NQ];
 #pragma unroll
     for (int p = 0; p < HP; ++p) {
-        const int head = head0 + p;
+        const int head = head0 + p * SIDE;
         const bool is_v = head >= nh + nkv;
         const int n = head >= heads ? 0 : is_v ? dv : d, col = is_v ? (nh + nkv) * d + (head - nh - nkv) * dv : head * d;
 #pragma unroll
         for (int i = 0; i < NQ; ++i) {
-            const int c = (lane + 32 * i) * 4;
+            const int c = (lane + LPH * i) * 4;
             v[p][i] = c < n ? Quad4<T>::load(row + col + c) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
     }
     const long long slot = write && s >= 0 ? key_slot(sa, t, s, pos, nkv, D) : -1;
-    const bool turn = rot.table != nullptr && s >= 0 && pos >= 0 && pos < rot.len && head0 < nh + nkv;
+    const bool turn = rot.table != nullptr && s >= 0 && pos >= 0 && pos < rot.len && first < nh + nkv;
     float4 cosine[NQ], sine[NQ];                                        // of this lane's elements, one token for all heads
     if (turn) {
         const float2* cs = rot.table + (size_t)pos * (rot.rd >> 1);
 #pragma unroll
-        for (int i = 0; i < NQ; ++i) turn_factors(cs, rot.rd, (lane + 32 * i) * 4, cosine[i], sine[i]);
+        for (int i = 0; i < NQ; ++i) turn_factors(cs, rot.rd, (lane + LPH * i) * 4, cosine[i], sine[i]);
     }
 #pragma unroll
     for (int p = 0; p < HP; ++p) {
-        const int head = head0 + p;
+        const int head = head0 + p * SIDE;
         const bool is_v = head >= nh + nkv;
         const int n = head >= heads ? 0 : is_v ? dv : d, col = is_v ? (nh + nkv) * d + (head - nh - nkv) * dv : head * d;
 #pragma unroll
         for (int i = 0; i < NQ; ++i) {
-            const int c = (lane + 32 * i) * 4;
+            const int c = (lane + LPH * i) * 4;
             if (s < 0) v[p][i] = make_float4(0.f, 0.f, 0.f, 0.f);
             if (bias != nullptr && c < n && s >= 0) {
                 const float4 b = Quad4<float>::load(bias + col + c);
@@ -464,37 +466,45 @@ __global__ void __launch_bounds__(256) unit_qkv_quads_kernel(const T* __restrict
     }
 #pragma unroll
     for (int p = 0; p < HP; ++p) {
-        const int head = head0 + p;
-        if (head >= heads) break;
+        const int head = head0 + p * SIDE;
+        if (first + p * SIDE >= heads) break;                           // (whole warps leave)
         const bool is_q = head < nh, is_v = head >= nh + nkv;
         float f = 1.f;
-        if (!is_v) {
+        if (first + p * SIDE < nh + nkv) {
             const float* hw = is_q ? qw : kw;
             float sq = 0.f;
+            float4 x[NQ];
 #pragma unroll
             for (int i = 0; i < NQ; ++i) {
-                float4& x = v[p][i];
-                sq += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
-                const int c = (lane + 32 * i) * 4;
+                x[i] = v[p][i];
+                sq += x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
+                const int c = (lane + LPH * i) * 4;
                 if (hw != nullptr && c < d) {
                     const float4 w = Quad4<float>::load(hw + c);
-                    x = make_float4(x.x * w.x, x.y * w.y, x.z * w.z, x.w * w.w);
+                    x[i] = make_float4(x[i].x * w.x, x[i].y * w.y, x[i].z * w.z, x[i].w * w.w);
                 }
             }
-            f = 1.0f / sqrtf(warp_sum(sq) / (float)d + eps);
+#pragma unroll
+            for (int o = LPH / 2; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
             if (turn) {
                 float4 other[NQ];
-                partner_quads<NQ>(rot.rd, lane, v[p], other);
+                partner_quads<LPH, NQ>(rot.rd, lane, x, other);
 #pragma unroll
-                for (int i = 0; i < NQ; ++i) v[p][i] = turned_by(v[p][i], other[i], cosine[i], sine[i]);
+                for (int i = 0; i < NQ; ++i) x[i] = turned_by(x[i], other[i], cosine[i], sine[i]);
+            }
+            if (!is_v) {                                                // (a value head beside a key head in this warp)
+                f = 1.0f / sqrtf(sq / (float)d + eps);
+#pragma unroll
+                for (int i = 0; i < NQ; ++i) v[p][i] = x[i];
             }
         }
+        if (head >= heads) continue;
         T* dst = is_q ? q_out + ((size_t)t * nh + head) * D
                  : slot >= 0 ? kv + slot + (size_t)(is_v ? head - nkv - nh : head - nh) * sa.ps * D + (is_v ? (size_t)nkv * sa.ps * D : 0) : nullptr;
         if (dst == nullptr) continue;
 #pragma unroll
         for (int i = 0; i < NQ; ++i) {
-            const int c = (lane + 32 * i) * 4;
+            const int c = (lane + LPH * i) * 4;
             const float4 x = v[p][i];
             if (c < D) Quad4<T>::store(dst + c, make_float4(x.x * f, x.y * f, x.z * f, x.w * f));
         }
@@ -547,20 +557,22 @@ template <typename T>
 static int launch_unit_qkv(const void* proj, int T_, int ld, const float* bias, float eps, const float* qw, const float* kw, RotTable rot,
                            void* q_out, void* kv, SlotArgs sa, int nh, int nkv, int d, int dv, int D, int write, int vec,
                            cudaStream_t stream) {
-    const int heads = nh + 2 * nkv, hp = vec && T_ >= 256 ? (D <= 128 ? 4 : 2) : 1;
+    const int heads = nh + 2 * nkv, hp = vec && T_ >= 256 ? (D <= 128 ? 4 : 2) : 1, side = vec && D <= 64 ? 2 : 1;
     const long long items = (long long)T_ * heads, blocks = (items + 7) / 8;
-    const dim3 grid((heads + hp - 1) / hp, (T_ + 7) / 8);
+    const dim3 grid((heads + hp * side - 1) / (hp * side), (T_ + 7) / 8);
     PL_REQUIRE(blocks < (1ll << 31) && grid.y <= 65535, "unit_qkv_write: %d tokens", T_);
-#define UNIT_QUADS(NQ, HP)                                                                                                              \
-    PL_CUDA(launch_pdl(unit_qkv_quads_kernel<T, NQ, HP>, grid, dim3(256), 0, stream, (const T*)proj, ld, bias, eps, qw, kw, rot, \
+#define UNIT_QUADS(LPH, NQ, HP)                                                                                                         \
+    PL_CUDA(launch_pdl(unit_qkv_quads_kernel<T, LPH, NQ, HP>, grid, dim3(256), 0, stream, (const T*)proj, ld, bias, eps, qw, kw, rot, \
                        (T*)q_out, (T*)kv, sa, nh, nkv, d, dv, D, write, T_))
     if (!vec)
         PL_CUDA(launch_pdl(unit_qkv_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, stream, (const T*)proj, ld, bias, eps, qw, kw, rot,
                            (T*)q_out, (T*)kv, sa, nh, nkv, d, dv, D, write, items));
-    else if (D <= 128) {
-        if (hp == 4) UNIT_QUADS(1, 4); else UNIT_QUADS(1, 1);
+    else if (D <= 64) {
+        if (hp == 4) UNIT_QUADS(16, 1, 4); else UNIT_QUADS(16, 1, 1);
+    } else if (D <= 128) {
+        if (hp == 4) UNIT_QUADS(32, 1, 4); else UNIT_QUADS(32, 1, 1);
     } else {
-        if (hp == 2) UNIT_QUADS(2, 2); else UNIT_QUADS(2, 1);
+        if (hp == 2) UNIT_QUADS(32, 2, 2); else UNIT_QUADS(32, 2, 1);
     }
 #undef UNIT_QUADS
     return 0;
